@@ -35,6 +35,71 @@ DLLM_EXPORT int dllm_embed_scaled(float* out, const void* table, const int* toke
   return DLLM_BAD_ARGUMENT;
 }
 
+// The same with a position vector added: entry 2i of the row of a token at position p gets sin(p f_i), entry 2i + 1
+// cos(p f_i). freqs[i] = (f_i in float32, what that rounding took off f_i): p f_i is formed as a float32 product, its own
+// rounding (exact, by a fused multiply-add) and p times the rest, and the small part turns the sine and cosine of the
+// large one by the addition theorem.
+template <typename T>
+__global__ void embed_sinusoid_kernel(float* __restrict__ out, const T* __restrict__ table,
+                                      const int* __restrict__ tokens, const int* __restrict__ positions,
+                                      const float2* __restrict__ freqs, int hidden, int vocab, float scale,
+                                      int* __restrict__ status) {
+  int row = blockIdx.x;
+  pdl_launch_dependents();
+  pdl_wait();
+  int token = tokens[row];
+  if (token < 0 || token >= vocab) {
+    if (threadIdx.x == 0) *(volatile int*)status = 64;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[(size_t)row * hidden + i] = 0.f;
+    return;
+  }
+  const T* src = table + (size_t)token * hidden;
+  const float p = (float)positions[row];
+  for (int i = threadIdx.x; 2 * i < hidden; i += blockDim.x) {
+    float2 f = freqs[i];
+    float angle = p * f.x;
+    float rest = fmaf(p, f.x, -angle) + p * f.y;
+    float s, c;
+    sincosf(angle, &s, &c);
+    float curve = 1.0f - 0.5f * rest * rest;
+    float* dst = out + (size_t)row * hidden + 2 * i;
+    dst[0] = to_float(src[2 * i]) * scale + fmaf(rest, c, s * curve);
+    if (2 * i + 1 < hidden) dst[1] = to_float(src[2 * i + 1]) * scale + fmaf(-rest, s, c * curve);
+  }
+}
+
+DLLM_EXPORT int dllm_embed_sinusoid(float* out, const void* table, const int* tokens, const int* positions,
+                                    const float* freqs, int rows, int hidden, int vocab, int dtype, float scale,
+                                    int* status, cudaStream_t stream) {
+  if (rows <= 0) return DLLM_OK;
+  if (hidden <= 0 || vocab <= 0 || !out || !table || !tokens || !positions || !freqs) return DLLM_BAD_ARGUMENT;
+  int threads = hidden >= 512 ? 256 : 64;
+  if (dtype == DLLM_F32)
+    return dllm_launch_pdl(embed_sinusoid_kernel<float>, dim3(rows), dim3(threads), 0, stream, out, (const float*)table,
+                           tokens, positions, (const float2*)freqs, hidden, vocab, scale, status);
+  if (dtype == DLLM_BF16)
+    return dllm_launch_pdl(embed_sinusoid_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, out,
+                           (const __nv_bfloat16*)table, tokens, positions, (const float2*)freqs, hidden, vocab, scale,
+                           status);
+  return DLLM_BAD_ARGUMENT;
+}
+
+// ---- x <- cap tanh(x / cap), in place (logits) --------------------------------------------------------------------
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long total, float cap, float inv) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total;
+       i += (long long)gridDim.x * blockDim.x)
+    x[i] = cap * tanhf(x[i] * inv);
+}
+
+DLLM_EXPORT int dllm_softcap(float* x, long long total, float cap, cudaStream_t stream) {
+  if (total <= 0) return DLLM_OK;
+  if (x == nullptr || !(cap > 0.f)) return DLLM_BAD_ARGUMENT;
+  int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  return dllm_launch_pdl(softcap_kernel, dim3(blocks), dim3(256), 0, stream, x, total, cap, 1.0f / cap);
+}
+
 DLLM_EXPORT int dllm_embed(float* out, const void* table, const int* tokens, int rows, int hidden, int vocab,
                            int dtype, int* status, cudaStream_t stream) {
   return dllm_embed_scaled(out, table, tokens, rows, hidden, vocab, dtype, 1.0f, status, stream);

@@ -3,6 +3,7 @@
 //
 //   decayed outer products:  S <- decay_h S + k_t v_t^T;                          o_t = S^T q_t
 //   gated delta rule:        S <- g_t S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+//   the same by channels:    S <- diag(g_t) S, a decay per key channel (row of S), then as the gated delta rule
 //   gated outer products:    S <- a_t S + b_t k_t v_t^T  (a_t, b_t per token and head);   o_t = S^T q_t, and the
 //                            same sum with v = 1 as one more column of S (the normaliser n_t), read out as n_t . q_t
 //
@@ -65,6 +66,9 @@ struct ScanArgs {
   // gated outer products: aux holds per token [a (heads) | b (heads) | -]; the state has vdim + 1 columns, the last
   // one written with v = 1, and its read-out goes to nq [tokens][heads]
   float* nq;
+  // delta rule by channels: a token's decays of head h start at decays + token * decay_stride + h * dim
+  const float* decays;
+  int decay_stride;
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -72,7 +76,8 @@ __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem) : "memory");
 }
 
-// MODE 0: decayed outer products; MODE 1: gated delta rule; MODE 2: gated outer products. TOKENS: tokens a stage. LPC lanes share a column (8 or
+// MODE 0: decayed outer products; MODE 1: gated delta rule; MODE 2: gated outer products; MODE 3: the delta rule with a
+// decay per row of S (whose stage rows hold the decays between q and v). TOKENS: tokens a stage. LPC lanes share a column (8 or
 // 16), each with RPL rows of it: the block has 16 * LPC threads. Few lanes a column mean few shuffles and few
 // instructions a token; many lanes mean more warps to hide latency behind, which is what a step with few sequences
 // and heads needs (one warp per scheduler issues a dependent instruction every four cycles and no faster).
@@ -81,9 +86,10 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   constexpr int DIMP = RPL * LPC;  // rows a stage holds per token (the head's dim rounded up)
   constexpr int CPW = 32 / LPC;    // columns a warp owns
   constexpr int SCAN_THREADS = SCAN_COLS * LPC;
-  constexpr int PER_TOKEN = 2 * DIMP + SCAN_COLS + 4;
+  constexpr int V_AT = (MODE == 3 ? 3 : 2) * DIMP;  // where the values start in a stage row
+  constexpr int PER_TOKEN = V_AT + SCAN_COLS + 4;
   constexpr int PIECES = PER_TOKEN / 4;  // 16-byte pieces of a token's stage row
-  extern __shared__ __align__(16) float stage[];  // [STAGES][TOKENS][PER_TOKEN]: k | q | v (16 columns) | g, beta, k.q, -
+  extern __shared__ __align__(16) float stage[];  // [STAGES][TOKENS][PER_TOKEN]: k | q | (decays) | v (16 columns) | g, beta, k.q, -
   pdl_launch_dependents();
   const int head = blockIdx.y, seq = blockIdx.z, col0 = blockIdx.x * SCAN_COLS;
   const int qk_head = head / (a.heads / a.qk_heads);
@@ -114,6 +120,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
       const float* k0 = a.k + (size_t)(first + t0) * a.stride + qk_head * a.dim;
       const float* q0 = a.q + (size_t)(first + t0) * a.stride + qk_head * a.dim;
       const float* v0 = a.v + (size_t)(first + t0) * a.stride + head * a.vdim + col0;
+      const float* d0 = MODE == 3 ? a.decays + (size_t)(first + t0) * a.decay_stride + head * a.dim : nullptr;
       for (int i = tid; i < here * PIECES; i += SCAN_THREADS) {
         int t = i / PIECES, e = (i - t * PIECES) * 4;
         float* to = dst + t * PER_TOKEN + e;
@@ -123,8 +130,10 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           if (e < a.dim) src = k0 + row + e;
         } else if (e < 2 * DIMP) {
           if (e - DIMP < a.dim) src = q0 + row + (e - DIMP);
-        } else if (e < 2 * DIMP + SCAN_COLS) {
-          if (col0 + e - 2 * DIMP < a.vdim) src = v0 + row + (e - 2 * DIMP);
+        } else if (MODE == 3 && e < 3 * DIMP) {
+          if (e - 2 * DIMP < a.dim) src = d0 + t * a.decay_stride + (e - 2 * DIMP);
+        } else if (e < V_AT + SCAN_COLS) {
+          if (col0 + e - V_AT < a.vdim) src = v0 + row + (e - V_AT);
         } else if (MODE >= 1) {
           const float* aux = a.aux + (size_t)(first + t0 + t) * a.aux_stride;
           cp_async4(to, aux + head);
@@ -144,11 +153,13 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           if (e < a.dim) src = a.k + token * a.stride + qk_head * a.dim + e;
         } else if (e < 2 * DIMP) {
           if (e - DIMP < a.dim) src = a.q + token * a.stride + qk_head * a.dim + (e - DIMP);
-        } else if (e < 2 * DIMP + SCAN_COLS) {
-          int c = col0 + e - 2 * DIMP;
+        } else if (MODE == 3 && e < 3 * DIMP) {
+          if (e - 2 * DIMP < a.dim) src = a.decays + token * a.decay_stride + head * a.dim + (e - 2 * DIMP);
+        } else if (e < V_AT + SCAN_COLS) {
+          int c = col0 + e - V_AT;
           if (c < a.vdim) src = a.v + token * a.stride + head * a.vdim + c;
         } else if (MODE >= 1) {
-          int which = e - 2 * DIMP - SCAN_COLS;
+          int which = e - V_AT - SCAN_COLS;
           if (which == 0) src = a.aux + token * a.aux_stride + head;
           else if (which == 1) src = a.aux + token * a.aux_stride + a.heads + head;
           else if (which == 2) src = a.aux + token * a.aux_stride + 2 * a.heads + qk_head;
@@ -271,8 +282,8 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
       const float* row = base + t * PER_TOKEN;
       float o;
       {
-        float v = row[2 * DIMP + warp * CPW + cc];
-        float g = row[2 * DIMP + SCAN_COLS], beta = row[2 * DIMP + SCAN_COLS + 1], kq = row[2 * DIMP + SCAN_COLS + 2];
+        float v = row[V_AT + warp * CPW + cc];
+        float g = MODE == 3 ? 1.f : row[V_AT + SCAN_COLS], beta = row[V_AT + SCAN_COLS + 1], kq = row[V_AT + SCAN_COLS + 2];
         float2 kk[RPL / 2];
         float2 sk2 = make_float2(0.f, 0.f), sq2 = make_float2(0.f, 0.f);  // S^T k and S^T q before this token
 #pragma unroll
@@ -282,6 +293,12 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           kk[j / 2] = make_float2(k4.x, k4.y);
           kk[j / 2 + 1] = make_float2(k4.z, k4.w);
           float2 s01 = make_float2(S[j], S[j + 1]), s23 = make_float2(S[j + 2], S[j + 3]);
+          if (MODE == 3) {  // the rows shrink first: what follows reads and moves on the shrunk state
+            float4 g4 = *reinterpret_cast<const float4*>(row + 2 * DIMP + rg * RPL + j);
+            s01 = __fmul2_rn(s01, make_float2(g4.x, g4.y));
+            s23 = __fmul2_rn(s23, make_float2(g4.z, g4.w));
+            S[j] = s01.x; S[j + 1] = s01.y; S[j + 2] = s23.x; S[j + 3] = s23.y;
+          }
           sk2 = __ffma2_rn(s01, kk[j / 2], sk2);
           sq2 = __ffma2_rn(s01, make_float2(q4.x, q4.y), sq2);
           sk2 = __ffma2_rn(s23, kk[j / 2 + 1], sk2);
@@ -299,7 +316,8 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
         const float2 uu = make_float2(u, u), gg = make_float2(g, g);
 #pragma unroll
         for (int j = 0; j < RPL; j += 2) {
-          float2 next = __ffma2_rn(kk[j / 2], uu, __fmul2_rn(gg, make_float2(S[j], S[j + 1])));
+          float2 now = make_float2(S[j], S[j + 1]);
+          float2 next = __ffma2_rn(kk[j / 2], uu, MODE == 3 ? now : __fmul2_rn(gg, now));
           S[j] = next.x; S[j + 1] = next.y;
         }
       }
@@ -315,8 +333,8 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
 
 template <int RPL, int LPC, int MODE, int TOKENS, int STAGES>
 static int launch_scan_case(const ScanArgs& a, dim3 grid, cudaStream_t stream) {
-  size_t bytes = (size_t)STAGES * TOKENS * (2 * RPL * LPC + SCAN_COLS + 4) * sizeof(float);
-  if (MODE != 1) bytes += (size_t)TOKENS * SCAN_COLS * (LPC + 4) * sizeof(float);  // the parts of the read-out
+  size_t bytes = (size_t)STAGES * TOKENS * ((MODE == 3 ? 3 : 2) * RPL * LPC + SCAN_COLS + 4) * sizeof(float);
+  if (MODE == 0 || MODE == 2) bytes += (size_t)TOKENS * SCAN_COLS * (LPC + 4) * sizeof(float);  // the parts of the read-out
   static bool allowed = false;  // (more than 48 KB of dynamic shared memory has to be asked for once)
   if (bytes > 48 * 1024 && !allowed) {
     if (cudaFuncSetAttribute(scan_kernel<RPL, LPC, MODE, TOKENS, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -391,6 +409,25 @@ DLLM_EXPORT int dllm_delta_scan(const float* q, const float* k, const float* v, 
   a.state = state; a.cu_seqlens = cu_seqlens; a.slots = slots; a.out = out; a.aux = aux; a.aux_stride = aux_stride;
   a.out_scale = 1.0f; a.vector = scan_vector(q, k, v, stride, dim, vdim);
   return launch_scan<1>(a, sequences, longest, stream);
+}
+
+// The delta rule with a decay per key channel over the new tokens of every sequence: as `dllm_delta_scan`, with the
+// decays of a token's head h at decays + token * decay_stride + h * dim instead of aux's first column group (which is not
+// read).
+DLLM_EXPORT int dllm_channel_delta_scan(const float* q, const float* k, const float* v, int stride, const float* decays,
+                                        int decay_stride, int heads, int qk_heads, int dim, int vdim, const float* aux,
+                                        int aux_stride, float* state, const int* cu_seqlens, const int* slots,
+                                        int sequences, int longest, float* out, cudaStream_t stream) {
+  if (sequences <= 0) return DLLM_OK;
+  if (!scan_sizes_ok(heads, qk_heads, dim, vdim, stride) || sequences >= 65536 || decay_stride < heads * dim)
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!q || !k || !v || !decays || !aux || !state || !cu_seqlens || !slots || !out) return DLLM_BAD_ARGUMENT;
+  ScanArgs a = {};
+  a.q = q; a.k = k; a.v = v; a.stride = stride; a.heads = heads; a.qk_heads = qk_heads; a.dim = dim; a.vdim = vdim;
+  a.state = state; a.cu_seqlens = cu_seqlens; a.slots = slots; a.out = out; a.aux = aux; a.aux_stride = aux_stride;
+  a.decays = decays; a.decay_stride = decay_stride; a.out_scale = 1.0f;
+  a.vector = scan_vector(q, k, v, stride, dim, vdim) && ((uintptr_t)decays & 15) == 0 && decay_stride % 4 == 0;
+  return launch_scan<3>(a, sequences, longest, stream);
 }
 
 // Gated outer products over the new tokens of every sequence: S <- a_t S + b_t k_t v_t^T per head, out = S^T q times
@@ -531,6 +568,11 @@ DLLM_EXPORT int dllm_normalised_readout(void* out, const float* x, const float* 
 // sqrt(sum of squares + 1e-6) per head, q also multiplied by dim^(-1/2). Written: prepared[t][channels] and
 // aux[t] = [g (heads) | beta (heads) | k.q (qk_heads)] with beta = sigmoid(b), g = exp(-exp(A_log) softplus(a +
 // dt_bias)). In a step of single tokens (`single` != 0) the block also moves the convolution's history on.
+//
+// The delta rule by channels has a decay per head and key channel instead: with `decays` given, z = rates[t][heads x
+// dim] (rows of `rate_stride` floats) takes the place of a, dt_bias is [heads x dim], and exp(-exp(A_log_h) softplus(z +
+// dt_bias)) goes to decays[t][heads x padded]. There q, k and the decays of a head are written in rows of `padded` values
+// (dim rounded up to what the scan takes; the rest of q and k is zero, of the decays one).
 #define DELTA_MAX_TAPS 16
 
 struct DeltaPrepareArgs {
@@ -542,6 +584,9 @@ struct DeltaPrepareArgs {
   int heads, qk_heads, dim, vdim;
   float* prepared; float* aux;
   int single;
+  int padded;            // values of a head's q and k in `prepared`
+  const float* rates; int rate_stride;
+  float* decays;         // null: a decay per head
 };
 
 // A block serves one token and one unit of its channels: q/k head j (both vectors: their norms and their product), or
@@ -572,16 +617,27 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(DeltaPrepareArgs a) 
   const int qk = a.qk_heads * a.dim, channels = 2 * qk + a.heads * a.vdim, history = a.n_taps - 1;
   const float* row = a.proj + (size_t)t * a.stride;
   float* kept = a.conv_state + (size_t)slot * history * channels;
-  float* prepared = a.prepared + (size_t)t * channels;
+  float* prepared = a.prepared + (size_t)t * (2 * a.qk_heads * a.padded + a.heads * a.vdim);
   float* aux = a.aux + (size_t)t * (2 * a.heads + a.qk_heads);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (unit >= a.qk_heads) {  // the values of one head, and the head's decay and step size
     const int h = unit - a.qk_heads;
     for (int i = threadIdx.x; i < a.vdim; i += blockDim.x) {
       int ch = 2 * qk + h * a.vdim + i;
-      prepared[ch] = delta_channel(a, row, kept, channels, local, ch);
+      prepared[2 * a.qk_heads * a.padded + h * a.vdim + i] = delta_channel(a, row, kept, channels, local, ch);
     }
-    if (threadIdx.x == 0) {
+    if (a.decays != nullptr) {
+      const float rate = -expf(a.a_log[h]);
+      for (int i = threadIdx.x; i < a.padded; i += blockDim.x) {
+        float g = 1.f;
+        if (i < a.dim) {
+          float z = a.rates[(size_t)t * a.rate_stride + h * a.dim + i] + a.dt_bias[h * a.dim + i];
+          g = expf(rate * (z > 20.f ? z : log1pf(expf(z))));
+        }
+        a.decays[((size_t)t * a.heads + h) * a.padded + i] = g;
+      }
+      if (threadIdx.x == 0) aux[a.heads + h] = sigmoid_exact(row[a.b_off + h]);
+    } else if (threadIdx.x == 0) {
       float z = row[a.a_off + h] + a.dt_bias[h];
       float softplus = z > 20.f ? z : log1pf(expf(z));
       aux[h] = expf(-expf(a.a_log[h]) * softplus);
@@ -607,7 +663,11 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(DeltaPrepareArgs a) 
   for (int i = threadIdx.x; i < 2 * a.dim; i += blockDim.x) {
     float value = values[i] * scale[i < a.dim ? 0 : 1];
     values[i] = value;
-    prepared[i < a.dim ? unit * a.dim + i : qk + unit * a.dim + (i - a.dim)] = value;
+    prepared[i < a.dim ? unit * a.padded + i : (a.qk_heads + unit) * a.padded + (i - a.dim)] = value;
+  }
+  if (threadIdx.x < a.padded - a.dim) {
+    prepared[unit * a.padded + a.dim + threadIdx.x] = 0.f;
+    prepared[(a.qk_heads + unit) * a.padded + a.dim + threadIdx.x] = 0.f;
   }
   __syncthreads();
   if (warp == 0) {
@@ -637,6 +697,13 @@ __global__ void __launch_bounds__(256) delta_history_kernel(DeltaPrepareArgs a) 
   }
 }
 
+static int launch_delta_prepare(const DeltaPrepareArgs& a, int tokens, int sequences, cudaStream_t stream) {
+  int status = dllm_launch_pdl(delta_prepare_kernel, dim3(tokens, a.qk_heads + a.heads), dim3(128), 0, stream, a);
+  if (status != DLLM_OK || a.single || a.n_taps == 1) return status;
+  int channels = 2 * a.qk_heads * a.dim + a.heads * a.vdim;
+  return dllm_launch_pdl(delta_history_kernel, dim3(sequences, (channels + 255) / 256), dim3(256), 0, stream, a);
+}
+
 DLLM_EXPORT int dllm_delta_prepare(const float* proj, int stride, int b_off, int a_off, const float* taps, int n_taps,
                                    const float* a_log, const float* dt_bias, float* conv_state, const int* tok_seq,
                                    const int* cu_seqlens, const int* slots, int tokens, int sequences, int heads,
@@ -645,23 +712,40 @@ DLLM_EXPORT int dllm_delta_prepare(const float* proj, int stride, int b_off, int
   if (tokens <= 0) return DLLM_OK;
   if (n_taps < 1 || n_taps > DELTA_MAX_TAPS || !scan_sizes_ok(heads, qk_heads, dim, vdim, stride))
     return DLLM_UNSUPPORTED_SIZE;
-  size_t channels = 2 * (size_t)qk_heads * dim + (size_t)heads * vdim;
   if (qk_heads + heads >= 65536) return DLLM_UNSUPPORTED_SIZE;
   if (!proj || !taps || !a_log || !dt_bias || !tok_seq || !cu_seqlens || !slots || !prepared || !aux ||
       (n_taps > 1 && !conv_state))
     return DLLM_BAD_ARGUMENT;
   DeltaPrepareArgs a = {proj, stride, b_off, a_off, taps, n_taps, a_log, dt_bias, conv_state, tok_seq, cu_seqlens,
-                        slots, heads, qk_heads, dim, vdim, prepared, aux, single};
-  int status = dllm_launch_pdl(delta_prepare_kernel, dim3(tokens, qk_heads + heads), dim3(128), 0, stream, a);
-  if (status != DLLM_OK || single || n_taps == 1) return status;
-  int across = (int)((channels + 255) / 256);
-  return dllm_launch_pdl(delta_history_kernel, dim3(sequences, across), dim3(256), 0, stream, a);
+                        slots, heads, qk_heads, dim, vdim, prepared, aux, single, dim, nullptr, 0, nullptr};
+  return launch_delta_prepare(a, tokens, sequences, stream);
+}
+
+// The same for the delta rule by channels (see above): rates [tokens][rate_stride], dt_bias [heads x dim], decays
+// [tokens][heads x padded]; dim any size up to 256, padded = dim rounded up to a multiple of 4.
+DLLM_EXPORT int dllm_channel_delta_prepare(const float* proj, int stride, int b_off, const float* rates, int rate_stride,
+                                           const float* taps, int n_taps, const float* a_log, const float* dt_bias,
+                                           float* conv_state, const int* tok_seq, const int* cu_seqlens,
+                                           const int* slots, int tokens, int sequences, int heads, int qk_heads, int dim,
+                                           int padded, int vdim, float* prepared, float* decays, float* aux, int single,
+                                           cudaStream_t stream) {
+  if (tokens <= 0) return DLLM_OK;
+  if (n_taps < 1 || n_taps > DELTA_MAX_TAPS || dim <= 0 || padded < dim || padded - dim > 3 ||
+      !scan_sizes_ok(heads, qk_heads, padded, vdim, stride) || rate_stride < heads * dim || qk_heads + heads >= 65536)
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!proj || !rates || !taps || !a_log || !dt_bias || !tok_seq || !cu_seqlens || !slots || !prepared || !decays ||
+      !aux || (n_taps > 1 && !conv_state))
+    return DLLM_BAD_ARGUMENT;
+  DeltaPrepareArgs a = {proj, stride, b_off, 0, taps, n_taps, a_log, dt_bias, conv_state, tok_seq, cu_seqlens, slots,
+                        heads, qk_heads, dim, vdim, prepared, aux, single, padded, rates, rate_stride, decays};
+  return launch_delta_prepare(a, tokens, sequences, stream);
 }
 
 // ---- read-out: norm, weight and gate ----------------------------------------------------------------------------
 // x [tokens, width] float32 is normed in groups of `group` values (a head's vdim, or the whole width): divided by
 // sqrt(mean square + eps), times weight[i % group] if a weight is given, times gate(z) with z the token's gate
-// pre-activations (rows of `gate_stride` floats; gate 1: silu, 2: sigmoid), rounded once to the output type.
+// pre-activations (rows of `gate_stride` floats; gate 1: silu, 2: sigmoid), rounded once to the output type. Output rows
+// have `out_stride` values, up to 31 more than `width`, and zeros behind it (a product may want longer rows).
 template <typename T>
 __device__ __forceinline__ void gated_store(T* dst, const float* row, const float* weight, const float* z, int i,
                                             int group, float inv, int gate_kind) {
@@ -677,7 +761,7 @@ __global__ void __launch_bounds__(128) gated_norm_groups_kernel(T* __restrict__ 
                                                                 const float* __restrict__ weight,
                                                                 const float* __restrict__ gate, int gate_stride,
                                                                 int tokens, int width, int group, float eps,
-                                                                int gate_kind) {
+                                                                int gate_kind, int out_stride) {
   pdl_launch_dependents();
   pdl_wait();
   const int groups = width / group, lane = threadIdx.x & 31;
@@ -690,8 +774,9 @@ __global__ void __launch_bounds__(128) gated_norm_groups_kernel(T* __restrict__ 
   ss = warp_sum(ss);
   float inv = 1.0f / sqrtf(ss / (float)group + eps);
   for (int i = lane; i < group; i += 32)
-    gated_store<T>(out + (size_t)t * width, row, weight, gate + (size_t)t * gate_stride, g * group + i, group, inv,
+    gated_store<T>(out + (size_t)t * out_stride, row, weight, gate + (size_t)t * gate_stride, g * group + i, group, inv,
                    gate_kind);
+  if (g == groups - 1 && width + lane < out_stride) out[(size_t)t * out_stride + width + lane] = from_float<T>(0.f);
 }
 
 // one group over the whole row: a block per token
@@ -699,7 +784,7 @@ template <typename T>
 __global__ void __launch_bounds__(512) gated_norm_row_kernel(T* __restrict__ out, const float* __restrict__ x,
                                                              const float* __restrict__ weight,
                                                              const float* __restrict__ gate, int gate_stride,
-                                                             int width, float eps, int gate_kind) {
+                                                             int width, float eps, int gate_kind, int out_stride) {
   __shared__ float scratch[16];
   pdl_launch_dependents();
   pdl_wait();
@@ -714,33 +799,37 @@ __global__ void __launch_bounds__(512) gated_norm_row_kernel(T* __restrict__ out
   for (int w = 0; w < warps; ++w) total += scratch[w];
   float inv = 1.0f / sqrtf(total / (float)width + eps);
   for (int i = threadIdx.x; i < width; i += blockDim.x)
-    gated_store<T>(out + (size_t)t * width, row, weight, gate + (size_t)t * gate_stride, i, width, inv, gate_kind);
+    gated_store<T>(out + (size_t)t * out_stride, row, weight, gate + (size_t)t * gate_stride, i, width, inv, gate_kind);
+  if (width + threadIdx.x < out_stride) out[(size_t)t * out_stride + width + threadIdx.x] = from_float<T>(0.f);
 }
 
 template <typename T>
 static int launch_gated_norm(T* out, const float* x, const float* weight, const float* gate, int gate_stride,
-                             int tokens, int width, int group, float eps, int gate_kind, cudaStream_t stream) {
+                             int tokens, int width, int group, float eps, int gate_kind, int out_stride,
+                             cudaStream_t stream) {
   if (group == width) {
     int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
     return dllm_launch_pdl(gated_norm_row_kernel<T>, dim3(tokens), dim3(threads), 0, stream, out, x, weight, gate,
-                           gate_stride, width, eps, gate_kind);
+                           gate_stride, width, eps, gate_kind, out_stride);
   }
   long long units = (long long)tokens * (width / group);
   return dllm_launch_pdl(gated_norm_groups_kernel<T>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, stream, out, x,
-                         weight, gate, gate_stride, tokens, width, group, eps, gate_kind);
+                         weight, gate, gate_stride, tokens, width, group, eps, gate_kind, out_stride);
 }
 
 DLLM_EXPORT int dllm_gated_norm(void* out, const float* x, const float* weight, const float* gate, int gate_stride,
-                                int tokens, int width, int group, float eps, int gate_kind, int out_dtype,
-                                cudaStream_t stream) {
+                                int tokens, int width, int group, float eps, int gate_kind, int out_stride,
+                                int out_dtype, cudaStream_t stream) {
   if (tokens <= 0) return DLLM_OK;
   if (width <= 0 || group <= 0 || width % group || (gate_kind != 1 && gate_kind != 2)) return DLLM_UNSUPPORTED_SIZE;
+  if (out_stride < width || out_stride > width + 31) return DLLM_UNSUPPORTED_SIZE;
   if (!out || !x || !gate) return DLLM_BAD_ARGUMENT;
   if (out_dtype == DLLM_F32)
-    return launch_gated_norm((float*)out, x, weight, gate, gate_stride, tokens, width, group, eps, gate_kind, stream);
+    return launch_gated_norm((float*)out, x, weight, gate, gate_stride, tokens, width, group, eps, gate_kind, out_stride,
+                             stream);
   if (out_dtype == DLLM_BF16)
     return launch_gated_norm((__nv_bfloat16*)out, x, weight, gate, gate_stride, tokens, width, group, eps, gate_kind,
-                             stream);
+                             out_stride, stream);
   return DLLM_BAD_ARGUMENT;
 }
 

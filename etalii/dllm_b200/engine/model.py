@@ -7,6 +7,7 @@ from typing import Mapping
 import torch
 
 from ..cache.paged import PagedCache
+from ..parts.norm import taken_normed
 from ..parts.registry import build_part, part_factory
 from ..parts.spec import ModelSpec
 from .runtime import Runtime
@@ -55,7 +56,8 @@ class Model:
         if torch.device(rt.device).type == "cuda":  # what the parts say they call, compiled side by side
             from ..kernels.build import prebuild
 
-            names = {"elementwise", "gemm_simt" if rt.dtype == torch.float32 else "gemv"}
+            names = {name for block in self.blocks for name in getattr(block, "LIBRARIES", ())}
+            names |= {"elementwise", "gemm_simt" if rt.dtype == torch.float32 else "gemv"}
             for part in (*self._layer_parts(), *self.reentries):
                 if hasattr(part, "kernel_libraries"):
                     names |= set(part.kernel_libraries(rt))
@@ -92,6 +94,17 @@ class Model:
             return self.cache.kv_view(index) if need.kind == "kv" else self.cache.state(index)
 
         self._views = [view_of(entry.cache) for entry in self.order]
+
+        # a block whose last kernel can leave the stream already normed for its next reader is told that reader's norm
+        for entry, following in zip(self.order, (*self.order[1:], None)):
+            leads_to = getattr(self.blocks[entry.layer], "leads_to", None)
+            if leads_to is None:
+                continue
+            if following is None:
+                leads_to(self.final_norm, last=True)
+            else:  # (something that rewrites the stream before the next run reads it from memory)
+                leads_to(None if following.reentry is not None
+                         else getattr(self.blocks[following.layer], "mixer_norm", None))
 
         self._plan_prefetch()
         # the C++ host side of prefill-sized steps, for models made of the parts it restates (else None)
@@ -151,7 +164,10 @@ class Model:
 
         rt = self.rt
         ops.prefetch_hints = self._prefetch  # this model's hints (they live and die with the model)
-        x = self.embedding.forward(batch.tokens, batch.n_tokens, rt)
+        if getattr(self.embedding, "wants_positions", False):
+            x = self.embedding.forward(batch.tokens, batch.n_tokens, rt, positions=batch.tok_pos)
+        else:
+            x = self.embedding.forward(batch.tokens, batch.n_tokens, rt)
         if self.native_layers is not None and self.native_layers.takes(batch):
             self.native_layers.run(x, batch, rt)  # every layer's launches from one C++ call
         else:
@@ -167,7 +183,9 @@ class Model:
             return None
         if batch.is_decode and batch.n_want == batch.n_tokens and hasattr(self.final_norm, "lazy") \
                 and getattr(self.head, "accepts_pending_norm", False):
-            pending = self.final_norm.lazy(x, rt)  # every row is wanted, in order: no gather
+            pending = taken_normed(self.final_norm, x, rt)  # every row is wanted, in order: no gather
+            if pending is None:
+                pending = self.final_norm.lazy(x, rt)
             if greedy_out is not None and hasattr(self.head, "choose_greedy") and \
                     self.head.choose_greedy(pending, rt, greedy_out):
                 return None

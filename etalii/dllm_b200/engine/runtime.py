@@ -67,6 +67,8 @@ class Runtime:
         self.stream_rounded = None
         """(address, shape, launch count, copy): the residual stream's rounding to the activation type where the kernel
         that last wrote the stream left one; valid only while no other kernel has been launched since."""
+        self.stream_normed = None
+        """(norm, address, shape, launch count, rows): the stream as that norm makes it, on the same terms."""
         self._keep: list = []
 
     def to_device(self, tensor: torch.Tensor, dtype: torch.dtype | None = None) -> torch.Tensor:

@@ -45,6 +45,8 @@ SOURCES = {
     "sigmoid_attention_tiled": "sigmoid_attention_tiled.cu",
     "moe": "moe.cu",
     "moe_grouped": "moe_grouped.cu",
+    "sink_attention": "sink_attention.cu",
+    "stream_update": "stream_update.cu",
     "sampling": "sampling.cu",
     "step_launcher": "step_launcher.cu",
 }

@@ -30,6 +30,12 @@ _prototypes = {
     ("elementwise", "dllm_embed"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     ("elementwise", "dllm_embed_scaled"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p,
                                            c_void_p],
+    ("elementwise", "dllm_embed_sinusoid"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                             c_int, c_float, c_void_p, c_void_p],
+    ("elementwise", "dllm_softcap"): [c_void_p, c_longlong, c_float, c_void_p],
+    ("stream_update", "dllm_stream_update"): [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
+                                              c_longlong, c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int,
+                                              c_int, c_int, c_void_p],
     ("elementwise", "dllm_rmsnorm"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     ("elementwise", "dllm_layernorm"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     ("elementwise", "dllm_glu_clamped"): [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
@@ -52,6 +58,9 @@ _prototypes = {
                                                                   c_int, c_void_p, c_int, c_void_p],
     ("sigmoid_attention", "dllm_sigmoid_combine"): [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                                     c_void_p],
+    ("sink_attention", "dllm_sink_attention"): [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                                c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                                c_float, c_float, c_int, c_int, c_int, c_int, c_void_p],
     ("elementwise", "dllm_norm_sum_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
                                                 c_float, c_void_p],
     ("elementwise", "dllm_norm_add_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
@@ -126,8 +135,15 @@ _prototypes = {
     ("recurrent", "dllm_delta_prepare"): [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                           c_void_p, c_void_p, c_int, c_void_p],
+    ("recurrent", "dllm_channel_delta_scan"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                                               c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                               c_void_p, c_void_p],
+    ("recurrent", "dllm_channel_delta_prepare"): [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
+                                                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                                  c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                                  c_void_p],
     ("recurrent", "dllm_gated_norm"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                                       c_int, c_int, c_void_p],
+                                       c_int, c_int, c_int, c_void_p],
     ("elementwise", "dllm_rope_cache_write"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                                c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                                c_int, c_int, c_longlong, c_void_p],
@@ -268,6 +284,62 @@ def embed(out: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, status: 
     _check(_fn("elementwise", "dllm_embed_scaled")(out.data_ptr(), table.data_ptr(), tokens.data_ptr(), rows, hidden,
                                                    table.shape[0], _code(table.dtype), float(scale),
                                                    status.data_ptr(), _stream()), "embed")
+
+
+def embed_sinusoid(out: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, positions: torch.Tensor,
+                   frequencies: torch.Tensor, status: torch.Tensor | None = None, scale: float = 1.0) -> None:
+    """`embed` with a position vector added: out[r, 2i] += sin(p f_i), out[r, 2i + 1] += cos(p f_i), p = positions[r];
+    `frequencies` float32 [ceil(hidden / 2), 2]: f_i and what its rounding to float32 took off."""
+    _cuda(out, table, tokens, positions, frequencies)
+    if status is None:
+        status = _status_word()
+    assert out.dtype == torch.float32 and tokens.dtype == torch.int32 and positions.dtype == torch.int32
+    rows, hidden = out.shape
+    assert tokens.numel() >= rows and positions.numel() >= rows and table.shape[1] == hidden
+    assert frequencies.dtype == torch.float32 and tuple(frequencies.shape) == ((hidden + 1) // 2, 2)
+    _check(_fn("elementwise", "dllm_embed_sinusoid")(
+        out.data_ptr(), table.data_ptr(), tokens.data_ptr(), positions.data_ptr(), frequencies.data_ptr(), rows, hidden,
+        table.shape[0], _code(table.dtype), float(scale), status.data_ptr(), _stream()), "embed_sinusoid")
+
+
+def softcap_rows(x: torch.Tensor, cap: float) -> None:
+    """x <- cap * tanh(x / cap) in place, float32."""
+    _cuda(x)
+    assert x.dtype == torch.float32 and cap > 0
+    _check(_fn("elementwise", "dllm_softcap")(x.data_ptr(), x.numel(), float(cap), _stream()), "softcap")
+
+
+def stream_update(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
+                  first_result: torch.Tensor | None = None, results: torch.Tensor | None = None, index: int = 0,
+                  coefficients: torch.Tensor | None = None, first_from_stream: bool = False,
+                  next_weight: torch.Tensor | None = None, next_eps: float = 0.0,
+                  normed: torch.Tensor | None = None) -> None:
+    """Behind a sublayer whose output y is normed: v = x + y / rms(y) * weight. Without `coefficients` x <- v; with them
+    (float32 [index + 2]) x <- sum_(j <= index) coefficients[j] results[j] + coefficients[index + 1] v, and v is kept as
+    results[index + 1] where `results` [layers, rows, hidden] has that place. `first_result`: x as it was is kept there
+    (results[0], say; with `first_from_stream` the same launch's sum takes it from x). `normed`: the new x divided by
+    its root mean square (`next_eps`) times `next_weight`, in normed's type. All else float32."""
+    _cuda(x, y, weight, first_result, results, coefficients, next_weight, normed)
+    rows, hidden = y.shape
+    assert x.dtype == y.dtype == weight.dtype == torch.float32 and tuple(x.shape) == (rows, hidden)
+    assert weight.numel() == hidden and (next_weight is None) == (normed is None)
+    assert first_result is None or (first_result.dtype == torch.float32 and first_result.numel() == rows * hidden)
+    assert next_weight is None or (next_weight.dtype == torch.float32 and next_weight.numel() == hidden)
+    assert normed is None or tuple(normed.shape) == (rows, hidden)
+    kept = None
+    if coefficients is not None:
+        assert coefficients.dtype == torch.float32 and coefficients.numel() == index + 2
+        assert results.dtype == torch.float32 and tuple(results.shape[1:]) == (rows, hidden)
+        assert results.shape[0] > index and (not first_from_stream or index == 0)
+        if index + 1 < results.shape[0]:
+            kept = results.data_ptr() + 4 * (index + 1) * rows * hidden
+    ptr = lambda tensor: tensor.data_ptr() if tensor is not None else None  # noqa: E731
+    _check(_fn("stream_update", "dllm_stream_update")(
+        x.data_ptr(), y.data_ptr(), weight.data_ptr(), float(eps), ptr(first_result), kept, ptr(results), rows * hidden,
+        index + 1 if coefficients is not None else 0, ptr(coefficients), 1 if first_from_stream else 0,
+        ptr(next_weight), float(next_eps), ptr(normed), rows, hidden,
+        _code(normed.dtype) if normed is not None else 0, _stream()), "stream_update",
+        lambda: f"hidden={hidden} (a multiple of 4 up to 8192)")
 
 
 def copy_to_device(dst_ptr: int, src_ptr: int, nbytes: int) -> None:
@@ -448,6 +520,28 @@ def sigmoid_attention_tiled(out: torch.Tensor, q: torch.Tensor, cache, heads: in
         _check(_fn("sigmoid_attention", "dllm_sigmoid_combine")(
             part.data_ptr(), gate_ptr, gate_ld, out.data_ptr(), tokens, heads * vdim, splits, _code(out.dtype),
             _stream()), "sigmoid_combine")
+
+
+def sink_attention(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
+                   sinks: torch.Tensor | None, window: int, keep: int, batch, split: bool | None = None) -> None:
+    """Softmax attention of every token over its own sequence's cache: scores q . k * scale, then softcap * tanh(score /
+    softcap) if softcap > 0, of the keys j <= i with i - j < window (0: all) or j < keep; the denominator also holds
+    exp(sinks[h]) where `sinks` float32 [heads] is given. q [tokens, heads x dim] and out [tokens, heads x value_dim, or
+    longer rows: zeros behind] in the cache's type. The general kernel: float32 arithmetic, every size up to 256.
+    `split`: a block of sixteen warps per (token, head) instead of a warp (default: for steps of few tokens)."""
+    _cuda(out, q, sinks)
+    dim, vdim, tokens = cache.head_dim, cache.value_dim, batch.n_tokens
+    assert q.dtype == cache.dtype and out.dtype == cache.dtype and not cache.keys_only
+    assert q.shape[1] == heads * dim and out.shape[1] >= heads * vdim
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
+    if split is None:
+        split = tokens * heads <= 4 * _multiprocessors()
+    _check(_fn("sink_attention", "dllm_sink_attention")(
+        q.data_ptr(), out.data_ptr(), out.shape[1], cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
+        cache.page_size, heads, cache.kv_heads, dim, vdim, sinks.data_ptr() if sinks is not None else None,
+        batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.slots.data_ptr(), tokens, float(scale),
+        float(softcap or 0.0), int(window or 0), int(keep or 0), 1 if split else 0, _code(cache.dtype), _stream()),
+        "sink_attention", lambda: f"dim={dim}, value_dim={vdim} (at most 256)")
 
 
 def glu_clamped_fuses(rows: int, outputs: int, inner: int) -> bool:
@@ -1091,20 +1185,67 @@ def delta_scan(out: torch.Tensor, prepared: torch.Tensor, aux: torch.Tensor, hea
         lambda: f"dim={dim} (a multiple of 4, at most 256)")
 
 
+def channel_delta_prepare(prepared: torch.Tensor, decays: torch.Tensor, aux: torch.Tensor, rows: torch.Tensor,
+                          b_at: int, rates: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor,
+                          dt_bias: torch.Tensor, history: torch.Tensor | None, heads: int, qk_heads: int, dim: int,
+                          vdim: int, batch) -> None:
+    """`delta_prepare` for a decay per head and key channel: decays[t, h, i] = exp(-exp(a_log[h]) softplus(rates[t, h *
+    dim + i] + dt_bias[h * dim + i])), `rates` float32 rows of heads x dim values or more. A head's q, k (in `prepared` =
+    [q | k | v]) and decays take rows of dim rounded up to a multiple of 4; `aux`'s first `heads` columns stay unused."""
+    _cuda(prepared, decays, aux, rows, rates, taps, a_log, dt_bias, history)
+    channels, padded = 2 * qk_heads * dim + heads * vdim, -(-dim // 4) * 4
+    assert all(t.dtype == torch.float32 for t in (prepared, decays, aux, rows, rates, taps, a_log, dt_bias))
+    assert taps.shape[0] == channels and prepared.shape[1] == 2 * qk_heads * padded + heads * vdim
+    assert decays.shape[1] == heads * padded and aux.shape[1] == 2 * heads + qk_heads
+    assert a_log.numel() == heads and dt_bias.numel() == heads * dim and rates.shape[1] >= heads * dim
+    assert rows.shape[1] >= max(channels, b_at + heads) and min(rows.shape[0], rates.shape[0]) >= batch.n_tokens
+    width = taps.shape[1]
+    assert history is None or (history.dtype == torch.float32 and tuple(history.shape[1:]) == (width - 1, channels))
+    _check(_fn("recurrent", "dllm_channel_delta_prepare")(
+        rows.data_ptr(), rows.shape[1], int(b_at), rates.data_ptr(), rates.shape[1], taps.data_ptr(), width,
+        a_log.data_ptr(), dt_bias.data_ptr(), history.data_ptr() if history is not None else None,
+        batch.tok_seq.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_tokens, batch.n_seqs,
+        heads, qk_heads, dim, padded, vdim, prepared.data_ptr(), decays.data_ptr(), aux.data_ptr(),
+        1 if batch.is_decode else 0, _stream()), "channel_delta_prepare",
+        lambda: f"taps={width} (at most 16), dim={dim} (at most 256)")
+    if not batch.is_decode and width > 1:
+        global launches
+        launches += 1  # (the history's own small kernel)
+
+
+def channel_delta_scan(out: torch.Tensor, prepared: torch.Tensor, decays: torch.Tensor, aux: torch.Tensor, heads: int,
+                       qk_heads: int, padded: int, vdim: int, state: torch.Tensor, batch) -> None:
+    """Per sequence and head, over the step's tokens in order: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T;
+    out = S^T q, from and to `state` [slots, heads, vdim, padded]: what `channel_delta_prepare` wrote, a head's q, k and
+    decays in rows of `padded` values."""
+    _cuda(out, prepared, decays, aux, state)
+    assert all(t.dtype == torch.float32 for t in (out, prepared, decays, aux, state))
+    assert tuple(state.shape[1:]) == (heads, vdim, padded) and out.shape[1] == heads * vdim
+    assert prepared.shape[1] == 2 * qk_heads * padded + heads * vdim and decays.shape[1] == heads * padded
+    _check(_fn("recurrent", "dllm_channel_delta_scan")(
+        prepared.data_ptr(), _columns(prepared, qk_heads * padded), _columns(prepared, 2 * qk_heads * padded),
+        prepared.shape[1], decays.data_ptr(), decays.shape[1], heads, qk_heads, padded, vdim, aux.data_ptr(),
+        aux.shape[1], state.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_seqs,
+        int(batch.max_new), out.data_ptr(), _stream()), "channel_delta_scan",
+        lambda: f"rows of {padded} values (a multiple of 4, at most 256)")
+
+
 GATE_SILU, GATE_SIGMOID = 1, 2
 
 
 def gated_norm(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor | None, rows: torch.Tensor, gate_at: int,
                group: int, eps: float, gate: int) -> None:
     """out = x / rms(x over groups of `group` values) * weight[i % group] * gate(z), z the token's gate values at
-    column offset gate_at of `rows` [tokens, n] float32; gate GATE_SILU or GATE_SIGMOID. x float32 [tokens, width]."""
+    column offset gate_at of `rows` [tokens, n] float32; gate GATE_SILU or GATE_SIGMOID. x float32 [tokens, width]; out may
+    have up to 31 columns more, which get zeros."""
     _cuda(out, x, weight, rows)
-    tokens, width = out.shape
-    assert x.dtype == torch.float32 and rows.dtype == torch.float32 and x.shape[1] == width
+    tokens, width = x.shape
+    assert x.dtype == torch.float32 and rows.dtype == torch.float32 and out.shape[0] == tokens
     assert weight is None or (weight.dtype == torch.float32 and weight.numel() == group)
     _check(_fn("recurrent", "dllm_gated_norm")(
         out.data_ptr(), x.data_ptr(), weight.data_ptr() if weight is not None else None, _columns(rows, gate_at),
-        rows.shape[1], tokens, width, int(group), float(eps), int(gate), _code(out.dtype), _stream()), "gated_norm")
+        rows.shape[1], tokens, width, int(group), float(eps), int(gate), out.shape[1], _code(out.dtype), _stream()),
+        "gated_norm")
 
 
 prefetch_hints: dict[int, torch.Tensor] = {}

@@ -6,14 +6,17 @@ in `forward(x, batch, cache, rt, write_cache)` on the float32 residual stream x.
 "output_norm": x += norm(mixer(x)); x += norm(feed_forward(x)): the sublayers read the stream itself and the norm sits
 on what they return.
 "filtered_pre_norm": x += mixer(filter(norm(x))); x += feed_forward(norm(x)); x += token_input(x): a filter over time
-sits between the first norm and the mixer; the feed-forward and the token input are optional."""
+sits between the first norm and the mixer; the feed-forward and the token input are optional.
+"sandwich_norm": x += norm(mixer(norm(x))); x += norm(feed_forward(norm(x))), the feed-forward optional; optionally the
+stream then becomes a weighted sum of all layers' results so far."""
 from __future__ import annotations
 
 import torch
 
 from ..kernels import ops
-from .norm import StreamOperand
+from .norm import RMSNorm, StreamOperand, leave_normed, taken_normed
 from .registry import register_part
+from .spec import ParamSpec
 
 
 def normed(norm, consumer, x, rt):
@@ -161,6 +164,105 @@ class FilteredPreNormBlock:
             self.token_input.forward(x, batch, rt)
 
 
+class DepthAverage:
+    """What leaves layer `index` of `layers`: the sum over j = 0 .. index + 1 of weight[j] X_j, with X_0 the embedding's
+    output and X_(i + 1) the result of layer i before this sum. The X_j of a step live in a work buffer [layers, tokens,
+    hidden] float32 (the last layer's result is read by nobody)."""
+
+    def __init__(self, index: int, layers: int) -> None:
+        self.index, self.layers = int(index), int(layers)
+        self.weight = None
+
+    @staticmethod
+    def parameters(index, layers) -> dict[str, ParamSpec]:
+        return {"weight": ParamSpec((int(index) + 2,), "last_one")}
+
+    def bind(self, tensors, rt) -> None:
+        self.weight = rt.to_device(tensors["weight"], torch.float32)
+
+    def results(self, x: torch.Tensor, rt) -> torch.Tensor:
+        return rt.ws.buffer("layer_results", (self.layers, *x.shape), torch.float32)
+
+
+class SandwichNormBlock:
+    """x += mixer_output_norm(mixer(mixer_norm(x))); then, where the layer has one, x += feed_forward_output_norm(
+    feed_forward(feed_forward_norm(x))); then, with a `depth_average`, the stream becomes the weighted sum of all layers'
+    results so far. (A multiplier of the sublayers is the output norms' `factor`.) Each sublayer writes its float32
+    output to a work buffer and ONE kernel does everything from there to the next product's operand: the output's norm,
+    the residual sum, the sum over the layers, and the norm in front of whoever reads the stream next (the model tells a
+    block whose norm that is: `leads_to`)."""
+
+    PARTS = {"mixer": "mixer", "mixer_norm": "norm", "mixer_output_norm": "norm"}
+    OPTIONAL_PARTS = {"feed_forward": "feed_forward", "feed_forward_norm": "norm", "feed_forward_output_norm": "norm",
+                      "depth_average": "stream_mix"}
+    LIBRARIES = ("stream_update",)
+
+    def __init__(self, mixer, mixer_norm, mixer_output_norm, feed_forward=None, feed_forward_norm=None,
+                 feed_forward_output_norm=None, depth_average=None) -> None:
+        together = (feed_forward, feed_forward_norm, feed_forward_output_norm)
+        if any(part is None for part in together) != all(part is None for part in together):
+            raise ValueError("a feed-forward and its two norms come together")
+        self.mixer, self.mixer_norm, self.mixer_output_norm = mixer, mixer_norm, mixer_output_norm
+        self.feed_forward, self.feed_forward_norm = feed_forward, feed_forward_norm
+        self.feed_forward_output_norm, self.depth_average = feed_forward_output_norm, depth_average
+        self.parts = {name: part for name, part in (
+            ("mixer", mixer), ("mixer_norm", mixer_norm), ("mixer_output_norm", mixer_output_norm),
+            ("feed_forward", feed_forward), ("feed_forward_norm", feed_forward_norm),
+            ("feed_forward_output_norm", feed_forward_output_norm), ("depth_average", depth_average))
+            if part is not None}
+        self._next = None  # (norm, last): the norm of whoever reads the stream behind this block
+        self._told = False
+
+    def leads_to(self, norm, last: bool = False) -> None:
+        """`norm`: what the next reader of the stream norms it by (None: not known); `last`: that reader wants single
+        rows of a prompt, so the whole stream is normed for it in steps of single tokens only. A block that runs
+        several times with different readers behind it norms for none."""
+        if self._told and (self._next is None or self._next[0] is not norm):
+            self._next = None
+        else:
+            self._next = (norm, bool(last)) if getattr(norm, "weight", None) is not None and \
+                isinstance(norm, RMSNorm) else None
+        self._told = True
+
+    def _update(self, x, out, output_norm, following, rt, average=None, keep_first=None, mix_first: bool = False) -> None:
+        """The kernel behind a sublayer: see `ops.stream_update`."""
+        normed_out = None
+        if following is not None:
+            normed_out = rt.ws.buffer("stream_normed", tuple(x.shape), rt.dtype)
+        results = average.results(x, rt) if average is not None else None
+        ops.stream_update(x, out, output_norm.weight, output_norm.eps,
+                          first_result=keep_first, results=results,
+                          index=average.index if average is not None else 0,
+                          coefficients=average.weight if average is not None else None,
+                          first_from_stream=mix_first,
+                          next_weight=following.weight if following is not None else None,
+                          next_eps=following.eps if following is not None else 0.0, normed=normed_out)
+        if following is not None:
+            leave_normed(following, x, rt, normed_out)
+
+    def forward(self, x, batch, cache, rt, write_cache: bool = True) -> None:
+        out = rt.ws.buffer("sublayer_out", tuple(x.shape), torch.float32)
+        following = None
+        if self._next is not None and (batch.is_decode or not self._next[1]):
+            following = self._next[0]
+        average = self.depth_average
+        # the first layer's input is the embedding's output: its first kernel keeps it for the sums over the layers
+        keep = average.results(x, rt)[0] if average is not None and average.index == 0 else None
+        h = taken_normed(self.mixer_norm, x, rt)
+        if h is None:
+            h = self.mixer_norm.forward(x, rt)
+        self.mixer.forward(h, out, batch, cache, rt, write_cache, epilogue=ops.EPI_STORE_F32)
+        if self.feed_forward is None:
+            self._update(x, out, self.mixer_output_norm, following, rt, average, keep, keep is not None)
+            return
+        self._update(x, out, self.mixer_output_norm, self.feed_forward_norm, rt, None, keep)
+        h = taken_normed(self.feed_forward_norm, x, rt)
+        self.feed_forward.forward(h, out, batch, rt, epilogue=ops.EPI_STORE_F32)
+        self._update(x, out, self.feed_forward_output_norm, following, rt, average)
+
+
+register_part("stream_mix", "depth_average", DepthAverage)
+register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "filtered_pre_norm", FilteredPreNormBlock)
 register_part("block", "output_norm", OutputNormBlock)

@@ -7,14 +7,18 @@ import torch
 
 from ..kernels import ops
 from .norm import project, row_rule
-from .registry import register_part
+from .registry import build_part, register_part
 from .spec import ParamSpec
 
 
 class TokenEmbedding:
-    def __init__(self, vocab_size: int, hidden_size: int, scale: float = 1.0) -> None:
-        """`scale`: every embedding row is multiplied by it on the way into the stream (in float32)."""
+    wants_positions = True
+
+    def __init__(self, vocab_size: int, hidden_size: int, scale: float = 1.0, position=None) -> None:
+        """`scale`: every embedding row is multiplied by it on the way into the stream (in float32). `position`: a
+        position part whose vector is then added (sinusoidal)."""
         self.vocab_size, self.hidden_size, self.scale = int(vocab_size), int(hidden_size), float(scale)
+        self.position = build_part("position", position) if position is not None else None
         self.weight = None
 
     @staticmethod
@@ -23,24 +27,31 @@ class TokenEmbedding:
 
     def bind(self, tensors, rt) -> None:
         self.weight = rt.to_device(tensors["weight"], rt.dtype)
+        if self.position is not None:
+            self.position.bind({}, rt)
 
-    def forward(self, tokens: torch.Tensor, n_tokens: int, rt) -> torch.Tensor:
+    def forward(self, tokens: torch.Tensor, n_tokens: int, rt, positions: torch.Tensor | None = None) -> torch.Tensor:
         # a token outside the table sets the kernels' shared status word, which the engine looks at after each
         # step it waits for (kernels/ops.py::raise_if_failed)
         x = rt.ws.buffer("residual", (n_tokens, self.hidden_size), torch.float32)
-        ops.embed(x, self.weight, tokens, scale=self.scale)
+        if self.position is not None:
+            ops.embed_sinusoid(x, self.weight, tokens, positions, self.position.frequencies(), scale=self.scale)
+        else:
+            ops.embed(x, self.weight, tokens, scale=self.scale)
         return x
 
 
 class LinearHead:
     accepts_pending_norm = True
 
-    def __init__(self, vocab_size: int, hidden_size: int) -> None:
-        self.vocab_size, self.hidden_size = int(vocab_size), int(hidden_size)
+    def __init__(self, vocab_size: int, hidden_size: int, softcap: float = 0.0) -> None:
+        """`softcap`: the logits become softcap * tanh(logits / softcap) (0: as they are). The cap keeps their order,
+        so the greedy choice inside the product is made before it."""
+        self.vocab_size, self.hidden_size, self.softcap = int(vocab_size), int(hidden_size), float(softcap or 0.0)
         self.weight = None
 
     @staticmethod
-    def parameters(vocab_size, hidden_size) -> dict[str, ParamSpec]:
+    def parameters(vocab_size, hidden_size, **_) -> dict[str, ParamSpec]:
         return {"weight": ParamSpec((vocab_size, hidden_size))}
 
     def bind(self, tensors, rt) -> None:
@@ -70,6 +81,8 @@ class LinearHead:
         """hidden: final-normed rows, or the norm still pending (`NormedInput`)."""
         logits = rt.ws.buffer("logits", (hidden.shape[0], self.vocab_size), torch.float32)
         project(logits, hidden, self.weight, ops.EPI_STORE_F32)
+        if self.softcap > 0.0:
+            ops.softcap_rows(logits, self.softcap)
         return logits
 
 

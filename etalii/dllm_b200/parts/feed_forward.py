@@ -15,12 +15,17 @@ from .spec import ParamSpec
 class SwiGLU:
     accepts_pending_norm = True
 
-    def __init__(self, hidden_size: int, intermediate_size: int) -> None:
+    def __init__(self, hidden_size: int, intermediate_size: int, pad: bool = False) -> None:
+        """`pad`: an intermediate size that the products' 16-byte rows do not take is filled up with rows and columns of
+        zeros (silu(0) * 0 = 0 adds nothing); without it such a size is refused."""
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.given_size = self.intermediate_size
+        if pad:
+            self.intermediate_size = -(-self.intermediate_size // 8) * 8
         self.w_gate_up = self.w_down = None
 
     @staticmethod
-    def parameters(hidden_size, intermediate_size) -> dict[str, ParamSpec]:
+    def parameters(hidden_size, intermediate_size, **_) -> dict[str, ParamSpec]:
         return {"gate": ParamSpec((intermediate_size, hidden_size)), "up": ParamSpec((intermediate_size, hidden_size)),
                 "down": ParamSpec((hidden_size, intermediate_size))}
 
@@ -29,9 +34,14 @@ class SwiGLU:
 
     def bind(self, tensors, rt) -> None:
         gate, up = tensors["gate"].to(rt.dtype), tensors["up"].to(rt.dtype)
+        down = tensors["down"]
+        if self.intermediate_size != self.given_size:
+            more = self.intermediate_size - self.given_size
+            gate, up = (torch.nn.functional.pad(w, (0, 0, 0, more)) for w in (gate, up))
+            down = torch.nn.functional.pad(down, (0, more))
         fused = torch.stack([gate, up], dim=1).reshape(2 * self.intermediate_size, self.hidden_size)
         self.w_gate_up = fused.contiguous().to(rt.device)
-        self.w_down = rt.to_device(tensors["down"], rt.dtype)
+        self.w_down = rt.to_device(down, rt.dtype)
 
     def absorb_input_scale(self, scale: torch.Tensor) -> bool:
         """Takes a per-input-feature scale (the weight of the norm in front) into the columns of the gate/up
@@ -42,9 +52,10 @@ class SwiGLU:
             .to(torch.bfloat16).contiguous()
         return True
 
-    def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, rt) -> None:
+    def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, rt, epilogue: int = ops.EPI_RESIDUAL) -> None:
+        """Adds into `residual` (float32), or with `epilogue=ops.EPI_STORE_F32` writes it."""
         rows = h.shape[0]
-        if ops.FUSED_FEED_FORWARD and isinstance(h, NormedInput) and h.x is residual and \
+        if ops.FUSED_FEED_FORWARD and epilogue == ops.EPI_RESIDUAL and isinstance(h, NormedInput) and h.x is residual and \
                 rt.dtype == torch.bfloat16 and ops.mlp_decode_supported(rows, self.hidden_size, self.intermediate_size):
             # (an option, off by default: norm, gate/up, SwiGLU, down and the residual sum in one kernel)
             scratch = rt.ws.buffer("mlp_partial", (ops.mlp_decode_scratch(rows, self.hidden_size,
@@ -54,7 +65,7 @@ class SwiGLU:
             return
         act = rt.ws.buffer("ffn_act", (h.shape[0], self.intermediate_size), rt.dtype)
         project(act, h, self.w_gate_up, ops.EPI_SWIGLU)
-        ops.gemm(residual, act, self.w_down, ops.EPI_RESIDUAL)
+        ops.gemm(residual, act, self.w_down, epilogue)
 
 
     def kernel_libraries(self, rt) -> set[str]:

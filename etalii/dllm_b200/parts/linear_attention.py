@@ -5,6 +5,7 @@ and what the write is:
   "decay_linear_attention": S <- decay_h S + k v^T with a fixed decay per head (retention, lightning attention);
   "gated_delta_rule":       S <- g S; S <- S + k (beta (v - S^T k))^T with a decay g and a step size beta per token
                             and head, q and k unit vectors after a short causal convolution over time;
+  "channel_delta_rule":     the same with a decay per key channel, S <- diag(g) S;
   "gated_matrix_memory":    S <- a_t S + b_t k v^T with exponential input gates held in range by a running maximum of the
                             log gates, a normaliser n carried beside S, the read-out divided by max(|n . q|, e^-m).
 
@@ -20,7 +21,7 @@ from ..cache.paged import CacheNeed
 from ..kernels import ops
 from .norm import row_rule
 from .registry import register_part
-from .spec import ParamSpec
+from .spec import FreeSize, ParamSpec
 
 _GATES = {"silu": ops.GATE_SILU, "sigmoid": ops.GATE_SIGMOID}
 
@@ -169,6 +170,105 @@ class GatedDeltaRule:
         return _libraries(rt)
 
 
+def _in_pieces(n: int) -> int:
+    """`n` rounded up to what a product reads in 16-byte pieces, whichever its type."""
+    return -(-int(n) // 8) * 8
+
+
+class ChannelDeltaRule:
+    """The gated delta rule with one decay per head and key channel: q, k, v, beta and the convolution as in
+    `GatedDeltaRule`; g = exp(-exp(A_log_h) softplus(W_a2 W_a1 h + dt_bias)) [heads x dim] acts on the rows of S; the
+    read-out is divided by its root mean square per head, times a weight [vdim] shared by the heads, times
+    sigmoid(W_g2 W_g1 h), and projected by W_o. The inner sizes of the two low-rank projections are the checkpoint's.
+
+    Three products make a token's inputs: [q | k | v | b]; the two inner projections together, rounded to the activation
+    type; and both outer ones together as one block-diagonal matrix. Sizes that a product or the scan does not read in
+    16-byte pieces are filled up with zeros."""
+
+    def __init__(self, hidden_size: int, heads: int, qk_heads: int, dim: int, vdim: int, conv: int,
+                 eps: float) -> None:
+        self.hidden_size, self.heads, self.qk_heads = int(hidden_size), int(heads), int(qk_heads)
+        self.dim, self.vdim, self.conv, self.eps = int(dim), int(vdim), int(conv), float(eps)
+        if self.heads % self.qk_heads:
+            raise ValueError(f"{self.heads} heads are not a multiple of {self.qk_heads} q/k heads")
+        self.channels = 2 * self.qk_heads * self.dim + self.heads * self.vdim
+        self.padded = -(-self.dim // 4) * 4
+        """A head's q, k and decays as the scan sees them, rows of a multiple of 4 values."""
+        self.w_in = self.w_low = self.w_wide = self.w_o = self.taps = self.a_log = self.dt_bias = self.weight = None
+
+    @staticmethod
+    def parameters(hidden_size, heads, qk_heads, dim, vdim, conv, **_) -> dict[str, ParamSpec]:
+        heads, dim, vdim = int(heads), int(dim), int(vdim)
+        qk, values = int(qk_heads) * dim, heads * vdim
+        a_rank, g_rank = FreeSize("decay rank", dim), FreeSize("gate rank", vdim)
+        return {"q": ParamSpec((qk, hidden_size)), "k": ParamSpec((qk, hidden_size)),
+                "v": ParamSpec((values, hidden_size)), "b": ParamSpec((heads, hidden_size)),
+                "a1": ParamSpec((a_rank, hidden_size)), "a2": ParamSpec((heads * dim, a_rank)),
+                "g1": ParamSpec((g_rank, hidden_size)), "g2": ParamSpec((values, g_rank)),
+                "q_conv": ParamSpec((qk, int(conv))), "k_conv": ParamSpec((qk, int(conv))),
+                "v_conv": ParamSpec((values, int(conv))), "A_log": ParamSpec((heads,)),
+                "dt_bias": ParamSpec((heads * dim,)), "norm": ParamSpec((vdim,), "ones"),
+                "o": ParamSpec((hidden_size, values))}
+
+    def supports(self, rt) -> str | None:
+        if self.dim > 256:
+            return f"dim {self.dim}: the scan keeps a head's rows in registers, at most 256"
+        if not 1 <= self.conv <= 16:
+            return f"a convolution of {self.conv} taps: the kernel takes 1 to 16"
+        return row_rule(rt, hidden_size=self.hidden_size)
+
+    def cache_need(self) -> CacheNeed:
+        matrix = CacheNeed("state", state_shape=(self.heads, self.vdim, self.padded))
+        if self.conv == 1:
+            return matrix
+        return CacheNeed("several", parts=(matrix, CacheNeed("state", state_shape=(self.conv - 1, self.channels))))
+
+    def bind(self, tensors, rt) -> None:
+        fused = torch.cat([tensors[name].to(rt.dtype) for name in ("q", "k", "v", "b")], dim=0)
+        self.w_in = fused.contiguous().to(rt.device)
+        values, decays = self.heads * self.vdim, self.heads * self.dim
+        a_rank, g_rank = tensors["a1"].shape[0], tensors["g1"].shape[0]
+        a_room, g_room = _in_pieces(a_rank), _in_pieces(g_rank)
+        low = torch.zeros(a_room + g_room, self.hidden_size, dtype=rt.dtype)
+        low[:a_rank], low[a_room:a_room + g_rank] = tensors["a1"].to(rt.dtype), tensors["g1"].to(rt.dtype)
+        wide = torch.zeros(decays + values, a_room + g_room, dtype=rt.dtype)
+        wide[:decays, :a_rank] = tensors["a2"].to(rt.dtype)
+        wide[decays:, a_room:a_room + g_rank] = tensors["g2"].to(rt.dtype)
+        self.w_low, self.w_wide = low.to(rt.device), wide.to(rt.device)
+        o = torch.zeros(self.hidden_size, _in_pieces(values), dtype=rt.dtype)
+        o[:, :values] = tensors["o"].to(rt.dtype)
+        self.w_o = o.to(rt.device)
+        taps = torch.cat([tensors[name].float() for name in ("q_conv", "k_conv", "v_conv")], dim=0)
+        self.taps = taps.contiguous().to(rt.device)
+        self.a_log = rt.to_device(tensors["A_log"], torch.float32)
+        self.dt_bias = rt.to_device(tensors["dt_bias"], torch.float32)
+        self.weight = rt.to_device(tensors["norm"], torch.float32)
+
+    def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, state, rt, write_cache: bool = True,
+                epilogue: int = ops.EPI_RESIDUAL) -> None:
+        n, heads, values = batch.n_tokens, self.heads, self.heads * self.vdim
+        matrix, history = (state, None) if self.conv == 1 else state
+        low = rt.ws.buffer("mixer_low", (n, self.w_low.shape[0]), rt.dtype)
+        ops.gemm(low, h, self.w_low, ops.EPI_STORE_T)
+        wide = rt.ws.buffer("mixer_wide", (n, self.w_wide.shape[0]), torch.float32)
+        ops.gemm(wide, low, self.w_wide, ops.EPI_STORE_F32)
+        rows = rt.ws.buffer("mixer_rows", (n, self.channels + heads), torch.float32)
+        ops.gemm(rows, h, self.w_in, ops.EPI_STORE_F32)
+        prepared = rt.ws.buffer("mixer_prepared", (n, 2 * self.qk_heads * self.padded + values), torch.float32)
+        decays = rt.ws.buffer("mixer_decays", (n, heads * self.padded), torch.float32)
+        aux = rt.ws.buffer("mixer_aux", (n, 2 * heads + self.qk_heads), torch.float32)
+        ops.channel_delta_prepare(prepared, decays, aux, rows, self.channels, wide, self.taps, self.a_log, self.dt_bias,
+                                  history, heads, self.qk_heads, self.dim, self.vdim, batch)
+        read = rt.ws.buffer("mixer_read", (n, values), torch.float32)
+        ops.channel_delta_scan(read, prepared, decays, aux, heads, self.qk_heads, self.padded, self.vdim, matrix, batch)
+        gated = rt.ws.buffer("mixer_gated", (n, self.w_o.shape[1]), rt.dtype)
+        ops.gated_norm(gated, read, self.weight, wide, heads * self.dim, self.vdim, self.eps, ops.GATE_SIGMOID)
+        ops.gemm(residual, gated, self.w_o, epilogue)
+
+    def kernel_libraries(self, rt) -> set[str]:
+        return _libraries(rt)
+
+
 class GatedMatrixMemory:
     """q = W_q h * dim^-1/2, k = W_k h [heads x dim], v = W_v h [heads x vdim]. Per head a log input gate
     i = cap tanh((W_i h + b_i) / cap) and a log forget gate f = logsigmoid(cap tanh((W_f h + b_f) / cap)); with a running
@@ -251,3 +351,4 @@ class GatedMatrixMemory:
 register_part("mixer", "decay_linear_attention", DecayLinearAttention)
 register_part("mixer", "gated_matrix_memory", GatedMatrixMemory)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
+register_part("mixer", "channel_delta_rule", ChannelDeltaRule)

@@ -46,18 +46,27 @@ class StreamOperand:
 
 
 class RMSNorm:
-    def __init__(self, hidden_size: int, eps: float, scalar: bool = False) -> None:
+    def __init__(self, hidden_size: int, eps: float, scalar: bool = False, zero_centred: bool = False,
+                 factor: float = 1.0) -> None:
         """`scalar`: the weight is ONE number for all coordinates (a tensor without dimensions in the checkpoint); on
-        the device it is spread over the row, so every kernel that applies a norm weight takes it."""
+        the device it is spread over the row, so every kernel that applies a norm weight takes it. `zero_centred`: the
+        checkpoint stores the weight minus one. `factor`: what the normed rows count for where they are added to the
+        stream. Both go into the device's weight once, in float32."""
         self.hidden_size, self.eps, self.scalar = int(hidden_size), float(eps), bool(scalar)
+        self.zero_centred, self.factor = bool(zero_centred), float(factor)
         self.weight = None
 
     @staticmethod
-    def parameters(hidden_size: int, eps: float, scalar: bool = False) -> dict[str, ParamSpec]:
-        return {"weight": ParamSpec(() if scalar else (int(hidden_size),), "ones")}
+    def parameters(hidden_size: int, eps: float, scalar: bool = False, zero_centred: bool = False,
+                   factor: float = 1.0) -> dict[str, ParamSpec]:
+        return {"weight": ParamSpec(() if scalar else (int(hidden_size),), "normal" if zero_centred else "ones")}
 
     def bind(self, tensors, rt) -> None:
-        if self.scalar:
+        if self.zero_centred or self.factor != 1.0:
+            weight = tensors["weight"].to(torch.float32) + (1.0 if self.zero_centred else 0.0)
+            weight = (weight * self.factor).reshape(-1)
+            self.weight = weight.expand(self.hidden_size).contiguous().to(rt.device)
+        elif self.scalar:
             self.weight = tensors["weight"].to(torch.float32).reshape(1).expand(self.hidden_size).contiguous() \
                 .to(rt.device)
         else:
@@ -145,6 +154,20 @@ class DynamicTanh:
         out = rt.ws.buffer(name, (n, self.hidden_size), rt.dtype)
         ops.dynamic_tanh(out, x, self.alpha, self.weight, self.bias, rows)
         return out
+
+
+def leave_normed(norm, x: torch.Tensor, rt, out: torch.Tensor) -> None:
+    """Notes that the kernel just launched, which wrote the stream `x`, left it normed by `norm` in `out`."""
+    rt.stream_normed = (norm, x.data_ptr(), tuple(x.shape), ops.launches, out)
+
+
+def taken_normed(norm, x: torch.Tensor, rt) -> torch.Tensor | None:
+    """The stream normed by `norm`, where the kernel that last wrote the stream left it and no other kernel has been
+    launched since; else None."""
+    kept = getattr(rt, "stream_normed", None)
+    if kept is not None and kept[0] is norm and kept[1:4] == (x.data_ptr(), tuple(x.shape), ops.launches):
+        return kept[4]
+    return None
 
 
 FUSE_NORM_LIMIT = 16 << 20

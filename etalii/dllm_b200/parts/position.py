@@ -127,4 +127,36 @@ class RotaryEmbedding:
             [2 * i + 1 for i in range(half)] + rest[len(rest) // 2:]
 
 
+class SinusoidalPosition:
+    """A position vector that is added to the embedding's rows: entry 2i of position p is sin(p f_i), entry 2i + 1
+    cos(p f_i), f_i = base^(-2i / hidden_size). The kernel that gathers the rows computes it: each frequency is kept as
+    a float32 and what rounding took off it, so that an angle is right to float32's precision of the angle itself
+    whatever the position, and there is no table over the positions."""
+
+    def __init__(self, hidden_size: int, base: float = 10000.0) -> None:
+        self.hidden_size, self.base = int(hidden_size), float(base)
+        if self.base <= 1:
+            raise ValueError(f"base {self.base} must be above 1")
+        self._frequencies = None
+
+    @staticmethod
+    def parameters(**_) -> dict:
+        return {}
+
+    def bind(self, tensors, rt) -> None:
+        def make() -> torch.Tensor:
+            i = torch.arange((self.hidden_size + 1) // 2, dtype=torch.float64)
+            exact = torch.exp(-2.0 * i / self.hidden_size * math.log(self.base))
+            high = exact.to(torch.float32)
+            return torch.stack([high, (exact - high.to(torch.float64)).to(torch.float32)], dim=-1).contiguous() \
+                .to(rt.device)
+
+        self._frequencies = rt.shared(("sinusoidal", self.hidden_size, self.base), make)
+
+    def frequencies(self) -> torch.Tensor:
+        """[ceil(hidden_size / 2), (float32, the rest)]."""
+        return self._frequencies
+
+
 register_part("position", "rotary", RotaryEmbedding)
+register_part("position", "sinusoidal", SinusoidalPosition)

@@ -1,12 +1,14 @@
 """Registries of part kinds. A part class is registered under a role ("norm", "position", "mixer", "feed_forward",
-"block", "embedding", "head", "reentry", "filter", "token_input") and a kind name; `build_part` makes an instance from a `PartSpec`."""
+"block", "embedding", "head", "reentry", "filter", "token_input", "stream_mix") and a kind name; `build_part` makes an instance from a `PartSpec`."""
 from __future__ import annotations
 
 from typing import Any, Callable
 
-ROLES = ("norm", "position", "mixer", "feed_forward", "block", "embedding", "head", "reentry", "filter", "token_input")
+ROLES = ("norm", "position", "mixer", "feed_forward", "block", "embedding", "head", "reentry", "filter", "token_input",
+         "stream_mix")
 """filter: something between a norm and the part that reads it, over time inside a sequence (a short causal
-convolution); token_input: something a layer adds to the stream from the step's token ids themselves."""
+convolution); token_input: something a layer adds to the stream from the step's token ids themselves;
+stream_mix: what a layer makes of the stream from its own result and earlier layers' results."""
 _PARTS: dict[str, dict[str, Callable[..., Any]]] = {role: {} for role in ROLES}
 
 

@@ -12,10 +12,24 @@ from dataclasses import dataclass, field
 from typing import Any, Mapping
 
 
+class FreeSize(int):
+    """A size that the configuration does not give and the checkpoint's tensors decide (the inner size of a low-rank
+    projection): a tensor may have any size there, the same wherever one part uses the same `name`. Its value as an
+    integer is what the random-weights mode takes."""
+
+    name: str
+
+    def __new__(cls, name: str, default: int) -> "FreeSize":
+        size = super().__new__(cls, default)
+        size.name = name
+        return size
+
+
 @dataclass(frozen=True)
 class ParamSpec:
-    """One tensor a part owns. `init` tells the random-weights mode how to fill it: "normal" ~ N(0, std),
-    "ones" ~ 1 + N(0, std / 2) (norm weights), "int" for integer tables (kept as int32)."""
+    """One tensor a part owns (its shape may hold `FreeSize`s). `init` tells the random-weights mode how to fill it: "normal" ~ N(0, std),
+    "ones" ~ 1 + N(0, std / 2) (norm weights), "last_one" ~ N(0, std) with 1 added to the last value (a sum of many of which
+    the last leads), "int" for integer tables (kept as int32)."""
 
     shape: tuple[int, ...]
     init: str = "normal"

@@ -13,7 +13,7 @@ from typing import Mapping
 import torch
 
 from ..parts.registry import part_factory
-from ..parts.spec import ModelSpec, ParamSpec
+from ..parts.spec import FreeSize, ModelSpec, ParamSpec
 from .safetensors_io import SafetensorsError, SafetensorsFile, checkpoint_files
 
 
@@ -45,10 +45,25 @@ def expected_tensors(spec: ModelSpec) -> dict[str, ParamSpec]:
             name = part_spec.names.get(local)
             if name is None:
                 raise ValueError(f"{path} ({part_spec.kind}) has no checkpoint name for its tensor {local!r}")
+            if any(isinstance(size, FreeSize) for size in param.shape):  # (free sizes agree inside one part)
+                param = ParamSpec(tuple(FreeSize(f"{path}.{size.name}", size) if isinstance(size, FreeSize) else size
+                                        for size in param.shape), param.init)
             if name in out and tuple(out[name].shape) != tuple(param.shape):
                 raise ValueError(f"tensor {name!r} is declared with shapes {out[name].shape} and {param.shape}")
             out.setdefault(name, param)
     return out
+
+
+def _fits(shape, wanted, free: dict[str, int]) -> bool:
+    """Whether a stored shape is the wanted one; `free` collects what the checkpoint decides for its free sizes."""
+    if len(shape) != len(wanted):
+        return False
+    for have, want in zip(shape, wanted):
+        if isinstance(want, FreeSize):
+            want = free.setdefault(want.name, int(have))
+        if have != want or have <= 0:
+            return False
+    return True
 
 
 def _keep(tensor: torch.Tensor) -> torch.Tensor:
@@ -74,9 +89,10 @@ def load_weights(folder: str, spec: ModelSpec) -> dict[str, torch.Tensor]:
                 where[name] = handle
         missing = [name for name in expected if name not in where]
         unexpected, wrong = [], []
+        free: dict[str, int] = {}
         for name, handle in where.items():
             if name in expected:
-                if tuple(handle.shape(name)) != tuple(expected[name].shape):
+                if not _fits(tuple(handle.shape(name)), tuple(expected[name].shape), free):
                     wrong.append((name, handle.shape(name), expected[name].shape))
                 elif handle.dtype(name) == torch.float64:
                     other.append(f"tensor {name} is stored as F64, which is not supported")

@@ -37,6 +37,8 @@ def random_tensors(config, seed: int, dtype: torch.dtype = torch.bfloat16, std: 
             values = 1.0 + values * (std / 2)
         else:
             values = values * std
+            if param.init == "last_one":
+                values[-1] += 1.0
         out[name] = values.to(dtype)
     return out
 
