@@ -1080,7 +1080,85 @@ def gaperax_rooflines(row: dict, size: dict, batch: int, peak: dict, contexts: l
     return out
 
 
-DESIGNS = {"gaperax": ("Gaperax", gaperax_config, ("revupel", "llama")), "tisalorn": ("Tisalorn", tisalorn_config, ("llama",)), "satavik": ("Satavik", satavik_config, ("llama",)),
+def tezinex_config(size: dict) -> dict:
+    """A Tezinex model of `size`: the delta rule by channels and windowed attention in turn, every second attention layer
+    reading the keys of the one before it; q and k heads of the delta rule as many as the other models' key/value heads,
+    a window of 1,024 positions that keeps the first 64, scores capped at 50, the dense feed-forward of the Llama model's
+    width behind every mixer."""
+    h, g, d = size["heads"], size["kv_heads"], size["dim"]
+    mlp = {"kind": "dense", "ff": size["ff"]}
+    layers = []
+    for i in range(size["layers"]):
+        if i % 2 == 0:
+            layers.append({"type": "channel_delta", "mlp": mlp, "mixer": {"heads": h, "kv_heads": g, "dim": d, "vdim": d,
+                                                                          "conv": 4}})
+            continue
+        mixer = {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 50.0,
+                 "mask": {"size": TEZINEX_WINDOW, "keep_first": TEZINEX_KEPT}}
+        if i % 4 == 3:
+            mixer["kv_from"] = i - 2
+        layers.append({"type": "attention", "mlp": mlp, "mixer": mixer})
+    return {"architecture": "Tezinex", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6},
+            "residual_mult": 0.5, "logit_softcap": 30.0, "max_position": 8192, "layers": layers}
+
+
+TEZINEX_WINDOW, TEZINEX_KEPT = 1024, 64
+
+
+def tezinex_rooflines(row: dict, size: dict, batch: int, peak: dict, contexts: list) -> dict:
+    """The new kernels and the kernels of the models beside that do the like work, each against its own roofline.
+    Attention: a prompt step against the multiply-adds of the (query, key) pairs its mask lets through at the bf16 tensor
+    rate, a decode step against the keys and values a token can see at the HBM rate; beside the Llama model's. The delta
+    rule's scan: a decode step against the matrices it reads and writes, a prompt step against its float32 multiply-adds
+    (three per matrix element and token: both read-outs and the write); beside the Tisalorn model's, whose decay is one
+    per head. What prepares the scan's inputs and what follows a sublayer: against the bytes they must move."""
+    h, g, d, width, ff = size["heads"], size["kv_heads"], size["dim"], size["width"], size["ff"]
+    reach, n = TEZINEX_WINDOW + TEZINEX_KEPT, PREFILL_TOKENS
+    out = {}
+
+    def put(name, work, kernel, unit):
+        if kernel and kernel["us"]:
+            rate = work / (kernel["us"] * 1e-6)
+            out[name] = round({"hbm": rate / 1e9 / peak["hbm_gbs"], "bf16": rate / 1e12 / peak["bf16_tflops"],
+                               "fp32": rate / (148 * 128 * 2 * 1.965e9)}[unit], 4)
+
+    pairs = sum(min(i + 1, reach) for i in range(n))
+    for model, name, seen, past in (("tezinex", "sink_attention", pairs, [min(c, reach) for c in contexts]),
+                                    ("llama", "attention", n * n / 2, contexts)):
+        put(f"{model}_attention_prefill_bf16_frac", 2 * h * 2 * d * seen, _first(row[model]["prefill_kernels"], name),
+            "bf16")
+        put(f"{model}_attention_decode_hbm_frac", 2 * sum(past) * g * 2 * d, _first(row[model]["decode_kernels"], name),
+            "hbm")
+    channels = 2 * g * d + h * d
+    for model, scan, prepare, more in (("tezinex", "channel_delta_scan", "channel_delta_prepare", 2 * h * d),
+                                       ("tisalorn", "delta_scan", "delta_prepare", 0)):
+        put(f"{model}_scan_decode_hbm_frac", 2 * 4 * batch * h * d * d, row[model]["decode_kernels"].get(scan), "hbm")
+        put(f"{model}_scan_prefill_fp32_frac", 2 * 3 * n * h * d * d, row[model]["prefill_kernels"].get(scan), "fp32")
+        put(f"{model}_prepare_prefill_hbm_frac", 4 * n * (2 * channels + more), row[model]["prefill_kernels"].get(prepare),
+            "hbm")
+        put(f"{model}_read_out_norm_prefill_hbm_frac", n * h * d * (4 + 4 + 2),
+            row[model]["prefill_kernels"].get("gated_norm"), "hbm")
+    # behind a sublayer: the stream in and out, the sublayer's output, the operand; at a layer's end also the earlier
+    # results and the new one (the mean over the model's launches)
+    layers = size["layers"]
+    moved = sum(14 + (14 + 4 * (i + 1) + 4) for i in range(layers)) / (2 * layers)
+    put("tezinex_stream_update_prefill_hbm_frac", moved * n * width, row["tezinex"]["prefill_kernels"].get("stream_update"),
+        "hbm")
+    put("tisalorn_norm_sum_prefill_hbm_frac", 16 * n * width, row["tisalorn"]["prefill_kernels"].get("norm_sum_residual"),
+        "hbm")
+    put("tisalorn_norm_prefill_hbm_frac", 6 * n * width, row["tisalorn"]["prefill_kernels"].get("layernorm"), "hbm")
+    for model in ("tezinex", "llama", "tisalorn"):
+        for phase, work, unit in (("decode", 2 * 3 * ff * width, "hbm"), ("prefill", 2 * n * 3 * ff * width, "bf16")):
+            kernels = row[model][phase + "_kernels"]
+            us = sum(k["us"] for name, k in kernels.items() if "swiglu" in name or "glu_clamped" in name
+                     or (name.startswith("gemm") and (f"K={ff}" in name or f"N={2 * ff} " in name)
+                         and "swiglu" not in name and "glu_clamped" not in name))
+            put(f"{model}_feed_forward_{phase}_{unit}_frac", work, {"us": us}, unit)
+    return out
+
+
+DESIGNS = {"gaperax": ("Gaperax", gaperax_config, ("revupel", "llama")),
+           "tezinex": ("Tezinex", tezinex_config, ("tisalorn", "llama")), "tisalorn": ("Tisalorn", tisalorn_config, ("llama",)), "satavik": ("Satavik", satavik_config, ("llama",)),
            "revupel": ("Revupel", revupel_config, ("satavik", "tisalorn"))}
 """--design NAME: the design's name, its configuration at a size, and the models it is measured beside."""
 
@@ -1166,6 +1244,8 @@ def design_comparison(args) -> int:
             row["roofline"] = tisalorn_rooflines(row, size, args.batch, peak)
         elif design == "satavik":
             row["roofline"] = satavik_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
+        elif design == "tezinex":
+            row["roofline"] = tezinex_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
         elif design == "gaperax":
             row["roofline"] = gaperax_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
         else:

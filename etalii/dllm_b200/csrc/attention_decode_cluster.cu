@@ -6,7 +6,11 @@
 // memory (mapa + ld.shared::cluster between two cluster barriers): no scratch in global memory, no atomics, and a
 // launch shape (blocks per pair, kv heads, sequences) that does not depend on the context length; the number of
 // blocks per pair follows from how many pairs there are. head_dim: a multiple of 16 up to 128.
-#include "common.cuh"
+//
+// Instantiated with OPTIONS (score_options.cuh; sink_attention_decode.cu does) the scores may be capped, the denominator
+// holds a sink, the window keeps a sequence's first positions (the tiles are then those of kept positions followed by
+// those of the window) and the values may have another size than the keys (HD covers both; multiples of 8).
+#include "score_options.cuh"
 
 namespace {
 typedef __nv_bfloat16 bf16;
@@ -51,10 +55,10 @@ __device__ __forceinline__ float remote_float(const float* local, unsigned rank)
 
 // CLUSTER blocks of WARPS warps serve one (sequence, kv head). Few (sequence, kv head) pairs: many blocks per pair
 // to fill the device and shorten every chain of pages; many pairs: one block per pair, no exchange between blocks.
-template <int HD, int CLUSTER, int WARPS>
+template <int HD, int CLUSTER, int WARPS, bool OPTIONS>
 __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
     bf16* __restrict__ out, const bf16* __restrict__ q, KvLayout cache, const int* __restrict__ tok_pos,
-    const int* __restrict__ slots, int heads, float scale_log2, int window) {
+    const int* __restrict__ slots, int heads, float scale_log2, int window, ScoreOptions options) {
   constexpr int LD = HD + 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* kv_s = reinterpret_cast<bf16*>(smem_raw);        // per warp: K [64][LD], V [64][LD]
@@ -67,25 +71,36 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
   int b = blockIdx.z, g = blockIdx.y;
   unsigned rank = blockIdx.x;  // cluster dims are (CLUSTER, 1, 1) and gridDim.x == CLUSTER
   int hd = cache.head_dim;
+  int vd = OPTIONS ? options.value_dim : hd;
   int group = heads / cache.kv_heads;
+  const WideKv wide{cache.base, cache.page_table, cache.max_pages, cache.page_size, cache.kv_heads, hd, vd};
+  auto keys_of = [&](int page, int row) { return OPTIONS ? key_at(wide, page, g, row) : kv_offset(cache, page, 0, g, row); };
+  auto values_of = [&](int page, int row) {
+    return OPTIONS ? value_at(wide, page, g, row) : kv_offset(cache, page, 1, g, row);
+  };
   pdl_launch_dependents();
   int end = tok_pos[b] + 1;    // positions and slots are written only by the step's last kernel
   int first = (window > 0 && end > window) ? end - window : 0;
   int base = (first / TILE_KEYS) * TILE_KEYS;
+  // tile number `it` of the walk starts at key key_of(it)
+  const KeyWalk walk(end - 1, end - 1, window, OPTIONS ? options.keep : 0, TILE_KEYS);
+  auto key_of = [&](int it) { return OPTIONS ? walk.tile(it) * TILE_KEYS : base + it * TILE_KEYS; };
+  const int tiles = OPTIONS ? walk.count : (end - base + TILE_KEYS - 1) / TILE_KEYS;
+  const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
   int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   int gq = lane >> 2, tq = lane & 3;
   const int* pages = cache.page_table + (size_t)slots[b] * cache.max_pages;
   bf16* k_s = kv_s + (size_t)warp * 2 * TILE_KEYS * LD;
   bf16* v_s = k_s + TILE_KEYS * LD;
-  int chunks16 = hd >> 3;
+  int chunks16 = hd >> 3, value_chunks = vd >> 3;
   int newest = end - 1;
-  constexpr int ROUND = CLUSTER * WARPS * TILE_KEYS;
+  constexpr int ROUND = CLUSTER * WARPS;  // tiles that all warps together take at a time
 
   auto copy_page = [&](int key0) {
     int page = pages[key0 / TILE_KEYS];
-    const bf16* ksrc = (const bf16*)cache.base + kv_offset(cache, page, 0, g, 0);
-    const bf16* vsrc = (const bf16*)cache.base + kv_offset(cache, page, 1, g, 0);
-    if (hd == HD) {
+    const bf16* ksrc = (const bf16*)cache.base + keys_of(page, 0);
+    const bf16* vsrc = (const bf16*)cache.base + values_of(page, 0);
+    if (hd == HD && vd == HD) {
 #pragma unroll
       for (int i = 0; i < TILE_KEYS * (HD / 8) / 32; ++i) {
         int idx = lane + 32 * i;
@@ -96,13 +111,10 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
     } else {
       for (int idx = lane; idx < TILE_KEYS * (HD / 8); idx += 32) {
         int r = idx / (HD / 8), cc = idx % (HD / 8);
-        if (cc < chunks16) {
-          cp_async_16(k_s + r * LD + cc * 8, ksrc + (size_t)r * hd + cc * 8);
-          cp_async_16(v_s + r * LD + cc * 8, vsrc + (size_t)r * hd + cc * 8);
-        } else {
-          *reinterpret_cast<uint4*>(k_s + r * LD + cc * 8) = make_uint4(0u, 0u, 0u, 0u);
-          *reinterpret_cast<uint4*>(v_s + r * LD + cc * 8) = make_uint4(0u, 0u, 0u, 0u);
-        }
+        if (cc < chunks16) cp_async_16(k_s + r * LD + cc * 8, ksrc + (size_t)r * hd + cc * 8);
+        else *reinterpret_cast<uint4*>(k_s + r * LD + cc * 8) = make_uint4(0u, 0u, 0u, 0u);
+        if (cc < value_chunks) cp_async_16(v_s + r * LD + cc * 8, vsrc + (size_t)r * vd + cc * 8);
+        else *reinterpret_cast<uint4*>(v_s + r * LD + cc * 8) = make_uint4(0u, 0u, 0u, 0u);
       }
     }
     asm volatile("cp.async.commit_group;\n" ::);
@@ -111,21 +123,22 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
 
   // this warp's first page: keys of earlier steps do not change any more, so it is copied before the wait on the
   // projection kernel; the row that kernel writes (position end - 1) is read again after the wait
-  int my_first = base + ((int)rank * WARPS + warp) * TILE_KEYS;
-  int page0 = 0;
-  if (my_first < end) page0 = copy_page(my_first);
+  int my_first = (int)rank * WARPS + warp;
+  if (my_first < tiles) copy_page(key_of(my_first));
   // The tile that holds the newest key belongs to one warp of the cluster. That warp asks for the row right after
   // the wait, together with the queries, and puts it into its shared-memory page when the tile's turn comes: the
   // round trip runs under the wait for the page instead of after it.
   int newest_tile = (newest / TILE_KEYS) * TILE_KEYS;
-  bool owns_newest = newest_tile >= my_first && (newest_tile - my_first) % ROUND == 0;
+  bool owns_newest = tiles - 1 >= my_first && (tiles - 1 - my_first) % ROUND == 0;  // (it is in the walk's last tile)
   uint4 newest_k = make_uint4(0u, 0u, 0u, 0u), newest_v = newest_k;
   pdl_wait();
-  if (owns_newest && lane < chunks16) {
+  if (owns_newest) {
     int page = pages[newest / TILE_KEYS];
     int r = newest - newest_tile;
-    newest_k = __ldcg(reinterpret_cast<const uint4*>((const bf16*)cache.base + kv_offset(cache, page, 0, g, r)) + lane);
-    newest_v = __ldcg(reinterpret_cast<const uint4*>((const bf16*)cache.base + kv_offset(cache, page, 1, g, r)) + lane);
+    if (lane < chunks16)
+      newest_k = __ldcg(reinterpret_cast<const uint4*>((const bf16*)cache.base + keys_of(page, r)) + lane);
+    if (lane < value_chunks)
+      newest_v = __ldcg(reinterpret_cast<const uint4*>((const bf16*)cache.base + values_of(page, r)) + lane);
   }
 
   for (int h0 = 0; h0 < group; h0 += 16) {
@@ -150,17 +163,15 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
       }
     }
     // (the very first page is already on its way; a later pass over the heads starts again at the first page)
-    int page = page0;
-    if (h0 != 0 && my_first < end) page = copy_page(my_first);
-    for (int key0 = my_first; key0 < end; key0 += ROUND) {
+    if (h0 != 0 && my_first < tiles) copy_page(key_of(my_first));
+    for (int it = my_first; it < tiles; it += ROUND) {
+      const int key0 = key_of(it);
       asm volatile("cp.async.wait_group 0;\n" ::);
       __syncwarp();
       if (key0 == newest_tile) {  // the row the projection kernel has just written (chunks16 <= 16 lanes hold it)
         int r = newest - key0;
-        if (lane < chunks16) {
-          *reinterpret_cast<uint4*>(k_s + r * LD + lane * 8) = newest_k;
-          *reinterpret_cast<uint4*>(v_s + r * LD + lane * 8) = newest_v;
-        }
+        if (lane < chunks16) *reinterpret_cast<uint4*>(k_s + r * LD + lane * 8) = newest_k;
+        if (lane < value_chunks) *reinterpret_cast<uint4*>(v_s + r * LD + lane * 8) = newest_v;
         __syncwarp();
       }
       float s[TILE_KEYS / 8][4];
@@ -179,13 +190,19 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
           mma_bf16(s[2 * jp + 1], q_frag[ks], bfr[2], bfr[3]);
         }
       }
+      if (OPTIONS) {  // from here on in units of log2 e
+#pragma unroll
+        for (int j = 0; j < TILE_KEYS / 8; ++j)
+#pragma unroll
+          for (int r = 0; r < 4; ++r) s[j][r] = score.any(s[j][r]);
+      }
       if (key0 < first || key0 + TILE_KEYS > end) {  // a tile with an edge: keys outside [first, end) do not count
 #pragma unroll
         for (int j = 0; j < TILE_KEYS / 8; ++j)
 #pragma unroll
           for (int r = 0; r < 4; ++r) {
             int key = key0 + j * 8 + tq * 2 + (r & 1);
-            if (key < first || key >= end) s[j][r] = -INFINITY;
+            if ((key < first && (!OPTIONS || key >= options.keep)) || key >= end) s[j][r] = -INFINITY;
           }
       }
       float tile_max[2] = {-INFINITY, -INFINITY};
@@ -194,11 +211,12 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
 #pragma unroll
         for (int r = 0; r < 4; ++r) tile_max[r >> 1] = fmaxf(tile_max[r >> 1], s[j][r]);
       float corr[2], neg_max[2];
+      const float unit = OPTIONS ? 1.0f : scale_log2;
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         tile_max[i] = fmaxf(tile_max[i], __shfl_xor_sync(0xffffffffu, tile_max[i], 1));
         tile_max[i] = fmaxf(tile_max[i], __shfl_xor_sync(0xffffffffu, tile_max[i], 2));
-        float m_new = fmaxf(m_run[i], tile_max[i] * scale_log2);  // maxima live in the scaled log2 domain
+        float m_new = fmaxf(m_run[i], tile_max[i] * unit);  // maxima live in the scaled log2 domain
         corr[i] = fast_exp2(m_run[i] - m_new);
         m_run[i] = m_new;
         neg_max[i] = -m_new;
@@ -207,8 +225,8 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
       unsigned p_frag[TILE_KEYS / 16][4];
 #pragma unroll
       for (int j = 0; j < TILE_KEYS / 8; ++j) {
-        float p0 = fast_exp2(fmaf(s[j][0], scale_log2, neg_max[0])), p1 = fast_exp2(fmaf(s[j][1], scale_log2, neg_max[0]));
-        float p2 = fast_exp2(fmaf(s[j][2], scale_log2, neg_max[1])), p3 = fast_exp2(fmaf(s[j][3], scale_log2, neg_max[1]));
+        float p0 = fast_exp2(fmaf(s[j][0], unit, neg_max[0])), p1 = fast_exp2(fmaf(s[j][1], unit, neg_max[0]));
+        float p2 = fast_exp2(fmaf(s[j][2], unit, neg_max[1])), p3 = fast_exp2(fmaf(s[j][3], unit, neg_max[1]));
         row_sum[0] += p0 + p1;
         row_sum[1] += p2 + p3;
         p_frag[j >> 1][(j & 1) * 2 + 0] = pack_bf16(p0, p1);
@@ -233,7 +251,7 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
         }
       }
       __syncwarp();  // the page's space is free for the next copy
-      if (key0 + ROUND < end) page = copy_page(key0 + ROUND);
+      if (it + ROUND < tiles) copy_page(key_of(it + ROUND));
     }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -268,21 +286,24 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
       cta_o[h * HD + d] = o;
       if (d == 0) { cta_ml[h][0] = m; cta_ml[h][1] = l; }
     }
+    const int out_row = OPTIONS ? options.out_stride : heads * hd;
     if (CLUSTER == 1) {
       __syncthreads();
-      for (int idx = threadIdx.x; idx < nh * hd; idx += WARPS * 32) {
-        int h = idx / hd, d = idx % hd;
-        out[((size_t)b * heads + g * group + h0 + h) * hd + d] = __float2bfloat16_rn(cta_o[h * HD + d] / cta_ml[h][1]);
+      for (int idx = threadIdx.x; idx < nh * vd; idx += WARPS * 32) {
+        int h = idx / vd, d = idx % vd, head = g * group + h0 + h;
+        float value = OPTIONS ? cta_o[h * HD + d] * sink_factor(cta_ml[h][0], cta_ml[h][1], options.sinks, head)
+                              : cta_o[h * HD + d] / cta_ml[h][1];
+        out[(size_t)b * out_row + head * vd + d] = __float2bfloat16_rn(value);
       }
     } else {
       cluster_sync();  // every block's partial result is in its shared memory
       // The outputs (head, dimension) are dealt out to the blocks of the cluster in equal runs; a thread asks for all
       // blocks' values of its output before it touches the first (one round trip through distributed shared memory,
       // not one per block), then sums in rank order.
-      int total = nh * hd, per = (total + CLUSTER - 1) / CLUSTER;
+      int total = nh * vd, per = (total + CLUSTER - 1) / CLUSTER;
       int stop = min(total, ((int)rank + 1) * per);
       for (int idx = (int)rank * per + threadIdx.x; idx < stop; idx += WARPS * 32) {
-        int h = idx / hd, d = idx % hd;
+        int h = idx / vd, d = idx % vd, head = g * group + h0 + h;
         float mr[CLUSTER], lr[CLUSTER], orr[CLUSTER];
 #pragma unroll
         for (unsigned r = 0; r < CLUSTER; ++r) {
@@ -300,7 +321,8 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
           o = fmaf(orr[r], f, o);
           l = fmaf(lr[r], f, l);
         }
-        out[((size_t)b * heads + g * group + h0 + h) * hd + d] = __float2bfloat16_rn(o / l);
+        out[(size_t)b * out_row + head * vd + d] =
+            __float2bfloat16_rn(OPTIONS ? o * sink_factor(m, l, options.sinks, head) : o / l);
       }
     }
     if (CLUSTER > 1) cluster_sync();  // nobody leaves (or reuses the space) while others still read its partial result
@@ -315,13 +337,13 @@ constexpr size_t block_smem() {
   return kv_bytes > red_bytes ? kv_bytes : red_bytes;
 }
 
-template <int HD, int CLUSTER, int WARPS>
+template <int HD, int CLUSTER, int WARPS, bool OPTIONS>
 int launch(void* out, const void* q, const KvLayout& cache, const int* tok_pos, const int* slots, int heads,
-           int sequences, float scale, int window, cudaStream_t stream) {
+           int sequences, float scale, int window, const ScoreOptions& options, cudaStream_t stream) {
   constexpr size_t smem = block_smem<HD, WARPS>();
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(decode_attention_cluster_kernel<HD, CLUSTER, WARPS>,
+    if (cudaFuncSetAttribute(decode_attention_cluster_kernel<HD, CLUSTER, WARPS, OPTIONS>,
                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return DLLM_LAUNCH_FAILED;
     configured = true;
@@ -340,8 +362,8 @@ int launch(void* out, const void* q, const KvLayout& cache, const int* tok_pos, 
   attributes[1].val.programmaticStreamSerializationAllowed = 1;
   config.attrs = attributes;
   config.numAttrs = dllm_pdl_enabled() ? 2 : 1;
-  return cudaLaunchKernelEx(&config, decode_attention_cluster_kernel<HD, CLUSTER, WARPS>, (bf16*)out, (const bf16*)q,
-                            cache, tok_pos, slots, heads, scale * 1.4426950408889634f, window) == cudaSuccess
+  return cudaLaunchKernelEx(&config, decode_attention_cluster_kernel<HD, CLUSTER, WARPS, OPTIONS>, (bf16*)out, (const bf16*)q,
+                            cache, tok_pos, slots, heads, scale * SCORE_LOG2E, window, options) == cudaSuccess
              ? DLLM_OK
              : DLLM_LAUNCH_FAILED;
 }
@@ -354,9 +376,9 @@ int launch(void* out, const void* q, const KvLayout& cache, const int* tok_pos, 
 constexpr int SHAPES = 5;
 constexpr size_t SMEM_PER_SM = 227 * 1024;
 
-template <int HD>
+template <int HD, bool OPTIONS>
 int launch_shape(int shape, void* out, const void* q, const KvLayout& cache, const int* tok_pos, const int* slots,
-                 int heads, int sequences, float scale, int window, cudaStream_t stream) {
+                 int heads, int sequences, float scale, int window, const ScoreOptions& options, cudaStream_t stream) {
   constexpr int NW = HD > 64 ? 2 : 4;
   if (shape < 0) {
     static int sms = 0;
@@ -377,7 +399,7 @@ int launch_shape(int shape, void* out, const void* q, const KvLayout& cache, con
     if (HD > 64 && shape == 0 && pairs <= 4 * places) shape = 1;
   }
 #define DLLM_GO(CL, WARPS) \
-  return launch<HD, CL, WARPS>(out, q, cache, tok_pos, slots, heads, sequences, scale, window, stream)
+  return launch<HD, CL, WARPS, OPTIONS>(out, q, cache, tok_pos, slots, heads, sequences, scale, window, options, stream)
   switch (shape) {
     case 0: DLLM_GO(1, NW);
     case 1: DLLM_GO(2, NW);
@@ -390,6 +412,7 @@ int launch_shape(int shape, void* out, const void* q, const KvLayout& cache, con
 }
 }  // namespace
 
+#ifndef DLLM_DECODE_CLUSTER_OPTIONS  // (a file that includes this one for the instantiations with options exports its own)
 // out, q: [sequences, heads * head_dim] bfloat16; sequence b's query is the token at tok_pos[b], whose key and value
 // are already in the cache. head_dim a multiple of 16 up to 128, pages of 64 positions, at most 65,535 sequences.
 // shape: -1 chooses by the number of (sequence, kv head) pairs; 0..4 name a launch shape (see above).
@@ -403,7 +426,11 @@ DLLM_EXPORT int dllm_attention_decode_cluster(void* out, const void* q, void* ca
       kv_heads > 65535)
     return DLLM_UNSUPPORTED_SIZE;
   KvLayout cache{cache_base, page_table, max_pages, page_size, kv_heads, head_dim};
-  if (head_dim <= 32) return launch_shape<32>(shape, out, q, cache, tok_pos, slots, heads, sequences, scale, window, stream);
-  if (head_dim <= 64) return launch_shape<64>(shape, out, q, cache, tok_pos, slots, heads, sequences, scale, window, stream);
-  return launch_shape<128>(shape, out, q, cache, tok_pos, slots, heads, sequences, scale, window, stream);
+  const ScoreOptions none = {};
+  if (head_dim <= 32)
+    return launch_shape<32, false>(shape, out, q, cache, tok_pos, slots, heads, sequences, scale, window, none, stream);
+  if (head_dim <= 64)
+    return launch_shape<64, false>(shape, out, q, cache, tok_pos, slots, heads, sequences, scale, window, none, stream);
+  return launch_shape<128, false>(shape, out, q, cache, tok_pos, slots, heads, sequences, scale, window, none, stream);
 }
+#endif

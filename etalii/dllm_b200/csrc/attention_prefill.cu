@@ -8,7 +8,11 @@
 //
 // head_dim: any multiple of 16 up to 128 (the kernel is instantiated for 32, 64 and 128 and pads with zeros).
 // The page size must be 64.
-#include "common.cuh"
+//
+// Instantiated with OPTIONS (score_options.cuh; sink_attention_prefill.cu does) the scores may be capped, the denominator
+// holds a sink, the window keeps a sequence's first positions and the values may have another size than the keys (HD
+// covers both; multiples of 8).
+#include "score_options.cuh"
 
 namespace {
 typedef __nv_bfloat16 bf16;
@@ -43,11 +47,11 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-template <int HD>
-__global__ void __launch_bounds__(THREADS) prefill_kernel(
+template <int HD, bool OPTIONS>
+__global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
     bf16* __restrict__ out, const bf16* __restrict__ q, KvLayout cache, const int* __restrict__ tile_seq,
     const int* __restrict__ tile_first, const int* __restrict__ cu_seqlens, const int* __restrict__ start,
-    const int* __restrict__ slots, int heads, float scale_log2, int window) {
+    const int* __restrict__ slots, int heads, float scale_log2, int window, ScoreOptions options) {
   constexpr int LD = HD + 8;  // padded row, keeps 16-byte alignment
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw);            // [BM][LD]
@@ -57,6 +61,7 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   int tile = blockIdx.x, h = blockIdx.y;
   int b = tile_seq[tile], q0 = tile_first[tile];
   int hd = cache.head_dim;
+  int vd = OPTIONS ? options.value_dim : hd;
   int g = h / (heads / cache.kv_heads);
   int n_new = cu_seqlens[b + 1] - cu_seqlens[b];
   int tok0 = cu_seqlens[b] + q0;           // first token row of this tile in the packed batch
@@ -65,7 +70,8 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   const int* pages = cache.page_table + (size_t)slots[b] * cache.max_pages;
   const bf16* base = (const bf16*)cache.base;
   int tid = threadIdx.x % (WARPS * 32), lane = tid & 31, warp = tid >> 5;  // within the group
-  int chunks = hd >> 3;                    // 16-byte pieces of a real row
+  int chunks = hd >> 3, value_chunks = vd >> 3;  // 16-byte pieces of a real row
+  const WideKv wide{cache.base, cache.page_table, cache.max_pages, cache.page_size, cache.kv_heads, hd, vd};
   auto group_sync = [&]() { asm volatile("bar.sync %0, %1;" ::"r"(group + 1), "r"(WARPS * 32) : "memory"); };
 
   // queries -> shared memory (rows beyond the tile and dims beyond head_dim are zero)
@@ -76,19 +82,20 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
     cp_async_16(q_s + r * LD + c * 8, src, ok);
   }
   int last_pos = pos0 + rows - 1;                                   // last query's position
-  int kt_end = last_pos / BN;                                       // last key tile any query of the tile sees
-  int kt_begin = (window > 0 && pos0 + 1 > window) ? (pos0 + 1 - window) / BN : 0;
+  // the key tiles the block's queries see between them, by their number in the walk
+  const KeyWalk walk(pos0, last_pos, window, OPTIONS ? options.keep : 0, BN);
+  const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
   // the pages of the key tiles this block will read, fetched once (not one dependent load per tile)
   __shared__ int page_s[MAX_TILES];
-  for (int i = threadIdx.x; i <= kt_end - kt_begin && i < MAX_TILES; i += THREADS) page_s[i] = pages[kt_begin + i];
+  for (int i = threadIdx.x; i < walk.count && i < MAX_TILES; i += THREADS) page_s[i] = pages[walk.tile(i)];
   __syncthreads();
 
   const int flat_dst = (tid / (HD / 8)) * LD + (tid % (HD / 8)) * 8, flat_src = tid * 8;
-  auto load_kv = [&](int stage, int kt) {
-    int page = kt - kt_begin < MAX_TILES ? page_s[kt - kt_begin] : pages[kt];
-    const bf16* ksrc = base + kv_offset(cache, page, 0, g, 0);
-    const bf16* vsrc = base + kv_offset(cache, page, 1, g, 0);
-    if (hd == HD) {
+  auto load_kv = [&](int stage, int it) {
+    int page = it < MAX_TILES ? page_s[it] : pages[walk.tile(it)];
+    const bf16* ksrc = base + (OPTIONS ? key_at(wide, page, g, 0) : kv_offset(cache, page, 0, g, 0));
+    const bf16* vsrc = base + (OPTIONS ? value_at(wide, page, g, 0) : kv_offset(cache, page, 1, g, 0));
+    if (hd == HD && vd == HD) {
       // the page is one flat piece; each thread's pieces sit at fixed offsets (computed once, below)
 #pragma unroll
       for (int i = 0; i < BN * (HD / 8) / (WARPS * 32); ++i) {
@@ -100,14 +107,13 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
     } else {
       for (int idx = tid; idx < BN * (HD / 8); idx += WARPS * 32) {
         int r = idx / (HD / 8), c = idx % (HD / 8);
-        bool ok = c < chunks;
+        bool ok = c < chunks, value_ok = c < value_chunks;
         cp_async_16(k_s + (stage * BN + r) * LD + c * 8, ok ? ksrc + (size_t)r * hd + c * 8 : ksrc, ok);
-        cp_async_16(v_s + (stage * BN + r) * LD + c * 8, ok ? vsrc + (size_t)r * hd + c * 8 : vsrc, ok);
+        cp_async_16(v_s + (stage * BN + r) * LD + c * 8, value_ok ? vsrc + (size_t)r * vd + c * 8 : vsrc, value_ok);
       }
     }
   };
-  int kt_first = kt_begin + group;          // this group's tiles: kt_first, kt_first + GROUPS, ...
-  if (kt_first <= kt_end) load_kv(0, kt_first);
+  if (group < walk.count) load_kv(0, group);  // this group's tiles: group, group + GROUPS, ... of the walk
   cp_async_commit();
   cp_async_wait<0>();
   __syncthreads();  // the queries were copied by all threads of the block: both groups may read them from here on
@@ -123,9 +129,9 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   int row_pos[2] = {pos0 + warp * 16 + gq, pos0 + warp * 16 + gq + 8};  // positions of this thread's two rows
 
   bool have_q = false;
-  for (int kt = kt_first; kt <= kt_end; kt += GROUPS) {
-    int stage = ((kt - kt_first) / GROUPS) & 1;
-    if (kt + GROUPS <= kt_end) load_kv(stage ^ 1, kt + GROUPS);
+  for (int it = group; it < walk.count; it += GROUPS) {
+    int stage = ((it - group) / GROUPS) & 1;
+    if (it + GROUPS < walk.count) load_kv(stage ^ 1, it + GROUPS);
     cp_async_commit();
     cp_async_wait<1>();
     group_sync();
@@ -154,8 +160,27 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
       }
     }
     // scale (log2 domain), masks, running maximum
-    int key0 = kt * BN;
+    int key0 = walk.tile(it) * BN;
     bool need_mask = key0 + BN - 1 > pos0 + warp * 16 || (window > 0 && key0 < pos0 + warp * 16 + 16 - window);
+    const float unit = OPTIONS ? 1.0f : scale_log2;  // what a score still has to be multiplied by
+    if (OPTIONS) {
+      float largest = 0.f;
+#pragma unroll
+      for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+        for (int r = 0; r < 4; ++r) largest = fmaxf(largest, fabsf(s[j][r]));
+      if (score.in == 0.f || __all_sync(0xffffffffu, largest <= score.small_up_to)) {
+#pragma unroll
+        for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+          for (int r = 0; r < 4; ++r) s[j][r] = score.small(s[j][r]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < BN / 8; ++j)
+#pragma unroll
+          for (int r = 0; r < 4; ++r) s[j][r] = score.any(s[j][r]);
+      }
+    }
     float tile_max[2] = {-INFINITY, -INFINITY};
     if (need_mask) {
 #pragma unroll
@@ -164,7 +189,7 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
         for (int r = 0; r < 4; ++r) {
           int key = key0 + j * 8 + tq * 2 + (r & 1);
           int qp = row_pos[r >> 1];
-          if (key > qp || (window > 0 && key < qp + 1 - window)) s[j][r] = -INFINITY;
+          if (key > qp || (window > 0 && key < qp + 1 - window && (!OPTIONS || key >= options.keep))) s[j][r] = -INFINITY;
         }
     }
 #pragma unroll
@@ -176,7 +201,7 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
     for (int i = 0; i < 2; ++i) {
       tile_max[i] = fmaxf(tile_max[i], __shfl_xor_sync(0xffffffffu, tile_max[i], 1));
       tile_max[i] = fmaxf(tile_max[i], __shfl_xor_sync(0xffffffffu, tile_max[i], 2));
-      tile_max[i] *= scale_log2;  // maxima live in the scaled log2 domain; the scores are scaled inside the exponent
+      tile_max[i] *= unit;  // maxima live in the scaled log2 domain; the scores are scaled inside the exponent
       float m_new = fmaxf(m_run[i], tile_max[i]);
       float m_use = m_new == -INFINITY ? 0.f : m_new;  // a row that sees nothing in this tile (and nothing before)
       corr[i] = fast_exp2(m_run[i] - m_use);
@@ -187,8 +212,8 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
     unsigned p_frag[BN / 16][4];
 #pragma unroll
     for (int j = 0; j < BN / 8; ++j) {
-      float p0 = fast_exp2(fmaf(s[j][0], scale_log2, -tile_max[0])), p1 = fast_exp2(fmaf(s[j][1], scale_log2, -tile_max[0]));
-      float p2 = fast_exp2(fmaf(s[j][2], scale_log2, -tile_max[1])), p3 = fast_exp2(fmaf(s[j][3], scale_log2, -tile_max[1]));
+      float p0 = fast_exp2(fmaf(s[j][0], unit, -tile_max[0])), p1 = fast_exp2(fmaf(s[j][1], unit, -tile_max[0]));
+      float p2 = fast_exp2(fmaf(s[j][2], unit, -tile_max[1])), p3 = fast_exp2(fmaf(s[j][3], unit, -tile_max[1]));
       row_sum[0] += p0 + p1;
       row_sum[1] += p2 + p3;
       p_frag[j >> 1][(j & 1) * 2 + 0] = pack_bf16(p0, p1);
@@ -247,6 +272,7 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
       mine[i] = fast_exp2(m_run[i] - m_use);
       theirs[i] = fast_exp2(other_m[i] - m_use);
       l_run[i] = l_run[i] * mine[i] + other_l[i] * theirs[i];
+      m_run[i] = m_use;
     }
 #pragma unroll
     for (int i = 0; i < HD / 8; ++i)
@@ -259,36 +285,37 @@ __global__ void __launch_bounds__(THREADS) prefill_kernel(
   for (int half = 0; half < 2; ++half) {
     int r = warp * 16 + gq + half * 8;
     if (r >= rows) continue;
-    float inv = 1.0f / l_run[half];
-    bf16* dst = out + ((size_t)(tok0 + r) * heads + h) * hd;
+    float inv = OPTIONS ? sink_factor(m_run[half], l_run[half], options.sinks, h) : 1.0f / l_run[half];
+    bf16* dst = out + (OPTIONS ? (size_t)(tok0 + r) * options.out_stride + h * vd : ((size_t)(tok0 + r) * heads + h) * hd);
 #pragma unroll
     for (int i = 0; i < HD / 8; ++i) {
       int d = i * 8 + tq * 2;
-      if (d < hd) *reinterpret_cast<__nv_bfloat162*>(dst + d) =
+      if (d < vd) *reinterpret_cast<__nv_bfloat162*>(dst + d) =
           __floats2bfloat162_rn(o_acc[i][half * 2] * inv, o_acc[i][half * 2 + 1] * inv);
     }
   }
 }
 
-template <int HD>
+template <int HD, bool OPTIONS>
 int launch(void* out, const void* q, const KvLayout& cache, const int* tile_seq, const int* tile_first,
            const int* cu_seqlens, const int* start, const int* slots, int tiles, int heads, float scale, int window,
-           cudaStream_t stream) {
+           const ScoreOptions& options, cudaStream_t stream) {
   size_t smem = (size_t)(BM + GROUPS * 4 * BN) * (HD + 8) * sizeof(bf16);
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(prefill_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(prefill_kernel<HD, OPTIONS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return DLLM_LAUNCH_FAILED;
     configured = true;
   }
   dim3 grid(tiles, heads);
-  prefill_kernel<HD><<<grid, THREADS, smem, stream>>>((bf16*)out, (const bf16*)q, cache, tile_seq, tile_first,
+  prefill_kernel<HD, OPTIONS><<<grid, THREADS, smem, stream>>>((bf16*)out, (const bf16*)q, cache, tile_seq, tile_first,
                                                       cu_seqlens, start, slots, heads,
-                                                      scale * 1.4426950408889634f, window);
+                                                      scale * SCORE_LOG2E, window, options);
   return dllm_launch_status();
 }
 }  // namespace
 
+#ifndef DLLM_PREFILL_OPTIONS  // (a file that includes this one for the instantiations with options exports its own)
 // out, q: [tokens, heads * head_dim] bfloat16. tile_seq / tile_first: for each tile of up to 64 new tokens, its
 // sequence and the index of its first token among the sequence's new tokens. The keys and values of the new tokens
 // are already in the cache.
@@ -302,9 +329,14 @@ DLLM_EXPORT int dllm_attention_prefill(void* out, const void* q, void* cache_bas
   if (head_dim <= 0 || head_dim > 128 || (head_dim & 15) || page_size != BN || heads > 65535)
     return DLLM_UNSUPPORTED_SIZE;
   KvLayout cache{cache_base, page_table, max_pages, page_size, kv_heads, head_dim};
+  const ScoreOptions none = {};
   if (head_dim <= 32)
-    return launch<32>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window, stream);
+    return launch<32, false>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window, none,
+                      stream);
   if (head_dim <= 64)
-    return launch<64>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window, stream);
-  return launch<128>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window, stream);
+    return launch<64, false>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window, none,
+                      stream);
+  return launch<128, false>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window, none,
+                      stream);
 }
+#endif

@@ -21,6 +21,11 @@
 // between the two sets of buffers itself) and the block has seven warps.
 // Every wait on an mbarrier is bounded; a role that gives up records a status word and leaves, the block still frees
 // its tensor memory and the host raises.
+//
+// Instantiated with OPTIONS (score_options.cuh; sink_attention_tcgen05.cu does) the scores may be capped, the denominator
+// holds a sink and the window keeps a sequence's first positions (the steps then walk the pages of kept positions and
+// after them those of the windows).
+#include "score_options.cuh"
 #include "tcgen05.cuh"
 
 namespace {
@@ -49,12 +54,12 @@ struct Barriers {
   uint64_t s_full[2], s_empty[2], p_full[2], o_full[2], o_empty[2];
 };
 
-template <int HD>
+template <int HD, bool OPTIONS>
 __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, bf16* __restrict__ out,
     KvLayout cache, const int* __restrict__ tile_seq, const int* __restrict__ tile_first,
     const int* __restrict__ cu_seqlens, const int* __restrict__ start, const int* __restrict__ slots, int heads,
-    float scale_log2, int window, int* __restrict__ status) {
+    float scale_log2, int window, int* __restrict__ status, ScoreOptions options) {
   typedef Shape<HD> S;
   constexpr int GROUPS = S::GROUPS, SOFT_WARPS = S::SOFT_WARPS, Q_BYTES = S::Q_BYTES, KV_BYTES = S::KV_BYTES;
   constexpr unsigned TMEM_COLS = S::TMEM_COLS;
@@ -79,9 +84,9 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
   int rows = min(BQ, n_new - q0);          // queries of this tile that exist
   int pos0 = start[b] + q0;                // absolute position of the tile's first query
   int last_pos = pos0 + rows - 1;
-  int kt_end = last_pos / BKV;             // last page any query of the tile sees
-  int kt_begin = (window > 0 && pos0 + 1 > window) ? (pos0 + 1 - window) / BKV : 0;
-  int steps = kt_end - kt_begin + 1;
+  // the pages the tile's queries see between them: step j takes page walk.tile(j) of the sequence
+  const KeyWalk walk(pos0, last_pos, window, OPTIONS ? options.keep : 0, BKV);
+  const int steps = walk.count;
   const int* pages = cache.page_table + (size_t)slots[b] * cache.max_pages;
 
   if (threadIdx.x == 0) {
@@ -115,7 +120,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
       for (int j = 0; j < steps; ++j) {
         int s = j % STAGES;
         unsigned parity = ((j / STAGES) - 1) & 1;
-        int page = pages[kt_begin + j];
+        int page = pages[walk.tile(j)];
         int row_k = ((page * 2 + 0) * cache.kv_heads + g) * BKV, row_v = ((page * 2 + 1) * cache.kv_heads + g) * BKV;
         if (j >= STAGES && !mbar_wait(&bar.k_empty[s], parity)) { *(volatile int*)status = 12; break; }
         mbar_expect_tx(&bar.k_full[s], KV_BYTES);
@@ -183,6 +188,8 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     for (int d = 0; d < HD; ++d) o[d] = 0.f;
     float m_run = -INFINITY, l_run = 0.f, corr_saved = 1.f;
     bool ok = true;
+    const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
+    const float unit = OPTIONS ? 1.0f : scale_log2;  // what a score still has to be multiplied by in the sweep
     // fold step i's output into the running one: O = O * corr + P V
     auto consume = [&](int i, float corr) -> bool {
       const int ob = i & 1;
@@ -218,10 +225,11 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
         break;
       }
       fence_after_sync();
-      int key0 = (kt_begin + j) * BKV;
+      int key0 = walk.tile(j) * BKV;
       // a tile with an edge for some row of the block: keys beyond the query, or before its window
       bool edge = key0 + BKV - 1 > pos0 || (window > 0 && key0 < pos0 + BQ - window);
-      int key_hi = qp - key0, key_lo = window > 0 ? qp + 1 - window - key0 : -1;  // columns key_lo .. key_hi count
+      int key_hi = qp - key0, key_lo = window > 0 ? qp + 1 - window - key0 : -1;  // columns key_lo .. key_hi count,
+      const int key_kept = OPTIONS ? options.keep - key0 : 0;                      // and those before key_kept
       // (the P tile of this step is free: the product that read it last, P_TILES steps ago, has been consumed)
       // One sweep over the scores gives the probabilities relative to the maximum the row has used so far, and the
       // tile's own maximum on the way. The used maximum need not be the true one: any constant cancels in the
@@ -240,12 +248,25 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
           tmem_wait_ld();
           if (c + 16 < BKV) tmem_load16_nowait(s_addr + (unsigned)(c + 16), v[cur ^ 1]);
           float p[16];
+          if (OPTIONS) {  // the capped scores, in units of log2 e
+            float largest[2] = {0.f, 0.f};
+#pragma unroll
+            for (int i = 0; i < 16; ++i) largest[i & 1] = fmaxf(largest[i & 1], fabsf(__uint_as_float(v[cur][i])));
+            if (score.in == 0.f || __all_sync(0xffffffffu, fmaxf(largest[0], largest[1]) <= score.small_up_to)) {
+#pragma unroll
+              for (int i = 0; i < 16; ++i) v[cur][i] = __float_as_uint(score.small(__uint_as_float(v[cur][i])));
+            } else {
+#pragma unroll
+              for (int i = 0; i < 16; ++i) v[cur][i] = __float_as_uint(score.any(__uint_as_float(v[cur][i])));
+            }
+          }
           if (edge) {  // (two copies of the loop: the compares cost as much as the rest of an element)
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
-              float x = (c + i > key_hi || c + i < key_lo) ? -INFINITY : __uint_as_float(v[cur][i]);
+              float x = (c + i > key_hi || (c + i < key_lo && (!OPTIONS || c + i >= key_kept)))
+                            ? -INFINITY : __uint_as_float(v[cur][i]);
               mx[i & 3] = fmaxf(mx[i & 3], x);
-              p[i] = fast_exp2(fmaf(x, scale_log2, -m_use));
+              p[i] = fast_exp2(fmaf(x, unit, -m_use));
               sum[i & 3] += p[i];
             }
           } else {
@@ -253,7 +274,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
             for (int i = 0; i < 16; ++i) {
               float x = __uint_as_float(v[cur][i]);
               mx[i & 3] = fmaxf(mx[i & 3], x);
-              p[i] = fast_exp2(fmaf(x, scale_log2, -m_use));
+              p[i] = fast_exp2(fmaf(x, unit, -m_use));
               sum[i & 3] += p[i];
             }
           }
@@ -266,7 +287,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
             *reinterpret_cast<uint4*>(p_row + ((((c >> 3) + half) ^ (r & 7)) << 4)) = packed;
           }
         }
-        tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2;  // in the scaled log2 domain
+        tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * unit;  // in the scaled log2 domain
         row_sum = (sum[0] + sum[1]) + (sum[2] + sum[3]);
       };
       float tile_max, row_sum, corr = 1.f;
@@ -295,7 +316,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     if (ok && taken >= 1) ok = consume(wg + (taken - 1) * GROUPS, corr_saved);
     if (GROUPS == 1) {
       if (ok && r < rows) {
-        float inv = 1.0f / l_run;
+        float inv = OPTIONS ? sink_factor(m_run, l_run, options.sinks, h) : 1.0f / l_run;
         bf16* dst = out + ((size_t)(tok0 + r) * heads + h) * HD;
 #pragma unroll
         for (int c = 0; c < HD / 8; ++c) {
@@ -323,7 +344,8 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
         float m = fmaxf(m_run, m_other);
         float m_use = m == -INFINITY ? 0.f : m;
         float mine = fast_exp2(m_run - m_use), theirs = fast_exp2(m_other - m_use);
-        float inv = 1.0f / (l_run * mine + l_other * theirs);
+        float l = l_run * mine + l_other * theirs;
+        float inv = OPTIONS ? sink_factor(m_use, l, options.sinks, h) : 1.0f / l;
         mine *= inv;
         theirs *= inv;
         bf16* dst = out + ((size_t)(tok0 + r) * heads + h) * HD;
@@ -347,35 +369,29 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
   if (warp == SOFT_WARPS + 1) tmem_dealloc(tmem_base, TMEM_COLS);
 }
 
-template <int HD>
+template <int HD, bool OPTIONS>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, void* out, const KvLayout& cache, const int* tile_seq,
            const int* tile_first, const int* cu_seqlens, const int* start, const int* slots, int tiles, int heads,
-           float scale, int window, int* status, cudaStream_t stream) {
+           float scale, int window, int* status, const ScoreOptions& options, cudaStream_t stream) {
   typedef Shape<HD> S;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(prefill_tcgen05_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(prefill_tcgen05_kernel<HD, OPTIONS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)S::SMEM) != cudaSuccess)
       return DLLM_LAUNCH_FAILED;
     configured = true;
   }
-  return dllm_launch_pdl(prefill_tcgen05_kernel<HD>, dim3(tiles, heads), dim3(S::THREADS), S::SMEM, stream, map_q,
+  return dllm_launch_pdl(prefill_tcgen05_kernel<HD, OPTIONS>, dim3(tiles, heads), dim3(S::THREADS), S::SMEM, stream, map_q,
                          map_kv, (bf16*)out, cache, tile_seq, tile_first, cu_seqlens, start, slots, heads,
-                         scale * 1.4426950408889634f, window, status);
+                         scale * SCORE_LOG2E, window, status, options);
 }
-}  // namespace
 
-// out, q: [tokens, heads * head_dim] bfloat16. tile_seq / tile_first: for each tile of up to 64 new tokens, its
-// sequence and the index of its first token among the sequence's new tokens (the kernel pairs them into tiles of
-// 128). The keys and values of the new tokens are already in the cache, which holds `cache_pages` pages of 64
-// positions. head_dim must be 64 or 128. `status` is a word the device can write; the kernel sets it non-zero if a
-// bounded wait ran out.
-DLLM_EXPORT int dllm_attention_prefill_tcgen05(void* out, const void* q, int tokens, void* cache_base,
-                                               long long cache_pages, const int* page_table, int max_pages,
-                                               int page_size, int heads, int kv_heads, int head_dim,
-                                               const int* tile_seq, const int* tile_first, const int* cu_seqlens,
-                                               const int* start, const int* slots, int tiles, float scale, int window,
-                                               int* status, cudaStream_t stream) {
+// Checks, tensor maps and launch, with or without options.
+template <bool OPTIONS>
+int run(void* out, const void* q, int tokens, void* cache_base, long long cache_pages, const int* page_table,
+        int max_pages, int page_size, int heads, int kv_heads, int head_dim, const int* tile_seq, const int* tile_first,
+        const int* cu_seqlens, const int* start, const int* slots, int tiles, float scale, int window, int* status,
+        const ScoreOptions& options, cudaStream_t stream) {
   if (tiles <= 0 || tokens <= 0) return DLLM_OK;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || status == nullptr) return DLLM_BAD_ARGUMENT;
   if ((head_dim != 64 && head_dim != 128) || page_size != BKV || heads > 65535 || ((uintptr_t)q & 15) ||
@@ -388,8 +404,27 @@ DLLM_EXPORT int dllm_attention_prefill_tcgen05(void* out, const void* q, int tok
     return DLLM_LAUNCH_FAILED;
   KvLayout cache{cache_base, page_table, max_pages, page_size, kv_heads, head_dim};
   if (head_dim == 64)
-    return launch<64>(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale,
-                      window, status, stream);
-  return launch<128>(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale,
-                     window, status, stream);
+    return launch<64, OPTIONS>(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale,
+                      window, status, options, stream);
+  return launch<128, OPTIONS>(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale,
+                     window, status, options, stream);
 }
+}  // namespace
+
+#ifndef DLLM_PREFILL_TCGEN05_OPTIONS  // (a file that includes this one for the instantiations with options has its own)
+
+// out, q: [tokens, heads * head_dim] bfloat16. tile_seq / tile_first: for each tile of up to 64 new tokens, its
+// sequence and the index of its first token among the sequence's new tokens (the kernel pairs them into tiles of
+// 128). The keys and values of the new tokens are already in the cache, which holds `cache_pages` pages of 64
+// positions. head_dim must be 64 or 128. `status` is a word the device can write; the kernel sets it non-zero if a
+// bounded wait ran out.
+DLLM_EXPORT int dllm_attention_prefill_tcgen05(void* out, const void* q, int tokens, void* cache_base,
+                                               long long cache_pages, const int* page_table, int max_pages,
+                                               int page_size, int heads, int kv_heads, int head_dim,
+                                               const int* tile_seq, const int* tile_first, const int* cu_seqlens,
+                                               const int* start, const int* slots, int tiles, float scale, int window,
+                                               int* status, cudaStream_t stream) {
+  return run<false>(out, q, tokens, cache_base, cache_pages, page_table, max_pages, page_size, heads, kv_heads, head_dim,
+                    tile_seq, tile_first, cu_seqlens, start, slots, tiles, scale, window, status, ScoreOptions{}, stream);
+}
+#endif

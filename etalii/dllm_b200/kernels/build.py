@@ -46,6 +46,9 @@ SOURCES = {
     "moe": "moe.cu",
     "moe_grouped": "moe_grouped.cu",
     "sink_attention": "sink_attention.cu",
+    "sink_attention_prefill": "sink_attention_prefill.cu",
+    "sink_attention_decode": "sink_attention_decode.cu",
+    "sink_attention_tcgen05": "sink_attention_tcgen05.cu",
     "stream_update": "stream_update.cu",
     "sampling": "sampling.cu",
     "step_launcher": "step_launcher.cu",

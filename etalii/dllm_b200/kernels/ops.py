@@ -61,6 +61,15 @@ _prototypes = {
     ("sink_attention", "dllm_sink_attention"): [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                 c_float, c_float, c_int, c_int, c_int, c_int, c_void_p],
+    ("sink_attention_prefill", "dllm_sink_attention_prefill"): [
+        c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+        c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_void_p],
+    ("sink_attention_decode", "dllm_sink_attention_decode"): [
+        c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+        c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+    ("sink_attention_tcgen05", "dllm_sink_attention_tcgen05"): [
+        c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
+        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p],
     ("elementwise", "dllm_norm_sum_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
                                                 c_float, c_void_p],
     ("elementwise", "dllm_norm_add_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
@@ -542,6 +551,68 @@ def sink_attention(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale:
         batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.slots.data_ptr(), tokens, float(scale),
         float(softcap or 0.0), int(window or 0), int(keep or 0), 1 if split else 0, _code(cache.dtype), _stream()),
         "sink_attention", lambda: f"dim={dim}, value_dim={vdim} (at most 256)")
+
+
+def sink_attention_tiles(dtype, dim: int, vdim: int, page_size: int = 64) -> bool:
+    """Whether the tensor-core kernels for tiles of queries and for single tokens run these sizes."""
+    return dtype == torch.bfloat16 and page_size == 64 and dim % 8 == 0 and vdim % 8 == 0 and max(dim, vdim) <= 128
+
+
+def sink_attention_prefill(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
+                           sinks: torch.Tensor | None, window: int, keep: int, batch) -> None:
+    """`sink_attention` for portions of prompts (bfloat16, mma.sync, tiles of 64 queries; sizes:
+    `sink_attention_tiles`)."""
+    _cuda(out, q, sinks)
+    dim, vdim = cache.head_dim, cache.value_dim
+    assert sink_attention_tiles(cache.dtype, dim, vdim, cache.page_size) and not cache.keys_only
+    assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    assert q.shape[1] == heads * dim and out.shape[1] == heads * vdim
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
+    _check(_fn("sink_attention_prefill", "dllm_sink_attention_prefill")(
+        out.data_ptr(), out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
+        cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(),
+        batch.cu_seqlens.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), batch.n_tiles, float(scale),
+        float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0),
+        _stream()), "sink_attention_prefill")
+
+
+def sink_attention_tcgen05_supported(cache) -> bool:
+    return attention_prefill_tcgen05_supported(cache) and cache.value_dim == cache.head_dim
+
+
+def sink_attention_tcgen05(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
+                           sinks: torch.Tensor | None, window: int, keep: int, batch) -> None:
+    """`sink_attention` for portions of prompts on the 5th-generation tensor cores (bfloat16, keys and values of 64 or
+    128 values)."""
+    _cuda(out, q, sinks)
+    assert sink_attention_tcgen05_supported(cache) and not cache.keys_only
+    assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    assert q.shape[1] == heads * cache.head_dim and out.shape[1] == q.shape[1]
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
+    _check(_fn("sink_attention_tcgen05", "dllm_sink_attention_tcgen05")(
+        out.data_ptr(), q.data_ptr(), batch.n_tokens, cache.base_ptr, cache.storage.shape[0],
+        cache.page_table.data_ptr(), cache.max_pages, cache.page_size, heads, cache.kv_heads, cache.head_dim,
+        batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(), batch.cu_seqlens.data_ptr(), batch.start.data_ptr(),
+        batch.slots.data_ptr(), batch.n_tiles, float(scale), float(softcap or 0.0),
+        sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0), _status_word().data_ptr(),
+        _stream()), "sink_attention_tcgen05")
+
+
+def sink_attention_decode(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
+                          sinks: torch.Tensor | None, window: int, keep: int, batch, shape: int = -1) -> None:
+    """`sink_attention` for a step of single tokens (bfloat16; sizes: `sink_attention_tiles`): the keys of a (sequence,
+    kv head) dealt to the blocks of a cluster; `shape` as for `attention_decode_cluster`."""
+    _cuda(out, q, sinks)
+    dim, vdim = cache.head_dim, cache.value_dim
+    assert sink_attention_tiles(cache.dtype, dim, vdim, cache.page_size) and not cache.keys_only
+    assert batch.n_tokens == batch.n_seqs and q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    assert q.shape[1] == heads * dim and out.shape[1] == heads * vdim
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
+    _check(_fn("sink_attention_decode", "dllm_sink_attention_decode")(
+        out.data_ptr(), out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
+        cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tok_pos.data_ptr(), batch.slots.data_ptr(),
+        batch.n_seqs, float(scale), float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None,
+        int(window or 0), int(keep or 0), int(shape), _stream()), "sink_attention_decode")
 
 
 def glu_clamped_fuses(rows: int, outputs: int, inner: int) -> bool:

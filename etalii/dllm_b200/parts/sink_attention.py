@@ -20,6 +20,7 @@ import torch
 
 from ..cache.paged import CacheNeed
 from ..kernels import ops
+from .attention import TCGEN05_ATTENTION_FROM
 from .norm import row_rule
 from .registry import register_part
 from .spec import ParamSpec
@@ -94,15 +95,30 @@ class SinkAttention:
         ops.sigmoid_prepare(rows, 0, k_at, k_at + groups * dim, q, cache, heads, self.bias_rows, None, 0.0, batch,
                             write_cache and not self.shares_keys)
         attended = rt.ws.buffer("attended", (n, self.padded), rt.dtype)
-        ops.sink_attention(attended, q, cache, heads, self.scale, self.softcap, self.sinks, self.window,
-                           self.keep_first, batch)
+        attend = ops.sink_attention
+        if ops.sink_attention_tiles(rt.dtype, dim, vdim, cache.page_size):
+            reach = batch.max_context
+            if self.window:
+                reach = min(reach, self.window + self.keep_first + 64)  # (keys a tile of queries walks)
+            if batch.is_decode:
+                attend = ops.sink_attention_decode
+            elif ops.sink_attention_tcgen05_supported(cache) and reach > TCGEN05_ATTENTION_FROM[dim]:
+                attend = ops.sink_attention_tcgen05
+            else:
+                attend = ops.sink_attention_prefill
+        attend(attended, q, cache, heads, self.scale, self.softcap, self.sinks, self.window, self.keep_first, batch)
         ops.gemm(residual, attended, self.w_o, epilogue)
 
     def kernel_libraries(self, rt) -> set[str]:
-        names = {"elementwise", "sigmoid_attention", "sink_attention"}
+        names = {"elementwise", "sigmoid_attention"}
         if rt.dtype != torch.bfloat16:
-            return names | {"gemm_simt"}
-        return names | {"gemv", "gemv_cluster", "gemm_tcgen05"}
+            return names | {"gemm_simt", "sink_attention"}
+        names |= {"gemv", "gemv_cluster", "gemm_tcgen05"}
+        if not ops.sink_attention_tiles(rt.dtype, self.dim, self.vdim):
+            return names | {"sink_attention"}
+        if self.dim == self.vdim and self.dim in TCGEN05_ATTENTION_FROM:
+            names.add("sink_attention_tcgen05")
+        return names | {"sink_attention_prefill", "sink_attention_decode"}
 
 
 register_part("mixer", "sink_attention", SinkAttention)

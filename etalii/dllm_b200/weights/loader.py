@@ -58,11 +58,13 @@ def _fits(shape, wanted, free: dict[str, int]) -> bool:
     """Whether a stored shape is the wanted one; `free` collects what the checkpoint decides for its free sizes."""
     if len(shape) != len(wanted):
         return False
+    found: dict[str, int] = {}
     for have, want in zip(shape, wanted):
         if isinstance(want, FreeSize):
-            want = free.setdefault(want.name, int(have))
+            want = found.setdefault(want.name, free.get(want.name, int(have)))
         if have != want or have <= 0:
             return False
+    free.update(found)
     return True
 
 
