@@ -169,16 +169,19 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
       for (int j = 0; j < BN / 8; ++j)
 #pragma unroll
         for (int r = 0; r < 4; ++r) largest = fmaxf(largest, fabsf(s[j][r]));
-      if (score.in == 0.f || __all_sync(0xffffffffu, largest <= score.small_up_to)) {
+      if (__all_sync(0xffffffffu, largest <= score.small_up_to)) {
 #pragma unroll
         for (int j = 0; j < BN / 8; ++j)
 #pragma unroll
-          for (int r = 0; r < 4; ++r) s[j][r] = score.small(s[j][r]);
+          for (int r = 0; r < 4; r += 2) {
+            float2 y = score.small2(make_float2(s[j][r], s[j][r + 1]), make_float2(0.f, 0.f));
+            s[j][r] = y.x; s[j][r + 1] = y.y;
+          }
       } else {
 #pragma unroll
         for (int j = 0; j < BN / 8; ++j)
 #pragma unroll
-          for (int r = 0; r < 4; ++r) s[j][r] = score.any(s[j][r]);
+          for (int r = 0; r < 4; ++r) s[j][r] = score.large(s[j][r]);
       }
     }
     float tile_max[2] = {-INFINITY, -INFINITY};

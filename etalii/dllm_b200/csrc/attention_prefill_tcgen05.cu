@@ -189,7 +189,6 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     float m_run = -INFINITY, l_run = 0.f, corr_saved = 1.f;
     bool ok = true;
     const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
-    const float unit = OPTIONS ? 1.0f : scale_log2;  // what a score still has to be multiplied by in the sweep
     // fold step i's output into the running one: O = O * corr + P V
     auto consume = [&](int i, float corr) -> bool {
       const int ob = i & 1;
@@ -247,34 +246,39 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
           const int cur = (c >> 4) & 1;
           tmem_wait_ld();
           if (c + 16 < BKV) tmem_load16_nowait(s_addr + (unsigned)(c + 16), v[cur ^ 1]);
-          float p[16];
-          if (OPTIONS) {  // the capped scores, in units of log2 e
+          float p[16];  // first the scores as they enter the exponential
+          if (OPTIONS) {
             float largest[2] = {0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < 16; ++i) largest[i & 1] = fmaxf(largest[i & 1], fabsf(__uint_as_float(v[cur][i])));
-            if (score.in == 0.f || __all_sync(0xffffffffu, fmaxf(largest[0], largest[1]) <= score.small_up_to)) {
+            if (__all_sync(0xffffffffu, fmaxf(largest[0], largest[1]) <= score.small_up_to)) {
 #pragma unroll
-              for (int i = 0; i < 16; ++i) v[cur][i] = __float_as_uint(score.small(__uint_as_float(v[cur][i])));
+              for (int i = 0; i < 16; i += 2) {
+                float2 y = score.small2(make_float2(__uint_as_float(v[cur][i]), __uint_as_float(v[cur][i + 1])),
+                                        make_float2(-m_use, -m_use));
+                p[i] = y.x; p[i + 1] = y.y;
+              }
             } else {
 #pragma unroll
-              for (int i = 0; i < 16; ++i) v[cur][i] = __float_as_uint(score.any(__uint_as_float(v[cur][i])));
+              for (int i = 0; i < 16; ++i) p[i] = score.large(__uint_as_float(v[cur][i])) - m_use;
             }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) p[i] = fmaf(__uint_as_float(v[cur][i]), scale_log2, -m_use);
           }
           if (edge) {  // (two copies of the loop: the compares cost as much as the rest of an element)
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
-              float x = (c + i > key_hi || (c + i < key_lo && (!OPTIONS || c + i >= key_kept)))
-                            ? -INFINITY : __uint_as_float(v[cur][i]);
-              mx[i & 3] = fmaxf(mx[i & 3], x);
-              p[i] = fast_exp2(fmaf(x, unit, -m_use));
+              bool unseen = c + i > key_hi || (c + i < key_lo && (!OPTIONS || c + i >= key_kept));
+              mx[i & 3] = fmaxf(mx[i & 3], unseen ? -INFINITY : __uint_as_float(v[cur][i]));
+              p[i] = fast_exp2(unseen ? -INFINITY : p[i]);
               sum[i & 3] += p[i];
             }
           } else {
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
-              float x = __uint_as_float(v[cur][i]);
-              mx[i & 3] = fmaxf(mx[i & 3], x);
-              p[i] = fast_exp2(fmaf(x, unit, -m_use));
+              mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(v[cur][i]));
+              p[i] = fast_exp2(p[i]);
               sum[i & 3] += p[i];
             }
           }
@@ -287,7 +291,10 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
             *reinterpret_cast<uint4*>(p_row + ((((c >> 3) + half) ^ (r & 7)) << 4)) = packed;
           }
         }
-        tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * unit;  // in the scaled log2 domain
+        tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));  // of the raw scores; now in the scaled log2 domain
+        // (the cap keeps the scores' order, so the largest one's capped value is the largest)
+        if (OPTIONS) tile_max = tile_max == -INFINITY ? -INFINITY : score.any(tile_max);
+        else tile_max *= scale_log2;
         row_sum = (sum[0] + sum[1]) + (sum[2] + sum[3]);
       };
       float tile_max, row_sum, corr = 1.f;

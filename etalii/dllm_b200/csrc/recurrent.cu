@@ -10,8 +10,9 @@
 // One kernel serves prompts and single tokens: a block owns 16 columns of one head's S for one sequence and walks
 // that sequence's new tokens in order, from the state the cache holds to the state it leaves there. A column's
 // recurrence does not involve the other columns, so columns are the parallel dimension besides heads and sequences.
-// Inside a warp a lane holds `RPL` consecutive rows of one column (8 or 16 lanes a column): the sums over
-// rows (S^T q, S^T k) are RPL multiply-adds a lane and three or four shuffles. The tokens' q, k and v come through two
+// Inside a warp a lane holds `RPL` rows of one column in pieces of four (8 or 16 lanes a column; piece i of lane r starts
+// at row 4 (i lanes + r), so the lanes of a column read one run of shared memory): the sums over rows (S^T q, S^T k) are
+// RPL multiply-adds a lane and three or four shuffles. The tokens' q, k and v come through two
 // shared-memory stages filled by cp.async (16-byte pieces where the rows allow it), so global latency is paid once per
 // 16 tokens and hidden behind the arithmetic of the stage before. Everything is float32: inputs, state, sums.
 //
@@ -101,13 +102,13 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   pdl_wait();
   const int first = a.cu_seqlens[seq], count = a.cu_seqlens[seq + 1] - first;
   const int slot = a.slots[seq];
-  float* my_state = a.state + (((size_t)slot * a.heads + head) * state_cols + col) * (size_t)a.dim + rg * RPL;
+  float* my_state = a.state + (((size_t)slot * a.heads + head) * state_cols + col) * (size_t)a.dim + rg * 4;
 
   float S[RPL];  // (dim is a multiple of 4 and so is a lane's first row: a piece of 4 rows is inside the head or not)
 #pragma unroll
   for (int j = 0; j < RPL; j += 4) {
-    float4 s4 = (col < state_cols && rg * RPL + j < a.dim) ? *reinterpret_cast<const float4*>(my_state + j)
-                                                         : make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 s4 = (col < state_cols && j * LPC + rg * 4 < a.dim) ? *reinterpret_cast<const float4*>(my_state + j * LPC)
+                                                             : make_float4(0.f, 0.f, 0.f, 0.f);
     S[j] = s4.x; S[j + 1] = s4.y; S[j + 2] = s4.z; S[j + 3] = s4.w;
   }
 
@@ -184,8 +185,8 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
     float2 p = make_float2(0.f, 0.f);
 #pragma unroll
     for (int j = 0; j < RPL; j += 4) {
-      float4 k4 = *reinterpret_cast<const float4*>(row + rg * RPL + j);
-      float4 q4 = *reinterpret_cast<const float4*>(row + DIMP + rg * RPL + j);
+      float4 k4 = *reinterpret_cast<const float4*>(row + j * LPC + rg * 4);
+      float4 q4 = *reinterpret_cast<const float4*>(row + DIMP + j * LPC + rg * 4);
       float2 s01 = __ffma2_rn(dd, make_float2(S[j], S[j + 1]), __fmul2_rn(make_float2(k4.x, k4.y), vv));
       float2 s23 = __ffma2_rn(dd, make_float2(S[j + 2], S[j + 3]), __fmul2_rn(make_float2(k4.z, k4.w), vv));
       S[j] = s01.x; S[j + 1] = s01.y; S[j + 2] = s23.x; S[j + 3] = s23.y;
@@ -211,16 +212,12 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
     __syncthreads();
     const float* base = stage + (size_t)buffer * TOKENS * PER_TOKEN;
     const int here = min(TOKENS, count - chunk * TOKENS);
-    float* out = a.out + (size_t)(first + chunk * TOKENS) * out_width + head * a.vdim + col;
-    const bool writes = rg == 0 && col < a.vdim;
-    int t = 0;
+    // Every lane leaves its part of a token's read-out in shared memory; after the chunk the block adds the parts up, a
+    // thread per token and column, and writes whole pieces of rows.
+    float* parts = stage + (size_t)STAGES * TOKENS * PER_TOKEN;  // [TOKENS][16 columns][LPC + 4]
+    constexpr int PADL = LPC + 4;
     if (MODE == 0 || MODE == 2) {
-      // The decayed sum's read-out does not feed the state, so its sum over the rows need not be finished token by
-      // token: every lane leaves its part in shared memory and goes on to the next token (nothing but the state's
-      // own multiply-add links two tokens); after the chunk the block adds the parts up, a thread per token and
-      // column, and writes whole pieces of rows.
-      float* parts = stage + (size_t)STAGES * TOKENS * PER_TOKEN;  // [TOKENS][16 columns][LPC + 4]
-      constexpr int PADL = LPC + 4;
+      // The decayed sum's read-out does not feed the state: nothing but the state's own multiply-add links two tokens.
       // a group of tokens at a time: all their rows are asked of shared memory first (the loads do not depend on the
       // state), then the state walks through them
       constexpr int GROUP = RPL <= 8 ? 4 : 2;
@@ -239,8 +236,8 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           }
 #pragma unroll
           for (int j = 0; j < RPL; j += 4) {
-            kq[w][j / 2] = *reinterpret_cast<const float4*>(row + rg * RPL + j);
-            kq[w][j / 2 + 1] = *reinterpret_cast<const float4*>(row + DIMP + rg * RPL + j);
+            kq[w][j / 2] = *reinterpret_cast<const float4*>(row + j * LPC + rg * 4);
+            kq[w][j / 2 + 1] = *reinterpret_cast<const float4*>(row + DIMP + j * LPC + rg * 4);
           }
         }
 #pragma unroll
@@ -261,80 +258,93 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
       }
       for (; u < here; ++u)
         parts[(u * SCAN_COLS + warp * CPW + cc) * PADL + rg] = decayed(base + u * PER_TOKEN);
-      __syncthreads();
-      for (int i = tid; i < here * SCAN_COLS; i += SCAN_THREADS) {
-        int u = i / SCAN_COLS, c = i % SCAN_COLS;
-        const float4* mine = reinterpret_cast<const float4*>(parts + i * PADL);
-        float sum = 0.f;
+    } else {
+      // The delta rule: what the state answers to k feeds the write, so the sum S^T k is finished token by token (the
+      // shuffles are most of the time from one token to the next); S^T q waits for the end of the chunk. A token's rows
+      // are asked of shared memory while the token before it is worked on.
+      constexpr bool AHEAD = RPL <= 16;  // (with 32 rows a lane there are no registers for a second token)
+      constexpr int V4 = RPL / 4;
+      float4 k4[V4], q4[V4], g4[MODE == 3 ? V4 : 1];
+      float v, beta, kq, g = 1.f;
+      auto fetch = [&](int t) {
+        const float* row = base + t * PER_TOKEN;
 #pragma unroll
-        for (int j = 0; j < LPC / 4; ++j) {
-          float4 p4 = mine[j];
-          sum += (p4.x + p4.y) + (p4.z + p4.w);
+        for (int j = 0; j < V4; ++j) {
+          if (MODE == 3) g4[j] = *reinterpret_cast<const float4*>(row + 2 * DIMP + 4 * (j * LPC + rg));
+          k4[j] = *reinterpret_cast<const float4*>(row + 4 * (j * LPC + rg));
+          q4[j] = *reinterpret_cast<const float4*>(row + DIMP + 4 * (j * LPC + rg));
         }
-        if (col0 + c < a.vdim)
-          a.out[(size_t)(first + chunk * TOKENS + u) * out_width + head * a.vdim + col0 + c] = sum * a.out_scale;
-        else if (MODE == 2 && col0 + c == a.vdim)
-          a.nq[(size_t)(first + chunk * TOKENS + u) * a.heads + head] = sum * a.out_scale;
-      }
-      t = here;
-    }
-    for (; t < here; ++t) {  // (the delta rule: its sums over the rows feed the state, token by token)
-      const float* row = base + t * PER_TOKEN;
-      float o;
-      {
-        float v = row[V_AT + warp * CPW + cc];
-        float g = MODE == 3 ? 1.f : row[V_AT + SCAN_COLS], beta = row[V_AT + SCAN_COLS + 1], kq = row[V_AT + SCAN_COLS + 2];
+        v = row[V_AT + warp * CPW + cc];
+        if (MODE == 1) g = row[V_AT + SCAN_COLS];
+        beta = row[V_AT + SCAN_COLS + 1];
+        kq = row[V_AT + SCAN_COLS + 2];
+      };
+      fetch(0);
+#pragma unroll 2
+      for (int t = 0; t < here; ++t) {
+        if (!AHEAD && t > 0) fetch(t);
+        float2 sk[2] = {}, sq[2] = {};  // S^T k and S^T q before this token's write, in two chains each
         float2 kk[RPL / 2];
-        float2 sk2 = make_float2(0.f, 0.f), sq2 = make_float2(0.f, 0.f);  // S^T k and S^T q before this token
 #pragma unroll
-        for (int j = 0; j < RPL; j += 4) {
-          float4 k4 = *reinterpret_cast<const float4*>(row + rg * RPL + j);
-          float4 q4 = *reinterpret_cast<const float4*>(row + DIMP + rg * RPL + j);
-          kk[j / 2] = make_float2(k4.x, k4.y);
-          kk[j / 2 + 1] = make_float2(k4.z, k4.w);
-          float2 s01 = make_float2(S[j], S[j + 1]), s23 = make_float2(S[j + 2], S[j + 3]);
+        for (int j = 0; j < V4; ++j) {
+          float2 s01 = make_float2(S[4 * j], S[4 * j + 1]), s23 = make_float2(S[4 * j + 2], S[4 * j + 3]);
           if (MODE == 3) {  // the rows shrink first: what follows reads and moves on the shrunk state
-            float4 g4 = *reinterpret_cast<const float4*>(row + 2 * DIMP + rg * RPL + j);
-            s01 = __fmul2_rn(s01, make_float2(g4.x, g4.y));
-            s23 = __fmul2_rn(s23, make_float2(g4.z, g4.w));
-            S[j] = s01.x; S[j + 1] = s01.y; S[j + 2] = s23.x; S[j + 3] = s23.y;
+            s01 = __fmul2_rn(s01, make_float2(g4[j].x, g4[j].y));
+            s23 = __fmul2_rn(s23, make_float2(g4[j].z, g4[j].w));
+            S[4 * j] = s01.x; S[4 * j + 1] = s01.y; S[4 * j + 2] = s23.x; S[4 * j + 3] = s23.y;
           }
-          sk2 = __ffma2_rn(s01, kk[j / 2], sk2);
-          sq2 = __ffma2_rn(s01, make_float2(q4.x, q4.y), sq2);
-          sk2 = __ffma2_rn(s23, kk[j / 2 + 1], sk2);
-          sq2 = __ffma2_rn(s23, make_float2(q4.z, q4.w), sq2);
+          kk[2 * j] = make_float2(k4[j].x, k4[j].y);
+          kk[2 * j + 1] = make_float2(k4[j].z, k4[j].w);
+          sk[0] = __ffma2_rn(s01, kk[2 * j], sk[0]);
+          sk[1] = __ffma2_rn(s23, kk[2 * j + 1], sk[1]);
+          sq[0] = __ffma2_rn(s01, make_float2(q4[j].x, q4[j].y), sq[0]);
+          sq[1] = __ffma2_rn(s23, make_float2(q4[j].z, q4[j].w), sq[1]);
         }
-        float sk = sk2.x + sk2.y, sq = sq2.x + sq2.y;
+        const float v_now = v, beta_now = beta, kq_now = kq, g_now = g;
+        if (AHEAD) fetch(min(t + 1, here - 1));
+        float answer = (sk[0].x + sk[0].y) + (sk[1].x + sk[1].y);
 #pragma unroll
-        for (int o2 = CPW; o2 <= 16; o2 <<= 1) {
-          sk += __shfl_xor_sync(0xffffffffu, sk, o2);
-          sq += __shfl_xor_sync(0xffffffffu, sq, o2);
-        }
-        // (g S + k u^T)^T q = g S^T q + u (k . q): the read-out of the state after the write, without a second sum
-        float u = beta * (v - g * sk);
-        o = fmaf(g, sq, u * kq);
-        const float2 uu = make_float2(u, u), gg = make_float2(g, g);
+        for (int o = CPW; o <= 16; o <<= 1) answer += __shfl_xor_sync(0xffffffffu, answer, o);
+        const float u = beta_now * (v_now - g_now * answer);
+        const float2 uu = make_float2(u, u), gg = make_float2(g_now, g_now);
 #pragma unroll
         for (int j = 0; j < RPL; j += 2) {
           float2 now = make_float2(S[j], S[j + 1]);
           float2 next = __ffma2_rn(kk[j / 2], uu, MODE == 3 ? now : __fmul2_rn(gg, now));
           S[j] = next.x; S[j + 1] = next.y;
         }
+        // (g S + k u^T)^T q = g S^T q + u (k . q): the read-out of the state after the write, without a second sum
+        float read = g_now * ((sq[0].x + sq[0].y) + (sq[1].x + sq[1].y));
+        parts[(t * SCAN_COLS + warp * CPW + cc) * PADL + rg] = rg == 0 ? fmaf(u, kq_now, read) : read;
       }
-      if (writes) out[(size_t)t * out_width] = o;
+    }
+    __syncthreads();
+    for (int i = tid; i < here * SCAN_COLS; i += SCAN_THREADS) {
+      int u = i / SCAN_COLS, c = i % SCAN_COLS;
+      const float4* mine = reinterpret_cast<const float4*>(parts + i * PADL);
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < LPC / 4; ++j) {
+        float4 p4 = mine[j];
+        sum += (p4.x + p4.y) + (p4.z + p4.w);
+      }
+      if (col0 + c < a.vdim)
+        a.out[(size_t)(first + chunk * TOKENS + u) * out_width + head * a.vdim + col0 + c] = sum * a.out_scale;
+      else if (MODE == 2 && col0 + c == a.vdim)
+        a.nq[(size_t)(first + chunk * TOKENS + u) * a.heads + head] = sum * a.out_scale;
     }
     __syncthreads();  // the stage is filled again in the next round
   }
 #pragma unroll
   for (int j = 0; j < RPL; j += 4)
-    if (col < state_cols && rg * RPL + j < a.dim)
-      *reinterpret_cast<float4*>(my_state + j) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
+    if (col < state_cols && j * LPC + rg * 4 < a.dim)
+      *reinterpret_cast<float4*>(my_state + j * LPC) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
 }
 
 template <int RPL, int LPC, int MODE, int TOKENS, int STAGES>
 static int launch_scan_case(const ScanArgs& a, dim3 grid, cudaStream_t stream) {
   size_t bytes = (size_t)STAGES * TOKENS * ((MODE == 3 ? 3 : 2) * RPL * LPC + SCAN_COLS + 4) * sizeof(float);
-  if (MODE == 0 || MODE == 2) bytes += (size_t)TOKENS * SCAN_COLS * (LPC + 4) * sizeof(float);  // the parts of the read-out
+  bytes += (size_t)TOKENS * SCAN_COLS * (LPC + 4) * sizeof(float);  // the parts of the read-out
   static bool allowed = false;  // (more than 48 KB of dynamic shared memory has to be asked for once)
   if (bytes > 48 * 1024 && !allowed) {
     if (cudaFuncSetAttribute(scan_kernel<RPL, LPC, MODE, TOKENS, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -355,10 +365,12 @@ static int launch_scan(const ScanArgs& a, int sequences, int longest, cudaStream
   long long blocks = (long long)grid.x * grid.y * grid.z;
   int dimp = a.dim <= 32 ? 32 : (a.dim <= 64 ? 64 : (a.dim <= 128 ? 128 : 256));
   int lanes = (blocks * 4 >= 148 * 16 || dimp / 16 < 4) ? 8 : 16;
-  bool deep = longest > 32;  // four stages for prompts, two for steps of single tokens and short portions
+  // The delta rule links two tokens by a sum over a column's lanes: the fewer lanes, the fewer shuffles in that chain.
+  if ((MODE == 1 || MODE == 3) && longest > 8 && dimp <= 128) lanes = 8;
+  bool deep = longest > 32;  // several stages for prompts, two for steps of single tokens and short portions
 #define SCAN_CASE(RPL, LPC, TOKENS)                                                                 \
   if (dimp == RPL * LPC && lanes == LPC)                                                            \
-    return deep ? launch_scan_case<RPL, LPC, MODE, TOKENS, 4>(a, grid, stream)                      \
+    return deep ? launch_scan_case<RPL, LPC, MODE, TOKENS, MODE == 3 ? 3 : 4>(a, grid, stream)      \
                 : launch_scan_case<RPL, LPC, MODE, TOKENS, 2>(a, grid, stream);
   SCAN_CASE(4, 8, 16)
   SCAN_CASE(8, 8, 16) SCAN_CASE(4, 16, 16)

@@ -101,6 +101,8 @@ __global__ void __launch_bounds__(256) sigmoid_prepare_kernel(
   pdl_wait();
   const int t = blockIdx.x, dim = cache.key_dim, vdim = cache.value_dim;
   const float* row = rows + (size_t)t * stride;
+  // (without norms over the whole row, blocks along y share a token's row)
+  const int begin = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
   const int q_size = heads * dim, k_size = cache.kv_heads * dim, v_size = cache.kv_heads * vdim;
   {
     float inv = 1.0f;
@@ -112,7 +114,7 @@ __global__ void __launch_bounds__(256) sigmoid_prepare_kernel(
       }
       inv = 1.0f / sqrtf(block_total(s, scratch) / (float)q_size + eps);
     }
-    for (int i = threadIdx.x; i < q_size; i += blockDim.x) {
+    for (int i = begin; i < q_size; i += step) {
       float x = row[q_at + i] + (q_bias != nullptr ? q_bias[i] : 0.f);
       q_out[(size_t)t * q_size + i] = from_float<T>(q_weight != nullptr ? x * inv * q_weight[i] : x);
     }
@@ -130,12 +132,12 @@ __global__ void __launch_bounds__(256) sigmoid_prepare_kernel(
     }
     inv = 1.0f / sqrtf(block_total(s, scratch) / (float)k_size + eps);
   }
-  for (int i = threadIdx.x; i < k_size; i += blockDim.x) {
+  for (int i = begin; i < k_size; i += step) {
     float x = row[k_at + i] + (k_bias != nullptr ? k_bias[i] : 0.f);
     int g = i / dim, d = i - g * dim;
     ((T*)cache.base)[key_at(cache, page, g, at) + d] = from_float<T>(k_weight != nullptr ? x * inv * k_weight[i] : x);
   }
-  for (int i = threadIdx.x; i < v_size; i += blockDim.x) {
+  for (int i = begin; i < v_size; i += step) {
     float x = row[v_at + i] + (v_bias != nullptr ? v_bias[i] : 0.f);
     int g = i / vdim, d = i - g * vdim;
     ((T*)cache.base)[value_at(cache, page, g, at) + d] = from_float<T>(x);
@@ -298,12 +300,18 @@ DLLM_EXPORT int dllm_sigmoid_prepare(const float* rows, int stride, int q_at, in
     return DLLM_UNSUPPORTED_SIZE;
   if (!rows || !q_out || !cache_base || !page_table || !tok_seq || !tok_pos || !slots) return DLLM_BAD_ARGUMENT;
   WideKv cache{cache_base, page_table, max_pages, page_size, kv_heads, dim, vdim};
+  int across = 1;
+  if (q_weight == nullptr && k_weight == nullptr) {  // few tokens: as many blocks a token as give every thread four values
+    int most = (heads * dim + 2 * kv_heads * (dim > vdim ? dim : vdim) + 1023) / 1024;
+    while (across < most && (long long)tokens * across < 296) ++across;
+  }
+  dim3 grid(tokens, across);
   if (dtype == DLLM_F32)
-    return dllm_launch_pdl(sigmoid_prepare_kernel<float>, dim3(tokens), dim3(256), 0, stream, rows, stride, q_at, k_at,
+    return dllm_launch_pdl(sigmoid_prepare_kernel<float>, grid, dim3(256), 0, stream, rows, stride, q_at, k_at,
                            v_at, heads, q_bias, k_bias, v_bias, q_weight, k_weight, eps, (float*)q_out, cache, tok_seq,
                            tok_pos, slots, write_cache);
   if (dtype == DLLM_BF16)
-    return dllm_launch_pdl(sigmoid_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, rows, stride,
+    return dllm_launch_pdl(sigmoid_prepare_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, rows, stride,
                            q_at, k_at, v_at, heads, q_bias, k_bias, v_bias, q_weight, k_weight, eps,
                            (__nv_bfloat16*)q_out, cache, tok_seq, tok_pos, slots, write_cache);
   return DLLM_BAD_ARGUMENT;
