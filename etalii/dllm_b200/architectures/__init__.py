@@ -1,1 +1,1 @@
-from . import gaperax, llama, revupel, satavik, tezinex, tisalorn  # noqa: F401  (register the architectures)
+from . import gaperax, llama, revupel, satavik, tezinex, tisalorn, zivazen  # noqa: F401  (register the architectures)

@@ -9,7 +9,7 @@
 //
 // Instantiated with OPTIONS (score_options.cuh; sink_attention_decode.cu does) the scores may be capped, the denominator
 // holds a sink, the window keeps a sequence's first positions (the tiles are then those of kept positions followed by
-// those of the window) and the values may have another size than the keys (HD covers both; multiples of 8).
+// those of the window), a token may see its own chunk of positions only, and the values may have another size than the keys (HD covers both; multiples of 8).
 #include "score_options.cuh"
 
 namespace {
@@ -80,10 +80,11 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
   };
   pdl_launch_dependents();
   int end = tok_pos[b] + 1;    // positions and slots are written only by the step's last kernel
-  int first = (window > 0 && end > window) ? end - window : 0;
+  const int chunk = OPTIONS ? options.chunk : 0;
+  int first = first_visible(end - 1, chunk, window);
   int base = (first / TILE_KEYS) * TILE_KEYS;
   // tile number `it` of the walk starts at key key_of(it)
-  const KeyWalk walk(end - 1, end - 1, window, OPTIONS ? options.keep : 0, TILE_KEYS);
+  const KeyWalk walk(end - 1, end - 1, window, OPTIONS ? options.keep : 0, TILE_KEYS, chunk);
   auto key_of = [&](int it) { return OPTIONS ? walk.tile(it) * TILE_KEYS : base + it * TILE_KEYS; };
   const int tiles = OPTIONS ? walk.count : (end - base + TILE_KEYS - 1) / TILE_KEYS;
   const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);

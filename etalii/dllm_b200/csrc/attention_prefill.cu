@@ -10,7 +10,8 @@
 // The page size must be 64.
 //
 // Instantiated with OPTIONS (score_options.cuh; sink_attention_prefill.cu does) the scores may be capped, the denominator
-// holds a sink, the window keeps a sequence's first positions and the values may have another size than the keys (HD
+// holds a sink, the window keeps a sequence's first positions, a token may see
+// its own chunk of positions only, and the values may have another size than the keys (HD
 // covers both; multiples of 8).
 #include "score_options.cuh"
 
@@ -83,7 +84,8 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
   }
   int last_pos = pos0 + rows - 1;                                   // last query's position
   // the key tiles the block's queries see between them, by their number in the walk
-  const KeyWalk walk(pos0, last_pos, window, OPTIONS ? options.keep : 0, BN);
+  const int chunk = OPTIONS ? options.chunk : 0;
+  const KeyWalk walk(pos0, last_pos, window, OPTIONS ? options.keep : 0, BN, chunk);
   const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
   // the pages of the key tiles this block will read, fetched once (not one dependent load per tile)
   __shared__ int page_s[MAX_TILES];
@@ -127,6 +129,9 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
   unsigned q_frag[HD / 16][4];
   int gq = lane >> 2, tq = lane & 3;
   int row_pos[2] = {pos0 + warp * 16 + gq, pos0 + warp * 16 + gq + 8};  // positions of this thread's two rows
+  // the first position each of them sees, and the largest such position of the warp's sixteen rows
+  const int row_first[2] = {first_visible(row_pos[0], chunk, window), first_visible(row_pos[1], chunk, window)};
+  const int warp_first = first_visible(pos0 + warp * 16 + 15, chunk, window);
 
   bool have_q = false;
   for (int it = group; it < walk.count; it += GROUPS) {
@@ -161,7 +166,7 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
     }
     // scale (log2 domain), masks, running maximum
     int key0 = walk.tile(it) * BN;
-    bool need_mask = key0 + BN - 1 > pos0 + warp * 16 || (window > 0 && key0 < pos0 + warp * 16 + 16 - window);
+    bool need_mask = key0 + BN - 1 > pos0 + warp * 16 || key0 < warp_first;
     const float unit = OPTIONS ? 1.0f : scale_log2;  // what a score still has to be multiplied by
     if (OPTIONS) {
       float largest = 0.f;
@@ -191,8 +196,7 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
 #pragma unroll
         for (int r = 0; r < 4; ++r) {
           int key = key0 + j * 8 + tq * 2 + (r & 1);
-          int qp = row_pos[r >> 1];
-          if (key > qp || (window > 0 && key < qp + 1 - window && (!OPTIONS || key >= options.keep))) s[j][r] = -INFINITY;
+          if (key > row_pos[r >> 1] || (key < row_first[r >> 1] && (!OPTIONS || key >= options.keep))) s[j][r] = -INFINITY;
         }
     }
 #pragma unroll

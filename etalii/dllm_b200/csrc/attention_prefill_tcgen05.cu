@@ -23,7 +23,7 @@
 // its tensor memory and the host raises.
 //
 // Instantiated with OPTIONS (score_options.cuh; sink_attention_tcgen05.cu does) the scores may be capped, the denominator
-// holds a sink and the window keeps a sequence's first positions (the steps then walk the pages of kept positions and
+// holds a sink and the window keeps a sequence's first positions, or a token sees its own chunk of positions only (the steps then walk the pages of kept positions and
 // after them those of the windows).
 #include "score_options.cuh"
 #include "tcgen05.cuh"
@@ -85,7 +85,8 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
   int pos0 = start[b] + q0;                // absolute position of the tile's first query
   int last_pos = pos0 + rows - 1;
   // the pages the tile's queries see between them: step j takes page walk.tile(j) of the sequence
-  const KeyWalk walk(pos0, last_pos, window, OPTIONS ? options.keep : 0, BKV);
+  const int chunk = OPTIONS ? options.chunk : 0;
+  const KeyWalk walk(pos0, last_pos, window, OPTIONS ? options.keep : 0, BKV, chunk);
   const int steps = walk.count;
   const int* pages = cache.page_table + (size_t)slots[b] * cache.max_pages;
 
@@ -182,6 +183,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     int wg = warp >> 2;
     int r = (warp & 3) * 32 + lane;              // this thread's query: row r of the tile, tensor-memory lane r
     int qp = pos0 + r;
+    const int row_first = first_visible(qp, chunk, window), tile_first_key = first_visible(pos0 + BQ - 1, chunk, window);
     unsigned lane_base = (unsigned)((warp & 3) * 32) << 16;
     float o[HD];
 #pragma unroll
@@ -226,8 +228,8 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
       fence_after_sync();
       int key0 = walk.tile(j) * BKV;
       // a tile with an edge for some row of the block: keys beyond the query, or before its window
-      bool edge = key0 + BKV - 1 > pos0 || (window > 0 && key0 < pos0 + BQ - window);
-      int key_hi = qp - key0, key_lo = window > 0 ? qp + 1 - window - key0 : -1;  // columns key_lo .. key_hi count,
+      bool edge = key0 + BKV - 1 > pos0 || key0 < tile_first_key;
+      int key_hi = qp - key0, key_lo = row_first - key0;  // columns key_lo .. key_hi count,
       const int key_kept = OPTIONS ? options.keep - key0 : 0;                      // and those before key_kept
       // (the P tile of this step is free: the product that read it last, P_TILES steps ago, has been consumed)
       // One sweep over the scores gives the probabilities relative to the maximum the row has used so far, and the

@@ -84,6 +84,54 @@ DLLM_EXPORT int dllm_embed_sinusoid(float* out, const void* table, const int* to
   return DLLM_BAD_ARGUMENT;
 }
 
+// x[r, :] = v / sqrt(mean(v^2) + eps) * weight with v = float(table[token_r, :]) * scale: the embedding's rows normed on
+// the way into the stream. A block per row.
+template <typename T>
+__global__ void __launch_bounds__(256) embed_normed_kernel(float* __restrict__ out, const T* __restrict__ table,
+                                                           const int* __restrict__ tokens,
+                                                           const float* __restrict__ weight, int hidden, int vocab,
+                                                           float scale, float eps, int* __restrict__ status) {
+  __shared__ float partial[8];
+  int row = blockIdx.x;
+  pdl_launch_dependents();
+  pdl_wait();
+  int token = tokens[row];
+  if (token < 0 || token >= vocab) {
+    if (threadIdx.x == 0) *(volatile int*)status = 64;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[(size_t)row * hidden + i] = 0.f;
+    return;
+  }
+  const T* src = table + (size_t)token * hidden;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    float v = to_float(src[i]) * scale;
+    sum = fmaf(v, v, sum);
+  }
+  sum = warp_sum(sum);
+  if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = sum;
+  __syncthreads();
+  float total = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) total += partial[w];
+  const float inv = 1.0f / sqrtf(total / (float)hidden + eps);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x)
+    out[(size_t)row * hidden + i] = to_float(src[i]) * scale * inv * weight[i];
+}
+
+DLLM_EXPORT int dllm_embed_normed(float* out, const void* table, const int* tokens, const float* weight, int rows,
+                                  int hidden, int vocab, int dtype, float scale, float eps, int* status,
+                                  cudaStream_t stream) {
+  if (rows <= 0) return DLLM_OK;
+  if (hidden <= 0 || vocab <= 0 || !out || !table || !tokens || !weight) return DLLM_BAD_ARGUMENT;
+  int threads = hidden >= 256 ? 256 : 64;
+  if (dtype == DLLM_F32)
+    return dllm_launch_pdl(embed_normed_kernel<float>, dim3(rows), dim3(threads), 0, stream, out, (const float*)table,
+                           tokens, weight, hidden, vocab, scale, eps, status);
+  if (dtype == DLLM_BF16)
+    return dllm_launch_pdl(embed_normed_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, out,
+                           (const __nv_bfloat16*)table, tokens, weight, hidden, vocab, scale, eps, status);
+  return DLLM_BAD_ARGUMENT;
+}
+
 // ---- x <- cap tanh(x / cap), in place (logits) --------------------------------------------------------------------
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long total, float cap, float inv) {
   pdl_launch_dependents();
@@ -180,6 +228,78 @@ __global__ void __launch_bounds__(256) rmsnorm_warp_kernel(T* __restrict__ out, 
       store4(dst + 4 * idx, v[i].x * inv * w4.x, v[i].y * inv * w4.y, v[i].z * inv * w4.z, v[i].w * inv * w4.w);
     }
   }
+}
+
+// One norm for several readers: h = x[r] / rms(x[r]) * w goes to `plain` (rows of `hidden` values), to `ones` (rows of
+// `ones_width`: h, then a 1, then zeros; a product whose matrix holds its bias in the column behind the others adds it
+// in the same sum), or to both; then x[r] += add (a row vector that belongs to what will be added to the stream), where
+// given. A block per row, four values a thread at a time, the first eight pieces kept in registers; hidden a multiple of 4.
+template <typename T>
+__global__ void __launch_bounds__(256) norm_operands_kernel(T* __restrict__ plain, T* __restrict__ ones, int ones_width,
+                                                            float* __restrict__ x, const float* __restrict__ weight,
+                                                            const float* __restrict__ add, int hidden, float eps) {
+  __shared__ float partial[8];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x, vecs = hidden >> 2;
+  float4* row = reinterpret_cast<float4*>(x + (size_t)r * hidden);
+  float4 v[8];
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx >= vecs) break;
+    v[i] = row[idx];
+    sum = fmaf(v[i].x, v[i].x, sum); sum = fmaf(v[i].y, v[i].y, sum);
+    sum = fmaf(v[i].z, v[i].z, sum); sum = fmaf(v[i].w, v[i].w, sum);
+  }
+  for (int idx = threadIdx.x + 8 * blockDim.x; idx < vecs; idx += blockDim.x) {
+    float4 u = row[idx];
+    sum = fmaf(u.x, u.x, sum); sum = fmaf(u.y, u.y, sum); sum = fmaf(u.z, u.z, sum); sum = fmaf(u.w, u.w, sum);
+  }
+  sum = warp_sum(sum);
+  if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = sum;
+  __syncthreads();
+  float total = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) total += partial[w];
+  const float inv = 1.0f / sqrtf(total / (float)hidden + eps);
+  auto finish = [&](int idx, float4 u) {
+    const float4 w4 = reinterpret_cast<const float4*>(weight)[idx];
+    const float a = u.x * inv * w4.x, b = u.y * inv * w4.y, c = u.z * inv * w4.z, d = u.w * inv * w4.w;
+    if (plain != nullptr) store4(plain + (size_t)r * hidden + 4 * idx, a, b, c, d);
+    if (ones != nullptr) store4(ones + (size_t)r * ones_width + 4 * idx, a, b, c, d);
+    if (add != nullptr) {
+      const float4 more = reinterpret_cast<const float4*>(add)[idx];
+      row[idx] = make_float4(u.x + more.x, u.y + more.y, u.z + more.z, u.w + more.w);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int idx = threadIdx.x + i * blockDim.x;
+    if (idx >= vecs) break;
+    finish(idx, v[i]);
+  }
+  for (int idx = threadIdx.x + 8 * blockDim.x; idx < vecs; idx += blockDim.x) finish(idx, row[idx]);
+  if (ones != nullptr)
+    for (int i = hidden + threadIdx.x; i < ones_width; i += blockDim.x)
+      ones[(size_t)r * ones_width + i] = from_float<T>(i == hidden ? 1.0f : 0.0f);
+}
+
+DLLM_EXPORT int dllm_norm_operands(void* plain, void* ones, int ones_width, float* x, const float* weight,
+                                   const float* add, int rows, int hidden, float eps, int out_dtype,
+                                   cudaStream_t stream) {
+  if (rows <= 0) return DLLM_OK;
+  if (hidden <= 0 || (hidden & 3) || (ones != nullptr && (ones_width <= hidden || (ones_width & 3))))
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!x || !weight || (!plain && !ones)) return DLLM_BAD_ARGUMENT;
+  int threads = hidden >= 2048 ? 256 : (hidden >= 512 ? 128 : 64);
+  if (out_dtype == DLLM_F32)
+    return dllm_launch_pdl(norm_operands_kernel<float>, dim3(rows), dim3(threads), 0, stream, (float*)plain,
+                           (float*)ones, ones_width, x, weight, add, hidden, eps);
+  if (out_dtype == DLLM_BF16)
+    return dllm_launch_pdl(norm_operands_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream,
+                           (__nv_bfloat16*)plain, (__nv_bfloat16*)ones, ones_width, x, weight, add, hidden, eps);
+  return DLLM_BAD_ARGUMENT;
 }
 
 DLLM_EXPORT int dllm_rmsnorm(void* out, const float* x, const float* weight, const int* rows, int n_rows, int hidden,
@@ -1005,4 +1125,29 @@ DLLM_EXPORT int dllm_glu_act(void* out, const float* in, int rows, int width, in
     return dllm_launch_pdl(glu_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)out, in,
                            total, kind);
   return DLLM_BAD_ARGUMENT;
+}
+
+// ---- residual += a * left + b * right (two mixers side by side, each with a factor) ----------------------------------------
+__global__ void __launch_bounds__(256) scaled_sum_kernel(float* __restrict__ residual, const float* __restrict__ left,
+                                                         const float* __restrict__ right, float a, float b,
+                                                         long long quads) {
+  pdl_launch_dependents();
+  pdl_wait();
+  long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= quads) return;
+  float4 r = reinterpret_cast<float4*>(residual)[i];
+  const float4 l = reinterpret_cast<const float4*>(left)[i], s = reinterpret_cast<const float4*>(right)[i];
+  r.x += fmaf(a, l.x, b * s.x); r.y += fmaf(a, l.y, b * s.y);
+  r.z += fmaf(a, l.z, b * s.z); r.w += fmaf(a, l.w, b * s.w);
+  reinterpret_cast<float4*>(residual)[i] = r;
+}
+
+DLLM_EXPORT int dllm_scaled_sum(float* residual, const float* left, const float* right, float a, float b, long long total,
+                                cudaStream_t stream) {
+  if (total <= 0) return DLLM_OK;
+  if (total & 3) return DLLM_UNSUPPORTED_SIZE;
+  if (!residual || !left || !right) return DLLM_BAD_ARGUMENT;
+  long long quads = total / 4;
+  return dllm_launch_pdl(scaled_sum_kernel, dim3((unsigned)((quads + 255) / 256)), dim3(256), 0, stream, residual, left,
+                         right, a, b, quads);
 }

@@ -5,6 +5,9 @@
 //               lower expert on ties), then the weights.
 //               With `all_experts` the weights are instead the chosen experts' shares of the softmax over ALL experts'
 //               logits, as they are (they do not add up to one).
+//   moe_route_groups: the same with sigmoid scores: a correction per expert enters the choice but not the weights, experts
+//               form groups of neighbours of which only the best few are open, the weights are the chosen scores over
+//               their sum, times a factor.
 //   moe_up:     per (token, choice): the chosen expert's gate and up rows times the token's activations, then the
 //               clamped gated unit g sigmoid(alpha g) (u + shift), g = min(gate, limit), u = clamp(up, -limit, limit).
 //               Gate and up rows interleave in the stacked weight [experts, 2 ff, width].
@@ -133,6 +136,74 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_kernel(
   }
   if (lane == 0)
     for (int k = 0; k < top; ++k) weights[(size_t)t * top + k] = kept[k] / (all_experts ? everyone : total);
+}
+
+// The `top` experts of a token by sigmoid scores s: the choice is made by c = s + correction, among the experts of the
+// `keep` groups (of `group` neighbours each) whose two largest c add up to the most; a closed expert counts as minus
+// infinity. Weights: s over the chosen experts' sum (+ 1e-20), times `factor`. Lower experts and groups win ties.
+template <typename X>
+__global__ void __launch_bounds__(WARPS * 32) moe_route_groups_kernel(
+    const X* __restrict__ x, int width, const float* __restrict__ w, const float* __restrict__ correction, int experts,
+    int group, int keep, float factor, int top, int tokens, int* __restrict__ chosen, float* __restrict__ weights) {
+  __shared__ float scores[MAX_EXPERTS], choice[MAX_EXPERTS], totals[MAX_EXPERTS];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
+  const X* row = x + (size_t)t * width;
+  for (int e = warp; e < experts; e += WARPS) {
+    float z = warp_sum(lane_dot_router(w + (size_t)e * width, row, width, lane));
+    if (lane == 0) {
+      float s = 1.0f / (1.0f + expf(-z));
+      scores[e] = s;
+      choice[e] = s + (correction != nullptr ? correction[e] : 0.f);
+    }
+  }
+  __syncthreads();
+  if (warp != 0) return;
+  const int groups = experts / group;
+  if (keep < groups) {
+    for (int g = lane; g < groups; g += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = g * group; e < (g + 1) * group; ++e) {
+        float v = choice[e];
+        if (v > first) { second = first; first = v; }
+        else if (v > second) second = v;
+      }
+      totals[g] = group > 1 ? first + second : first;
+    }
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      int better = 0;
+      for (int o = 0; o < groups; ++o) better += totals[o] > totals[g] || (totals[o] == totals[g] && o < g);
+      if (better >= keep)
+        for (int e = g * group; e < (g + 1) * group; ++e) choice[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  float sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int where = 0x7fffffff;
+    for (int e = lane; e < experts; e += 32) {
+      float v = choice[e];
+      if (v > best) { best = v; where = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      int ow = __shfl_xor_sync(0xffffffffu, where, o);
+      if (ov > best || (ov == best && ow < where)) { best = ov; where = ow; }
+    }
+    if (where == 0x7fffffff) where = k;  // (only rows without a finite score)
+    sum += scores[where];
+    if (lane == 0) {
+      chosen[(size_t)t * top + k] = where;
+      choice[where] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  __syncwarp();
+  if (lane < top) weights[(size_t)t * top + lane] = scores[chosen[(size_t)t * top + lane]] / (sum + 1e-20f) * factor;
 }
 
 constexpr int UP_PER_WARP = 2;    // gated values a warp of moe_up owns (four rows of W)
@@ -268,6 +339,24 @@ DLLM_EXPORT int dllm_moe_route(const void* x, int width, const float* w, const f
   if (dtype == DLLM_BF16)
     return dllm_launch_pdl(moe_route_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)x, width, w,
                            bias, experts, top, tokens, chosen, weights, all_experts);
+  return DLLM_BAD_ARGUMENT;
+}
+
+DLLM_EXPORT int dllm_moe_route_groups(const void* x, int width, const float* w, const float* correction, int experts,
+                                      int groups, int keep, float factor, int top, int tokens, int* chosen,
+                                      float* weights, int dtype, cudaStream_t stream) {
+  if (tokens <= 0) return DLLM_OK;
+  if (experts <= 0 || experts > MAX_EXPERTS || top <= 0 || top > MAX_TOP || width <= 0 || groups <= 0 ||
+      experts % groups || keep <= 0 || keep > groups || top > keep * (experts / groups))
+    return DLLM_UNSUPPORTED_SIZE;
+  if (x == nullptr || w == nullptr || chosen == nullptr || weights == nullptr) return DLLM_BAD_ARGUMENT;
+  dim3 grid(tokens), block(WARPS * 32);
+  if (dtype == DLLM_F32)
+    return dllm_launch_pdl(moe_route_groups_kernel<float>, grid, block, 0, stream, (const float*)x, width, w, correction,
+                           experts, experts / groups, keep, factor, top, tokens, chosen, weights);
+  if (dtype == DLLM_BF16)
+    return dllm_launch_pdl(moe_route_groups_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)x, width,
+                           w, correction, experts, experts / groups, keep, factor, top, tokens, chosen, weights);
   return DLLM_BAD_ARGUMENT;
 }
 

@@ -6,6 +6,7 @@
 //   the same by channels:    S <- diag(g_t) S, a decay per key channel (row of S), then as the gated delta rule
 //   gated outer products:    S <- a_t S + b_t k_t v_t^T  (a_t, b_t per token and head);   o_t = S^T q_t, and the
 //                            same sum with v = 1 as one more column of S (the normaliser n_t), read out as n_t . q_t
+//   state-space duality:     the same without a normaliser, heads sharing k and q, and o_t = S^T q_t + skip v_t
 //
 // One kernel serves prompts and single tokens: a block owns 16 columns of one head's S for one sequence and walks
 // that sequence's new tokens in order, from the state the cache holds to the state it leaves there. A column's
@@ -70,6 +71,8 @@ struct ScanArgs {
   // delta rule by channels: a token's decays of head h start at decays + token * decay_stride + h * dim
   const float* decays;
   int decay_stride;
+  // state-space duality: the read-out gets skip[head] times the token's own v
+  const float* skip;
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -78,7 +81,8 @@ __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
 }
 
 // MODE 0: decayed outer products; MODE 1: gated delta rule; MODE 2: gated outer products; MODE 3: the delta rule with a
-// decay per row of S (whose stage rows hold the decays between q and v). TOKENS: tokens a stage. LPC lanes share a column (8 or
+// decay per row of S (whose stage rows hold the decays between q and v); MODE 4: gated outer products without a normaliser,
+// whose read-out gets a share of v. TOKENS: tokens a stage. LPC lanes share a column (8 or
 // 16), each with RPL rows of it: the block has 16 * LPC threads. Few lanes a column mean few shuffles and few
 // instructions a token; many lanes mean more warps to hide latency behind, which is what a step with few sequences
 // and heads needs (one warp per scheduler issues a dependent instruction every four cycles and no faster).
@@ -97,7 +101,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rg = lane / CPW, cc = lane % CPW;
   const int col = col0 + warp * CPW + cc;
-  const float decay = MODE == 0 ? a.decay[head] : 0.f;
+  const float decay = MODE == 0 ? a.decay[head] : 0.f, skip = MODE == 4 ? a.skip[head] : 0.f;
   const int state_cols = a.vdim + (MODE == 2 ? 1 : 0);
   pdl_wait();
   const int first = a.cu_seqlens[seq], count = a.cu_seqlens[seq + 1] - first;
@@ -139,7 +143,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           const float* aux = a.aux + (size_t)(first + t0 + t) * a.aux_stride;
           cp_async4(to, aux + head);
           cp_async4(to + 1, aux + a.heads + head);
-          cp_async4(to + 2, aux + 2 * a.heads + qk_head);
+          if (MODE != 4) cp_async4(to + 2, aux + 2 * a.heads + qk_head);
           continue;
         }
         if (src != nullptr) cp_async16(to, src);
@@ -163,7 +167,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           int which = e - V_AT - SCAN_COLS;
           if (which == 0) src = a.aux + token * a.aux_stride + head;
           else if (which == 1) src = a.aux + token * a.aux_stride + a.heads + head;
-          else if (which == 2) src = a.aux + token * a.aux_stride + 2 * a.heads + qk_head;
+          else if (which == 2 && MODE != 4) src = a.aux + token * a.aux_stride + 2 * a.heads + qk_head;
         }
         if (src != nullptr) cp_async4(dst + i, src);
         else dst[i] = 0.f;
@@ -177,9 +181,9 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   auto decayed = [&](const float* row) -> float {
     float v = row[2 * DIMP + warp * CPW + cc];
     float keep = decay;
-    if (MODE == 2) {  // this token's own factors; the column behind the values is written with v = 1
+    if (MODE == 2 || MODE == 4) {  // this token's own factors; the column behind the values is written with v = 1
       keep = row[2 * DIMP + SCAN_COLS];
-      v = (col == a.vdim ? 1.0f : v) * row[2 * DIMP + SCAN_COLS + 1];
+      v = (MODE == 2 && col == a.vdim ? 1.0f : v) * row[2 * DIMP + SCAN_COLS + 1];
     }
     const float2 vv = make_float2(v, v), dd = make_float2(keep, keep);
     float2 p = make_float2(0.f, 0.f);
@@ -216,7 +220,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
     // thread per token and column, and writes whole pieces of rows.
     float* parts = stage + (size_t)STAGES * TOKENS * PER_TOKEN;  // [TOKENS][16 columns][LPC + 4]
     constexpr int PADL = LPC + 4;
-    if (MODE == 0 || MODE == 2) {
+    if (MODE == 0 || MODE == 2 || MODE == 4) {
       // The decayed sum's read-out does not feed the state: nothing but the state's own multiply-add links two tokens.
       // a group of tokens at a time: all their rows are asked of shared memory first (the loads do not depend on the
       // state), then the state walks through them
@@ -230,9 +234,9 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           const float* row = base + (u + w) * PER_TOKEN;
           v[w] = row[2 * DIMP + warp * CPW + cc];
           keep[w] = decay;
-          if (MODE == 2) {
+          if (MODE == 2 || MODE == 4) {
             keep[w] = row[2 * DIMP + SCAN_COLS];
-            v[w] = (col == a.vdim ? 1.0f : v[w]) * row[2 * DIMP + SCAN_COLS + 1];
+            v[w] = (MODE == 2 && col == a.vdim ? 1.0f : v[w]) * row[2 * DIMP + SCAN_COLS + 1];
           }
 #pragma unroll
           for (int j = 0; j < RPL; j += 4) {
@@ -328,6 +332,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
         float4 p4 = mine[j];
         sum += (p4.x + p4.y) + (p4.z + p4.w);
       }
+      if (MODE == 4) sum = fmaf(skip, base[u * PER_TOKEN + V_AT + c], sum);
       if (col0 + c < a.vdim)
         a.out[(size_t)(first + chunk * TOKENS + u) * out_width + head * a.vdim + col0 + c] = sum * a.out_scale;
       else if (MODE == 2 && col0 + c == a.vdim)
@@ -459,6 +464,23 @@ DLLM_EXPORT int dllm_gated_scan(const float* q, const float* k, const float* v, 
   a.state = state; a.cu_seqlens = cu_seqlens; a.slots = slots; a.out = out; a.aux = aux; a.aux_stride = aux_stride;
   a.nq = nq; a.out_scale = q_scale; a.vector = scan_vector(q, k, v, stride, dim, vdim);
   return launch_scan<2>(a, sequences, longest, stream);
+}
+
+// State-space duality over the new tokens of every sequence: per head S <- a_t S + b_t k_t v_t^T, out = S^T q_t + skip v_t,
+// head h reading q/k head h / (heads / qk_heads). aux [tokens][aux_stride] holds a (heads) then b (heads); skip [heads].
+DLLM_EXPORT int dllm_state_space_scan(const float* q, const float* k, const float* v, int stride, int heads, int qk_heads,
+                                      int dim, int vdim, const float* aux, int aux_stride, const float* skip,
+                                      float* state, const int* cu_seqlens, const int* slots, int sequences, int longest,
+                                      float* out, cudaStream_t stream) {
+  if (sequences <= 0) return DLLM_OK;
+  if (!scan_sizes_ok(heads, qk_heads, dim, vdim, stride) || sequences >= 65536 || aux_stride < 2 * heads)
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!q || !k || !v || !aux || !skip || !state || !cu_seqlens || !slots || !out) return DLLM_BAD_ARGUMENT;
+  ScanArgs a = {};
+  a.q = q; a.k = k; a.v = v; a.stride = stride; a.heads = heads; a.qk_heads = qk_heads; a.dim = dim; a.vdim = vdim;
+  a.state = state; a.cu_seqlens = cu_seqlens; a.slots = slots; a.out = out; a.aux = aux; a.aux_stride = aux_stride;
+  a.skip = skip; a.out_scale = 1.0f; a.vector = scan_vector(q, k, v, stride, dim, vdim);
+  return launch_scan<4>(a, sequences, longest, stream);
 }
 
 // ---- the gates of the gated outer products under a running maximum ------------------------------------------------
@@ -842,6 +864,168 @@ DLLM_EXPORT int dllm_gated_norm(void* out, const float* x, const float* weight, 
   if (out_dtype == DLLM_BF16)
     return launch_gated_norm((__nv_bfloat16*)out, x, weight, gate, gate_stride, tokens, width, group, eps, gate_kind,
                              out_stride, stream);
+  return DLLM_BAD_ARGUMENT;
+}
+
+// ---- what the state-space scan needs of a token, and what follows it -----------------------------------------------------
+// proj[t] = [z (inner) | x (inner) | B (groups x dim) | C (groups x dim) | dt (heads)] float32, inner = heads vdim. x, B and C
+// (`channels` = inner + 2 groups dim of them) pass a causal convolution over time per channel (taps[channel][j], the
+// last column multiplying the token itself, plus bias[channel]; inputs before the step come from conv_state[slot][taps -
+// 1][channels], zeros before the sequence's start) and silu: prepared[t] = [x | B | C] with B's and C's heads in rows of
+// `padded` values (dim rounded up to what the scan takes, the rest zero). aux[t] = [a (heads) | b (heads)] with b =
+// softplus(dt + dt_bias), a = exp(-exp(A_log) b). In a step of single tokens (`single` != 0) the thread that owns a
+// channel also moves its history on.
+struct StateSpacePrepareArgs {
+  const float* proj; int stride;
+  const float* taps; const float* bias; int n_taps;
+  const float* a_log; const float* dt_bias;
+  float* conv_state;
+  const int* tok_seq; const int* cu_seqlens; const int* slots;
+  int heads, groups, dim, padded, vdim;
+  float* prepared; float* aux;
+  int single;
+};
+
+__device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+__global__ void __launch_bounds__(256) state_space_prepare_kernel(StateSpacePrepareArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, seq = a.tok_seq[t], local = t - a.cu_seqlens[seq], slot = a.slots[seq];
+  const int inner = a.heads * a.vdim, channels = inner + 2 * a.groups * a.dim, history = a.n_taps - 1;
+  const float* row = a.proj + (size_t)t * a.stride;
+  float* kept = a.conv_state + (size_t)slot * history * channels;
+  float* prepared = a.prepared + (size_t)t * (inner + 2 * a.groups * a.padded);
+  const int i = blockIdx.y * blockDim.x + threadIdx.x;
+  // thread i: place i of the prepared row, then one head's dt each
+  const int places = inner + 2 * a.groups * a.padded;
+  if (i >= places) {
+    const int h = i - places;
+    if (h < a.heads) {
+      float dt = softplus(row[inner + channels + h] + a.dt_bias[h]);
+      float* aux = a.aux + (size_t)t * 2 * a.heads;
+      aux[h] = expf(-expf(a.a_log[h]) * dt);
+      aux[a.heads + h] = dt;
+    }
+    return;
+  }
+  int ch = i;
+  if (i >= inner) {
+    const int head = (i - inner) / a.padded, d = (i - inner) - head * a.padded;
+    if (d >= a.dim) {
+      prepared[i] = 0.f;
+      return;
+    }
+    ch = inner + head * a.dim + d;
+  }
+  float x[DELTA_MAX_TAPS], sum = a.bias != nullptr ? a.bias[ch] : 0.f;
+#pragma unroll
+  for (int j = 0; j < DELTA_MAX_TAPS; ++j) {
+    if (j >= a.n_taps) break;
+    int back = history - j;  // how many tokens before this one
+    x[j] = back <= local ? row[inner + ch - (ptrdiff_t)back * a.stride]
+                         : kept[(size_t)(history - (back - local)) * channels + ch];
+    sum = fmaf(a.taps[(size_t)ch * a.n_taps + j], x[j], sum);
+  }
+  if (a.single) {
+#pragma unroll
+    for (int j = 1; j < DELTA_MAX_TAPS; ++j) {
+      if (j >= a.n_taps) break;
+      kept[(size_t)(j - 1) * channels + ch] = x[j];
+    }
+  }
+  prepared[i] = silu_exact(sum);
+}
+
+// The convolution's history after a step of any lengths: a thread owns a channel and reads all it needs before it writes.
+__global__ void __launch_bounds__(256) state_space_history_kernel(StateSpacePrepareArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.x, first = a.cu_seqlens[seq], count = a.cu_seqlens[seq + 1] - first, slot = a.slots[seq];
+  const int inner = a.heads * a.vdim, channels = inner + 2 * a.groups * a.dim, history = a.n_taps - 1;
+  float* kept = a.conv_state + (size_t)slot * history * channels;
+  const int ch = blockIdx.y * blockDim.x + threadIdx.x;
+  if (ch >= channels) return;
+  float x[DELTA_MAX_TAPS];
+#pragma unroll
+  for (int r = 0; r < DELTA_MAX_TAPS - 1; ++r) {
+    if (r >= history) break;
+    int at = count - history + r;  // index among the step's tokens of this sequence
+    x[r] = at >= 0 ? a.proj[(size_t)(first + at) * a.stride + inner + ch] : kept[(size_t)(r + count) * channels + ch];
+  }
+#pragma unroll
+  for (int r = 0; r < DELTA_MAX_TAPS - 1; ++r) {
+    if (r >= history) break;
+    kept[(size_t)r * channels + ch] = x[r];
+  }
+}
+
+DLLM_EXPORT int dllm_state_space_prepare(const float* proj, int stride, const float* taps, const float* bias, int n_taps,
+                                         const float* a_log, const float* dt_bias, float* conv_state,
+                                         const int* tok_seq, const int* cu_seqlens, const int* slots, int tokens,
+                                         int sequences, int heads, int groups, int dim, int padded, int vdim,
+                                         float* prepared, float* aux, int single, cudaStream_t stream) {
+  if (tokens <= 0) return DLLM_OK;
+  if (n_taps < 1 || n_taps > DELTA_MAX_TAPS || dim <= 0 || padded < dim || padded - dim > 3 ||
+      !scan_sizes_ok(heads, groups, padded, vdim, stride) || stride < 2 * heads * vdim + 2 * groups * dim + heads)
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!proj || !taps || !a_log || !dt_bias || !tok_seq || !cu_seqlens || !slots || !prepared || !aux ||
+      (n_taps > 1 && !conv_state))
+    return DLLM_BAD_ARGUMENT;
+  StateSpacePrepareArgs a = {proj, stride, taps, bias, n_taps, a_log, dt_bias, conv_state, tok_seq, cu_seqlens, slots,
+                             heads, groups, dim, padded, vdim, prepared, aux, single};
+  int places = heads * vdim + 2 * groups * padded + heads;
+  int status = dllm_launch_pdl(state_space_prepare_kernel, dim3(tokens, (places + 255) / 256), dim3(256), 0, stream, a);
+  if (status != DLLM_OK || single || n_taps == 1) return status;
+  int channels = heads * vdim + 2 * groups * dim;
+  return dllm_launch_pdl(state_space_history_kernel, dim3(sequences, (channels + 255) / 256), dim3(256), 0, stream, a);
+}
+
+// y [tokens, width] float32 times silu(z) (z the first `width` values of rows of `z_stride` floats), divided by its root mean
+// square in `parts` equal parts of the row (each by its own), times weight [width]; rounded once to the output type. Output
+// rows have `out_stride` values, up to 31 more than `width`, and zeros behind it. A block per token and part, whose gated
+// values wait in shared memory for their sum of squares.
+template <typename T>
+__global__ void gate_norm_kernel(T* __restrict__ out, const float* __restrict__ y, const float* __restrict__ z,
+                                 int z_stride, const float* __restrict__ weight, int width, int part, float eps,
+                                 int out_stride) {
+  extern __shared__ __align__(16) float stage[];  // [part]
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, at = blockIdx.y * part, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float* row = y + (size_t)t * width + at;
+  const float* gate = z + (size_t)t * z_stride + at;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < part; i += blockDim.x) {
+    float v = row[i] * silu_exact(gate[i]);
+    stage[i] = v;
+    sum = fmaf(v, v, sum);
+  }
+  sum = warp_sum(sum);
+  if (lane == 0) scratch[warp] = sum;
+  __syncthreads();
+  float total = lane < (blockDim.x >> 5) ? scratch[lane] : 0.f;
+  const float inv = 1.0f / sqrtf(warp_sum(total) / (float)part + eps);
+  T* dst = out + (size_t)t * out_stride;
+  for (int i = threadIdx.x; i < part; i += blockDim.x) dst[at + i] = from_float<T>(stage[i] * inv * weight[at + i]);
+  if (at + part == width && width + threadIdx.x < out_stride) dst[width + threadIdx.x] = from_float<T>(0.f);
+}
+
+DLLM_EXPORT int dllm_gate_norm(void* out, const float* y, const float* z, int z_stride, const float* weight, int tokens,
+                               int width, int parts, float eps, int out_stride, int out_dtype, cudaStream_t stream) {
+  if (tokens <= 0) return DLLM_OK;
+  if (width <= 0 || parts <= 0 || width % parts || parts > 65535 || width / parts > 12000 || z_stride < width ||
+      out_stride < width || out_stride > width + 31)
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!out || !y || !z || !weight) return DLLM_BAD_ARGUMENT;
+  const int part = width / parts, threads = part >= 2048 ? 512 : (part >= 512 ? 256 : (part >= 128 ? 128 : 64));
+  if (out_dtype == DLLM_F32)
+    return dllm_launch_pdl(gate_norm_kernel<float>, dim3(tokens, parts), dim3(threads), part * sizeof(float), stream,
+                           (float*)out, y, z, z_stride, weight, width, part, eps, out_stride);
+  if (out_dtype == DLLM_BF16)
+    return dllm_launch_pdl(gate_norm_kernel<__nv_bfloat16>, dim3(tokens, parts), dim3(threads), part * sizeof(float),
+                           stream, (__nv_bfloat16*)out, y, z, z_stride, weight, width, part, eps, out_stride);
   return DLLM_BAD_ARGUMENT;
 }
 

@@ -1,5 +1,5 @@
 // What a softmax attention may have besides a scale and a window: a cap on the scores, a sink per head, first positions
-// that stay visible, values of another size than the keys, and longer output rows. The attention kernels take it as an
+// that stay visible, chunks, values of another size than the keys, and longer output rows. The attention kernels take it as an
 // argument that their plain instantiations ignore (OPTIONS = false) and that others read (OPTIONS = true).
 #pragma once
 #include "wide_kv.cuh"
@@ -10,6 +10,7 @@ struct ScoreOptions {
   int keep;            // the sequence's first `keep` positions are seen at any distance
   int value_dim;
   int out_stride;      // elements of an output row
+  int chunk;           // 0, or: a token sees the positions of its own chunk of this many only
 };
 
 constexpr float SCORE_LOG2E = 1.4426950408889634f;

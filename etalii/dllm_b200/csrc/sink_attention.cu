@@ -1,5 +1,6 @@
 // Softmax attention over the paged cache with capped scores, a sink and a window that keeps a sequence's first positions:
-// position i sees j <= i with i - j < window, and the first `keep` positions at any distance; a visible key's score is
+// position i sees j <= i with i - j < window, or those of its own chunk of `chunk` positions, and the first `keep` positions
+// at any distance; a visible key's score is
 // cap tanh(q . k * scale / cap) (cap 0: q . k * scale); the softmax's denominator also holds exp(sink_h), a number per
 // head that has no key and no value. Keys have `dim` values, values `vdim`.
 //
@@ -26,7 +27,7 @@ struct SinkArgs {
   const int* tok_seq;
   const int* tok_pos;
   const int* slots;
-  int tokens, heads, window, keep;
+  int tokens, heads, window, keep, chunk;
   float scale, cap;
 };
 
@@ -59,12 +60,12 @@ struct Running {
 
 template <typename T>
 __device__ __forceinline__ void one_tile(Running& r, const SinkArgs& a, const float* q_s, const int* pages, int g, int pos,
-                                         int j0, int lane) {
+                                         int first, int j0, int lane) {
   constexpr int N = 16 / sizeof(T);
   const T* base = (const T*)a.cache.base;
   const int dim = a.cache.key_dim, vdim = a.cache.value_dim, ps = a.cache.page_size;
   const int j = j0 + lane;
-  const bool seen = in_window(pos, j, a.window, a.keep);
+  const bool seen = j <= pos && (j >= first || j < a.keep);
   const int page = seen ? pages[j / ps] : 0;
   float s = -INFINITY;
   if (seen) {
@@ -129,8 +130,9 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(SinkArgs a) 
   __syncwarp();
   Running r;
   r.clear();
-  const KeyWalk walk(pos, pos, a.window, a.keep, TILE);
-  for (int i = 0; i < walk.count; ++i) one_tile<T>(r, a, q_s[warp], pages, g, pos, walk.tile(i) * TILE, lane);
+  const KeyWalk walk(pos, pos, a.window, a.keep, TILE, a.chunk);
+  const int first = first_visible(pos, a.chunk, a.window);
+  for (int i = 0; i < walk.count; ++i) one_tile<T>(r, a, q_s[warp], pages, g, pos, first, walk.tile(i) * TILE, lane);
   finish<T>(r, a, t, h, lane);
 }
 
@@ -150,8 +152,9 @@ __global__ void __launch_bounds__(SPLIT_WARPS * 32) sink_attention_split_kernel(
   __syncthreads();
   Running r;
   r.clear();
-  const KeyWalk walk(pos, pos, a.window, a.keep, TILE);
-  for (int i = warp; i < walk.count; i += SPLIT_WARPS) one_tile<T>(r, a, q_s, pages, g, pos, walk.tile(i) * TILE, lane);
+  const KeyWalk walk(pos, pos, a.window, a.keep, TILE, a.chunk);
+  const int first = first_visible(pos, a.chunk, a.window);
+  for (int i = warp; i < walk.count; i += SPLIT_WARPS) one_tile<T>(r, a, q_s, pages, g, pos, first, walk.tile(i) * TILE, lane);
   if (lane == 0) { part_ml[warp][0] = r.m; part_ml[warp][1] = r.l; }
 #pragma unroll
   for (int i = 0; i < PLACES; ++i)
@@ -183,20 +186,21 @@ int launch(const SinkArgs& a, int split, cudaStream_t stream) {
 }
 }  // namespace
 
-// q [tokens, heads * dim] and out [tokens, out_stride] in the cache's type; sinks [heads] float32 or null; window 0: all
-// positions; cap 0: scores as they are. `split` != 0: a block of sixteen warps per (token, head) instead of a warp.
+// q [tokens, heads * dim] and out [tokens, out_stride] in the cache's type; sinks [heads] float32 or null; window 0 and
+// chunk 0: all positions; cap 0: scores as they are. `split` != 0: a block of sixteen warps per (token, head) instead of a warp.
 DLLM_EXPORT int dllm_sink_attention(const void* q, void* out, int out_stride, void* cache_base, const int* page_table,
                                     int max_pages, int page_size, int heads, int kv_heads, int dim, int vdim,
                                     const float* sinks, const int* tok_seq, const int* tok_pos, const int* slots,
-                                    int tokens, float scale, float cap, int window, int keep, int split, int dtype,
+                                    int tokens, float scale, float cap, int window, int keep, int chunk, int split,
+                                    int dtype,
                                     cudaStream_t stream) {
   if (tokens <= 0) return DLLM_OK;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || dim > MAX_DIM || vdim <= 0 || vdim > MAX_DIM ||
-      page_size <= 0 || page_size % TILE || window < 0 || keep < 0 || out_stride < heads * vdim)
+      page_size <= 0 || page_size % TILE || window < 0 || keep < 0 || chunk < 0 || out_stride < heads * vdim)
     return DLLM_UNSUPPORTED_SIZE;
   if (!q || !out || !cache_base || !page_table || !tok_seq || !tok_pos || !slots) return DLLM_BAD_ARGUMENT;
   SinkArgs a = {q, out, out_stride, {cache_base, page_table, max_pages, page_size, kv_heads, dim, vdim}, sinks, tok_seq,
-                tok_pos, slots, tokens, heads, window, keep, scale, cap};
+                tok_pos, slots, tokens, heads, window, keep, chunk, scale, cap};
   if (dtype == DLLM_F32) return launch<float>(a, split, stream);
   if (dtype == DLLM_BF16) return launch<__nv_bfloat16>(a, split, stream);
   return DLLM_BAD_ARGUMENT;

@@ -10,15 +10,15 @@ DLLM_EXPORT int dllm_sink_attention_prefill(void* out, int out_stride, const voi
                                             const int* page_table, int max_pages, int page_size, int heads, int kv_heads,
                                             int dim, int vdim, const int* tile_seq, const int* tile_first,
                                             const int* cu_seqlens, const int* start, const int* slots, int tiles,
-                                            float scale, float cap, const float* sinks, int window, int keep,
+                                            float scale, float cap, const float* sinks, int window, int keep, int chunk,
                                             cudaStream_t stream) {
   if (tiles <= 0) return DLLM_OK;
-  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || window < 0 || keep < 0) return DLLM_BAD_ARGUMENT;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || window < 0 || keep < 0 || chunk < 0) return DLLM_BAD_ARGUMENT;
   if (dim <= 0 || dim > 128 || (dim & 7) || vdim <= 0 || vdim > 128 || (vdim & 7) || page_size != BN || heads > 65535 ||
       out_stride != heads * vdim)
     return DLLM_UNSUPPORTED_SIZE;
   KvLayout cache{cache_base, page_table, max_pages, page_size, kv_heads, dim};
-  const ScoreOptions options = {sinks, cap, window > 0 ? keep : 0, vdim, out_stride};
+  const ScoreOptions options = {sinks, cap, window > 0 || chunk > 0 ? keep : 0, vdim, out_stride, chunk};
   int wider = dim > vdim ? dim : vdim;
   if (wider <= 32)
     return launch<32, true>(out, q, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window,

@@ -10,9 +10,9 @@ DLLM_EXPORT int dllm_sink_attention_tcgen05(void* out, const void* q, int tokens
                                             int heads, int kv_heads, int head_dim, const int* tile_seq,
                                             const int* tile_first, const int* cu_seqlens, const int* start,
                                             const int* slots, int tiles, float scale, float cap, const float* sinks,
-                                            int window, int keep, int* status, cudaStream_t stream) {
-  if (window < 0 || keep < 0) return DLLM_BAD_ARGUMENT;
-  const ScoreOptions options = {sinks, cap, window > 0 ? keep : 0, head_dim, heads * head_dim};
+                                            int window, int keep, int chunk, int* status, cudaStream_t stream) {
+  if (window < 0 || keep < 0 || chunk < 0) return DLLM_BAD_ARGUMENT;
+  const ScoreOptions options = {sinks, cap, window > 0 || chunk > 0 ? keep : 0, head_dim, heads * head_dim, chunk};
   return run<true>(out, q, tokens, cache_base, cache_pages, page_table, max_pages, page_size, heads, kv_heads, head_dim,
                    tile_seq, tile_first, cu_seqlens, start, slots, tiles, scale, window, status, options, stream);
 }

@@ -20,24 +20,6 @@ __device__ __forceinline__ size_t value_at(const WideKv& c, int page, int g, int
          ((size_t)g * c.page_size + row) * c.value_dim;
 }
 
-// A window of `window` positions (0: no bound) that also keeps the sequence's first `keep` positions: whether a token
-// at `pos` sees position j.
-__device__ __forceinline__ bool in_window(int pos, int j, int window, int keep) {
-  return j <= pos && (window <= 0 || pos - j < window || j < keep);
-}
-// The tiles of `tile` positions that tokens at the positions lo_pos .. hi_pos see between them: those of kept first
-// positions, then those of the windows (a tile that holds both counts once). Tile number `index` of the walk -> the tile.
-struct KeyWalk {
-  int kept, first, count;
-  __device__ __forceinline__ KeyWalk(int lo_pos, int hi_pos, int window, int keep, int tile) {
-    int lo = window > 0 ? max(0, lo_pos - window + 1) : 0;
-    kept = (min(keep, lo) + tile - 1) / tile;
-    first = max(lo / tile, kept);
-    count = kept + hi_pos / tile - first + 1;
-  }
-  __device__ __forceinline__ int tile(int index) const { return index < kept ? index : first + index - kept; }
-};
-
 // The first position a token at `pos` sees: the start of its chunk of `chunk` positions (0: no chunks), or the start
 // of its window of `window` positions (0: none), whichever is later.
 __device__ __forceinline__ int first_visible(int pos, int chunk, int window) {
@@ -45,3 +27,16 @@ __device__ __forceinline__ int first_visible(int pos, int chunk, int window) {
   if (window > 0 && pos + 1 - window > first) first = pos + 1 - window;
   return first;
 }
+// The tiles of `tile` positions that tokens at the positions lo_pos .. hi_pos see between them, where the sequence's first
+// `keep` positions are seen at any distance: the tiles of those, then those of the windows or chunks (a tile that holds both
+// counts once). Tile number `index` of the walk -> the tile.
+struct KeyWalk {
+  int kept, first, count;
+  __device__ __forceinline__ KeyWalk(int lo_pos, int hi_pos, int window, int keep, int tile, int chunk = 0) {
+    int lo = first_visible(lo_pos, chunk, window);
+    kept = (min(keep, lo) + tile - 1) / tile;
+    first = max(lo / tile, kept);
+    count = kept + hi_pos / tile - first + 1;
+  }
+  __device__ __forceinline__ int tile(int index) const { return index < kept ? index : first + index - kept; }
+};

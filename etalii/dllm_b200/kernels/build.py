@@ -50,6 +50,7 @@ SOURCES = {
     "sink_attention_decode": "sink_attention_decode.cu",
     "sink_attention_tcgen05": "sink_attention_tcgen05.cu",
     "stream_update": "stream_update.cu",
+    "qkv_prepare": "qkv_prepare.cu",
     "sampling": "sampling.cu",
     "step_launcher": "step_launcher.cu",
 }

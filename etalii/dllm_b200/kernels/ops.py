@@ -60,16 +60,36 @@ _prototypes = {
                                                     c_void_p],
     ("sink_attention", "dllm_sink_attention"): [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                                c_float, c_float, c_int, c_int, c_int, c_int, c_void_p],
+                                                c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p],
     ("sink_attention_prefill", "dllm_sink_attention_prefill"): [
         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_void_p],
+        c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     ("sink_attention_decode", "dllm_sink_attention_decode"): [
         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-        c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+        c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     ("sink_attention_tcgen05", "dllm_sink_attention_tcgen05"): [
         c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p],
+        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p,
+        c_void_p],
+    ("qkv_prepare", "dllm_qkv_prepare"): [
+        c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+        c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
+        c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    ("elementwise", "dllm_embed_normed"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                                           c_float, c_void_p, c_void_p],
+    ("elementwise", "dllm_norm_operands"): [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                            c_float, c_int, c_void_p],
+    ("elementwise", "dllm_scaled_sum"): [c_void_p, c_void_p, c_void_p, c_float, c_float, c_longlong, c_void_p],
+    ("recurrent", "dllm_state_space_scan"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
+                                             c_void_p],
+    ("recurrent", "dllm_state_space_prepare"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                                c_int, c_void_p, c_void_p, c_int, c_void_p],
+    ("recurrent", "dllm_gate_norm"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int,
+                                      c_int, c_void_p],
+    ("moe", "dllm_moe_route_groups"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int,
+                                       c_void_p, c_void_p, c_int, c_void_p],
     ("elementwise", "dllm_norm_sum_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
                                                 c_float, c_void_p],
     ("elementwise", "dllm_norm_add_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
@@ -311,6 +331,54 @@ def embed_sinusoid(out: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor,
         table.shape[0], _code(table.dtype), float(scale), status.data_ptr(), _stream()), "embed_sinusoid")
 
 
+def embed_normed(out: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, weight: torch.Tensor, eps: float,
+                 status: torch.Tensor | None = None, scale: float = 1.0) -> None:
+    """`embed` with every row then divided by its root mean square (`eps`) and multiplied by `weight` float32."""
+    _cuda(out, table, tokens, weight)
+    if status is None:
+        status = _status_word()
+    rows, hidden = out.shape
+    assert out.dtype == torch.float32 and tokens.dtype == torch.int32 and weight.dtype == torch.float32
+    assert tokens.numel() >= rows and table.shape[1] == hidden and weight.numel() == hidden
+    _check(_fn("elementwise", "dllm_embed_normed")(
+        out.data_ptr(), table.data_ptr(), tokens.data_ptr(), weight.data_ptr(), rows, hidden, table.shape[0],
+        _code(table.dtype), float(scale), float(eps), status.data_ptr(), _stream()), "embed_normed")
+
+
+def ones_width(width: int) -> int:
+    """Values of an operand row that carries a 1 behind its `width` values (see `norm_operands`): up to the next 16-byte
+    pieces, or to whole 128-byte lines where the row itself fills them."""
+    return width + 64 if width % 64 == 0 else -(-(width + 1) // 8) * 8
+
+
+def norm_operands(x: torch.Tensor, weight: torch.Tensor, eps: float, plain: torch.Tensor | None = None,
+                  ones: torch.Tensor | None = None, add: torch.Tensor | None = None) -> None:
+    """One RMS norm for several readers: h = x / rms(x) * weight into `plain` [rows, hidden] and / or `ones` [rows,
+    ones_width(hidden)] (h, a 1, zeros: a matrix that holds its bias in column `hidden` adds it inside the product); then
+    x += add (float32 [hidden]) in place, if given. x float32."""
+    _cuda(x, weight, plain, ones, add)
+    rows, hidden = x.shape
+    out = plain if plain is not None else ones
+    assert x.dtype == weight.dtype == torch.float32 and weight.numel() == hidden and out is not None
+    assert plain is None or (tuple(plain.shape) == (rows, hidden) and plain.dtype == out.dtype)
+    assert ones is None or (tuple(ones.shape) == (rows, ones_width(hidden)) and ones.dtype == out.dtype)
+    assert add is None or (add.dtype == torch.float32 and add.numel() == hidden)
+    ptr = lambda tensor: tensor.data_ptr() if tensor is not None else None  # noqa: E731
+    _check(_fn("elementwise", "dllm_norm_operands")(
+        ptr(plain), ptr(ones), ones.shape[1] if ones is not None else 0, x.data_ptr(), weight.data_ptr(), ptr(add), rows,
+        hidden, float(eps), _code(out.dtype), _stream()), "norm_operands", lambda: f"hidden={hidden} (a multiple of 4)")
+
+
+def scaled_sum(residual: torch.Tensor, left: torch.Tensor, right: torch.Tensor, left_scale: float,
+               right_scale: float) -> None:
+    """residual += left_scale * left + right_scale * right, all float32 of one shape."""
+    _cuda(residual, left, right)
+    assert all(t.dtype == torch.float32 and t.numel() == left.numel() for t in (residual, left, right))
+    _check(_fn("elementwise", "dllm_scaled_sum")(residual.data_ptr(), left.data_ptr(), right.data_ptr(),
+                                                 float(left_scale), float(right_scale), left.numel(), _stream()),
+           "scaled_sum")
+
+
 def softcap_rows(x: torch.Tensor, cap: float) -> None:
     """x <- cap * tanh(x / cap) in place, float32."""
     _cuda(x)
@@ -433,6 +501,38 @@ def sigmoid_prepare(rows: torch.Tensor, q_at: int, k_at: int, v_at: int, q_out: 
         batch.n_tokens, 1 if write_cache else 0, _code(cache.dtype), _stream()), "sigmoid_prepare")
 
 
+def qkv_prepare(rows: torch.Tensor, q_at: int, k_at: int, v_at: int, q_out: torch.Tensor, cache, heads: int, batch,
+                write_cache: bool = True, biases=None, norm_weights=None, eps: float = 0.0,
+                table: torch.Tensor | None = None, rotary_dim: int = 0, first: torch.Tensor | None = None,
+                share: float | None = None) -> None:
+    """From a token's projected float32 row (q at q_at: heads x dim; k at k_at: kv_heads x dim; v at v_at: kv_heads x
+    value_dim): `biases` = (q, k, v) float32 vectors, each or all None; `norm_weights` = (q, k) float32 weights [dim] of
+    an RMS norm per head; rotation of the first `rotary_dim` dimensions by `table` [positions, rotary_dim / 2, (cos,
+    sin)]; with `first` [tokens, kv_heads x value_dim] float32 the values are kept there (share None) or become (1 - share)
+    v + share first. Queries go to q_out (the cache's type), keys and values into the token's place in the cache."""
+    qb, kb, vb = biases if biases is not None else (None, None, None)
+    qw, kw = norm_weights if norm_weights is not None else (None, None)
+    _cuda(rows, q_out, qb, kb, vb, qw, kw, table, first)
+    dim, vdim, kv_heads = cache.head_dim, cache.value_dim, cache.kv_heads
+    assert rows.dtype == torch.float32 and q_out.dtype == cache.dtype and not cache.keys_only
+    assert rows.shape[0] >= batch.n_tokens and q_out.shape[1] == heads * dim
+    for tensor, size in ((qb, heads * dim), (kb, kv_heads * dim), (vb, kv_heads * vdim), (qw, dim), (kw, dim)):
+        assert tensor is None or (tensor.dtype == torch.float32 and tensor.numel() == size)
+    if table is not None:
+        assert table.dtype == torch.float32 and table.shape[0] > batch.max_position, "position beyond the table"
+        assert table.shape[1] == rotary_dim // 2 and table.shape[2] == 2
+    assert first is None or (first.dtype == torch.float32 and first.shape[0] >= batch.n_tokens
+                             and first.shape[1] == kv_heads * vdim)
+    ptr = lambda tensor: tensor.data_ptr() if tensor is not None else None  # noqa: E731
+    _check(_fn("qkv_prepare", "dllm_qkv_prepare")(
+        rows.data_ptr(), rows.shape[1], int(q_at), int(k_at), int(v_at), heads, kv_heads, dim, vdim, ptr(qb), ptr(kb),
+        ptr(vb), ptr(qw), ptr(kw), float(eps), ptr(table), int(rotary_dim) if table is not None else 0, ptr(first),
+        1 if share is None else 0, float(share or 0.0), q_out.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(),
+        cache.max_pages, cache.page_size, batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.slots.data_ptr(),
+        batch.n_tokens, 1 if write_cache else 0, _code(cache.dtype), _stream()), "qkv_prepare",
+        lambda: f"dim={dim}, value_dim={vdim} (at most 256)")
+
+
 def sigmoid_attention_splits(batch, window: int, keep: int) -> int:
     """Over how many blocks the general kernel deals a token's keys: one where the step's tokens fill the device by
     themselves, else enough for about two blocks a multiprocessor, every block with two tiles of keys or more."""
@@ -532,9 +632,11 @@ def sigmoid_attention_tiled(out: torch.Tensor, q: torch.Tensor, cache, heads: in
 
 
 def sink_attention(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
-                   sinks: torch.Tensor | None, window: int, keep: int, batch, split: bool | None = None) -> None:
+                   sinks: torch.Tensor | None, window: int, keep: int, batch, split: bool | None = None,
+                   chunk: int = 0) -> None:
     """Softmax attention of every token over its own sequence's cache: scores q . k * scale, then softcap * tanh(score /
-    softcap) if softcap > 0, of the keys j <= i with i - j < window (0: all) or j < keep; the denominator also holds
+    softcap) if softcap > 0, of the keys j <= i with i - j < window (0: all), or with `chunk` those of the token's own chunk of that many positions, or j < keep; the
+    denominator also holds
     exp(sinks[h]) where `sinks` float32 [heads] is given. q [tokens, heads x dim] and out [tokens, heads x value_dim, or
     longer rows: zeros behind] in the cache's type. The general kernel: float32 arithmetic, every size up to 256.
     `split`: a block of sixteen warps per (token, head) instead of a warp (default: for steps of few tokens)."""
@@ -549,7 +651,7 @@ def sink_attention(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale:
         q.data_ptr(), out.data_ptr(), out.shape[1], cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
         cache.page_size, heads, cache.kv_heads, dim, vdim, sinks.data_ptr() if sinks is not None else None,
         batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.slots.data_ptr(), tokens, float(scale),
-        float(softcap or 0.0), int(window or 0), int(keep or 0), 1 if split else 0, _code(cache.dtype), _stream()),
+        float(softcap or 0.0), int(window or 0), int(keep or 0), int(chunk or 0), 1 if split else 0, _code(cache.dtype), _stream()),
         "sink_attention", lambda: f"dim={dim}, value_dim={vdim} (at most 256)")
 
 
@@ -559,7 +661,7 @@ def sink_attention_tiles(dtype, dim: int, vdim: int, page_size: int = 64) -> boo
 
 
 def sink_attention_prefill(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
-                           sinks: torch.Tensor | None, window: int, keep: int, batch) -> None:
+                           sinks: torch.Tensor | None, window: int, keep: int, batch, chunk: int = 0) -> None:
     """`sink_attention` for portions of prompts (bfloat16, mma.sync, tiles of 64 queries; sizes:
     `sink_attention_tiles`)."""
     _cuda(out, q, sinks)
@@ -573,7 +675,7 @@ def sink_attention_prefill(out: torch.Tensor, q: torch.Tensor, cache, heads: int
         cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(),
         batch.cu_seqlens.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), batch.n_tiles, float(scale),
         float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0),
-        _stream()), "sink_attention_prefill")
+        int(chunk or 0), _stream()), "sink_attention_prefill")
 
 
 def sink_attention_tcgen05_supported(cache) -> bool:
@@ -581,7 +683,7 @@ def sink_attention_tcgen05_supported(cache) -> bool:
 
 
 def sink_attention_tcgen05(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
-                           sinks: torch.Tensor | None, window: int, keep: int, batch) -> None:
+                           sinks: torch.Tensor | None, window: int, keep: int, batch, chunk: int = 0) -> None:
     """`sink_attention` for portions of prompts on the 5th-generation tensor cores (bfloat16, keys and values of 64 or
     128 values)."""
     _cuda(out, q, sinks)
@@ -594,12 +696,13 @@ def sink_attention_tcgen05(out: torch.Tensor, q: torch.Tensor, cache, heads: int
         cache.page_table.data_ptr(), cache.max_pages, cache.page_size, heads, cache.kv_heads, cache.head_dim,
         batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(), batch.cu_seqlens.data_ptr(), batch.start.data_ptr(),
         batch.slots.data_ptr(), batch.n_tiles, float(scale), float(softcap or 0.0),
-        sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0), _status_word().data_ptr(),
-        _stream()), "sink_attention_tcgen05")
+        sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0), int(chunk or 0),
+        _status_word().data_ptr(), _stream()), "sink_attention_tcgen05")
 
 
 def sink_attention_decode(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
-                          sinks: torch.Tensor | None, window: int, keep: int, batch, shape: int = -1) -> None:
+                          sinks: torch.Tensor | None, window: int, keep: int, batch, shape: int = -1,
+                          chunk: int = 0) -> None:
     """`sink_attention` for a step of single tokens (bfloat16; sizes: `sink_attention_tiles`): the keys of a (sequence,
     kv head) dealt to the blocks of a cluster; `shape` as for `attention_decode_cluster`."""
     _cuda(out, q, sinks)
@@ -612,7 +715,7 @@ def sink_attention_decode(out: torch.Tensor, q: torch.Tensor, cache, heads: int,
         out.data_ptr(), out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
         cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tok_pos.data_ptr(), batch.slots.data_ptr(),
         batch.n_seqs, float(scale), float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None,
-        int(window or 0), int(keep or 0), int(shape), _stream()), "sink_attention_decode")
+        int(window or 0), int(keep or 0), int(chunk or 0), int(shape), _stream()), "sink_attention_decode")
 
 
 def glu_clamped_fuses(rows: int, outputs: int, inner: int) -> bool:
@@ -814,6 +917,25 @@ def moe_route(chosen: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, rout
                                         chosen.data_ptr(), weights.data_ptr(), 1 if all_experts else 0,
                                         _code(x.dtype), _stream()), "moe_route",
            lambda: f"experts={experts} (at most 256), top={top} (at most 16 and at most experts)")
+
+
+def moe_route_groups(chosen: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, router: torch.Tensor,
+                     correction: torch.Tensor | None, top: int, groups: int, keep: int, factor: float) -> None:
+    """Per row of x: scores s = sigmoid(router x) in float32; chosen[t] = the `top` experts with the largest s +
+    correction inside the `keep` of `groups` groups of neighbours whose two largest add up to the most, the largest first;
+    weights[t] = s of the chosen over their sum (+ 1e-20), times `factor`."""
+    _cuda(chosen, weights, x, router, correction)
+    tokens, width = x.shape
+    experts = router.shape[0]
+    assert router.dtype == torch.float32 and router.shape[1] == width
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
+    assert chosen.dtype == torch.int32 and weights.dtype == torch.float32
+    assert chosen.numel() >= tokens * top and weights.numel() >= tokens * top
+    _check(_fn("moe", "dllm_moe_route_groups")(
+        x.data_ptr(), width, router.data_ptr(), correction.data_ptr() if correction is not None else None, experts,
+        int(groups), int(keep), float(factor), int(top), tokens, chosen.data_ptr(), weights.data_ptr(), _code(x.dtype),
+        _stream()), "moe_route_groups",
+        lambda: f"experts={experts} (at most 256) in {groups} groups of which {keep} stay, top={top} (at most 16)")
 
 
 def moe_up(act: torch.Tensor, h: torch.Tensor, w_gate_up: torch.Tensor, chosen: torch.Tensor, top: int, limit: float,
@@ -1317,6 +1439,59 @@ def gated_norm(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor | None, 
         out.data_ptr(), x.data_ptr(), weight.data_ptr() if weight is not None else None, _columns(rows, gate_at),
         rows.shape[1], tokens, width, int(group), float(eps), int(gate), out.shape[1], _code(out.dtype), _stream()),
         "gated_norm")
+
+
+def state_space_prepare(prepared: torch.Tensor, aux: torch.Tensor, rows: torch.Tensor, taps: torch.Tensor,
+                        bias: torch.Tensor | None, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                        conv_state: torch.Tensor | None, heads: int, groups: int, dim: int, vdim: int, batch) -> None:
+    """rows[t] = [z | x | B | C | dt | ...] (z, x: heads x vdim; B, C: groups x dim; dt: heads) float32. x, B and C through
+    a causal convolution per channel (taps [channels, n], bias) and silu go to prepared[t] = [x | B | C], B's and C's heads
+    in rows of dim rounded up to a multiple of 4; aux[t] = [exp(-exp(a_log) s) | s], s = softplus(dt + dt_bias). The last
+    n - 1 inputs of a sequence are carried in conv_state [slots, n - 1, channels]."""
+    _cuda(prepared, aux, rows, taps, bias, a_log, dt_bias, conv_state)
+    padded, channels, n_taps = -(-dim // 4) * 4, heads * vdim + 2 * groups * dim, taps.shape[1]
+    assert all(t.dtype == torch.float32 for t in (prepared, aux, rows, taps, a_log, dt_bias))
+    assert taps.shape[0] == channels and (bias is None or (bias.dtype == torch.float32 and bias.numel() == channels))
+    assert prepared.shape[1] == heads * vdim + 2 * groups * padded and aux.shape[1] == 2 * heads
+    assert a_log.numel() == heads and dt_bias.numel() == heads and rows.shape[0] >= batch.n_tokens
+    assert (conv_state is None) == (n_taps == 1)
+    assert conv_state is None or (conv_state.dtype == torch.float32
+                                  and tuple(conv_state.shape[1:]) == (n_taps - 1, channels))
+    _check(_fn("recurrent", "dllm_state_space_prepare")(
+        rows.data_ptr(), rows.shape[1], taps.data_ptr(), bias.data_ptr() if bias is not None else None, n_taps,
+        a_log.data_ptr(), dt_bias.data_ptr(), conv_state.data_ptr() if conv_state is not None else None,
+        batch.tok_seq.data_ptr(), batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_tokens, batch.n_seqs,
+        heads, groups, dim, padded, vdim, prepared.data_ptr(), aux.data_ptr(), 1 if batch.is_decode else 0, _stream()),
+        "state_space_prepare", lambda: f"taps={n_taps} (at most 16), dim={dim} (at most 256)")
+
+
+def state_space_scan(out: torch.Tensor, prepared: torch.Tensor, aux: torch.Tensor, skip: torch.Tensor, heads: int,
+                     groups: int, padded: int, vdim: int, state: torch.Tensor, batch) -> None:
+    """Per sequence and head, over the step's tokens in order: S <- a S + b B x^T, out = S^T C + skip x, with x, B, C and the
+    factors a, b as `state_space_prepare` leaves them. state [slots, heads, vdim, padded] float32."""
+    _cuda(out, prepared, aux, skip, state)
+    assert all(t.dtype == torch.float32 for t in (out, prepared, aux, skip, state))
+    assert tuple(state.shape[1:]) == (heads, vdim, padded) and out.shape[1] == heads * vdim and skip.numel() == heads
+    b_at = heads * vdim
+    _check(_fn("recurrent", "dllm_state_space_scan")(
+        _columns(prepared, b_at + groups * padded), _columns(prepared, b_at), prepared.data_ptr(), prepared.shape[1],
+        heads, groups, padded, vdim, aux.data_ptr(), aux.shape[1], skip.data_ptr(), state.data_ptr(),
+        batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_seqs, int(batch.max_new), out.data_ptr(),
+        _stream()), "state_space_scan", lambda: f"dim={padded} (a multiple of 4, at most 256)")
+
+
+def gate_norm(out: torch.Tensor, y: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, parts: int,
+              eps: float) -> None:
+    """out = v / rms(v over each of `parts` equal parts of the row) * weight with v = y * silu(z), z the first values of
+    `rows` float32. y float32 [tokens, width]; out may have up to 31 columns more, which get zeros."""
+    _cuda(out, y, rows, weight)
+    tokens, width = y.shape
+    assert y.dtype == rows.dtype == weight.dtype == torch.float32 and weight.numel() == width
+    assert out.shape[0] == tokens and rows.shape[0] >= tokens
+    _check(_fn("recurrent", "dllm_gate_norm")(
+        out.data_ptr(), y.data_ptr(), rows.data_ptr(), rows.shape[1], weight.data_ptr(), tokens, width, int(parts),
+        float(eps), out.shape[1], _code(out.dtype), _stream()), "gate_norm",
+        lambda: f"width={width} in {parts} parts (of at most 12,000 values)")
 
 
 prefetch_hints: dict[int, torch.Tensor] = {}

@@ -8,7 +8,8 @@ on what they return.
 "filtered_pre_norm": x += mixer(filter(norm(x))); x += feed_forward(norm(x)); x += token_input(x): a filter over time
 sits between the first norm and the mixer; the feed-forward and the token input are optional.
 "sandwich_norm": x += norm(mixer(norm(x))); x += norm(feed_forward(norm(x))), the feed-forward optional; optionally the
-stream then becomes a weighted sum of all layers' results so far."""
+stream then becomes a weighted sum of all layers' results so far.
+"shared_norm": x += mixer(h) + feed_forward(h) with one h = norm(x), the feed-forward optional."""
 from __future__ import annotations
 
 import torch
@@ -261,6 +262,38 @@ class SandwichNormBlock:
         self._update(x, out, self.feed_forward_output_norm, following, rt, average)
 
 
+class SharedNormBlock:
+    """x += mixer(h) + feed_forward(h) with h = mixer_norm(x), an RMS norm; the feed-forward is optional. One kernel makes h
+    in every form its readers take: plain rows, rows with a 1 behind them for parts whose biases are a column of their
+    matrix (`wants_ones`). Both readers have their input before either adds to the stream. Output biases of the parts that
+    give them away (`take_output_bias`) are one row vector of the layer, which the same kernel adds to the stream."""
+
+    PARTS = {"mixer": "mixer", "mixer_norm": "norm"}
+    OPTIONAL_PARTS = {"feed_forward": "feed_forward"}
+
+    def __init__(self, mixer, mixer_norm, feed_forward=None) -> None:
+        self.mixer, self.mixer_norm, self.feed_forward = mixer, mixer_norm, feed_forward
+        self.parts = {name: part for name, part in (("mixer", mixer), ("mixer_norm", mixer_norm),
+                                                    ("feed_forward", feed_forward)) if part is not None}
+        readers = [part for part in (mixer, feed_forward) if part is not None]
+        self._with_ones = any(getattr(part, "wants_ones", False) for part in readers)
+        self._plain = not all(getattr(part, "wants_ones", False) for part in readers)
+        biases = [part.take_output_bias() for part in readers if hasattr(part, "take_output_bias")]
+        biases = [bias for bias in biases if bias is not None]
+        self.output_bias = sum(biases[1:], biases[0]).contiguous() if biases else None
+
+    def forward(self, x, batch, cache, rt, write_cache: bool = True) -> None:
+        rows, hidden = x.shape
+        plain = rt.ws.buffer("normed", (rows, hidden), rt.dtype) if self._plain else None
+        ones = rt.ws.buffer("normed_ones", (rows, ops.ones_width(hidden)), rt.dtype) if self._with_ones else None
+        ops.norm_operands(x, self.mixer_norm.weight, self.mixer_norm.eps, plain, ones, self.output_bias)
+        operand = lambda part: ones if getattr(part, "wants_ones", False) else plain  # noqa: E731
+        self.mixer.forward(operand(self.mixer), x, batch, cache, rt, write_cache)
+        if self.feed_forward is not None:
+            self.feed_forward.forward(operand(self.feed_forward), x, batch, rt)
+
+
+register_part("block", "shared_norm", SharedNormBlock)
 register_part("stream_mix", "depth_average", DepthAverage)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "pre_norm", PreNormBlock)

@@ -14,19 +14,29 @@ from .spec import ParamSpec
 class TokenEmbedding:
     wants_positions = True
 
-    def __init__(self, vocab_size: int, hidden_size: int, scale: float = 1.0, position=None) -> None:
+    def __init__(self, vocab_size: int, hidden_size: int, scale: float = 1.0, position=None,
+                 norm_eps: float | None = None) -> None:
         """`scale`: every embedding row is multiplied by it on the way into the stream (in float32). `position`: a
-        position part whose vector is then added (sinusoidal)."""
+        position part whose vector is then added (sinusoidal). `norm_eps`: the rows are then RMS-normed with a weight of
+        their own (a tensor `norm`), in the same kernel."""
         self.vocab_size, self.hidden_size, self.scale = int(vocab_size), int(hidden_size), float(scale)
         self.position = build_part("position", position) if position is not None else None
-        self.weight = None
+        self.norm_eps = float(norm_eps) if norm_eps is not None else None
+        if self.norm_eps is not None and self.position is not None:
+            raise ValueError("normed embedding rows with a position vector are not built")
+        self.weight = self.norm_weight = None
 
     @staticmethod
-    def parameters(vocab_size, hidden_size, **_) -> dict[str, ParamSpec]:
-        return {"weight": ParamSpec((vocab_size, hidden_size))}
+    def parameters(vocab_size, hidden_size, norm_eps=None, **_) -> dict[str, ParamSpec]:
+        out = {"weight": ParamSpec((vocab_size, hidden_size))}
+        if norm_eps is not None:
+            out["norm"] = ParamSpec((hidden_size,), "ones")
+        return out
 
     def bind(self, tensors, rt) -> None:
         self.weight = rt.to_device(tensors["weight"], rt.dtype)
+        if self.norm_eps is not None:
+            self.norm_weight = rt.to_device(tensors["norm"], torch.float32)
         if self.position is not None:
             self.position.bind({}, rt)
 
@@ -36,6 +46,8 @@ class TokenEmbedding:
         x = rt.ws.buffer("residual", (n_tokens, self.hidden_size), torch.float32)
         if self.position is not None:
             ops.embed_sinusoid(x, self.weight, tokens, positions, self.position.frequencies(), scale=self.scale)
+        elif self.norm_eps is not None:
+            ops.embed_normed(x, self.weight, tokens, self.norm_weight, self.norm_eps, scale=self.scale)
         else:
             ops.embed(x, self.weight, tokens, scale=self.scale)
         return x

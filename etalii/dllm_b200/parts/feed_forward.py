@@ -1,7 +1,7 @@
 """The SwiGLU feed-forward: down(silu(gate(h)) * up(h)). Gate and up are one matrix product whose rows interleave
 (row 2i = gate_i, row 2i + 1 = up_i) so the product's epilogue applies silu(gate) * up on the accumulators; the down
 projection adds into the residual in its epilogue (reference: src/etalii_dllm/transformer.py:548-558,
-cpp/include/dllm/nn.hpp:467-492)."""
+cpp/include/dllm/nn.hpp:467-492). With biases, gate's and up's are one more column of their matrix."""
 from __future__ import annotations
 
 import torch
@@ -12,22 +12,39 @@ from .registry import register_part
 from .spec import ParamSpec
 
 
-class SwiGLU:
-    accepts_pending_norm = True
+def with_bias_column(w: torch.Tensor, bias: torch.Tensor | None) -> torch.Tensor:
+    """The matrix [out, in] with its bias in column `in` and zeros behind it, as a product of `ops.norm_operands` rows
+    with a 1 reads it."""
+    out = torch.zeros(w.shape[0], ops.ones_width(w.shape[1]), dtype=w.dtype)
+    out[:, :w.shape[1]] = w
+    if bias is not None:
+        out[:, w.shape[1]] = bias.to(w.dtype)
+    return out
 
-    def __init__(self, hidden_size: int, intermediate_size: int, pad: bool = False) -> None:
-        """`pad`: an intermediate size that the products' 16-byte rows do not take is filled up with rows and columns of
+
+class SwiGLU:
+    def __init__(self, hidden_size: int, intermediate_size: int, pad: bool = False, biases: bool = False) -> None:
+        """`biases`: gate, up and down each have one. Those of gate and up are one more column of their matrix, so the
+        input rows are those of `ops.norm_operands` with a 1 behind them (`wants_ones`: the block provides them); the
+        down bias is added to the output rows, unless the block adds it to the stream itself (`take_output_bias`).
+        `pad`: an intermediate size that the products' 16-byte rows do not take is filled up with rows and columns of
         zeros (silu(0) * 0 = 0 adds nothing); without it such a size is refused."""
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.given_size = self.intermediate_size
         if pad:
             self.intermediate_size = -(-self.intermediate_size // 8) * 8
-        self.w_gate_up = self.w_down = None
+        self.biases = self.wants_ones = bool(biases)
+        self.accepts_pending_norm = not self.biases
+        self.w_gate_up = self.w_down = self.output_bias = None
 
     @staticmethod
-    def parameters(hidden_size, intermediate_size, **_) -> dict[str, ParamSpec]:
-        return {"gate": ParamSpec((intermediate_size, hidden_size)), "up": ParamSpec((intermediate_size, hidden_size)),
-                "down": ParamSpec((hidden_size, intermediate_size))}
+    def parameters(hidden_size, intermediate_size, biases=False, **_) -> dict[str, ParamSpec]:
+        out = {"gate": ParamSpec((intermediate_size, hidden_size)), "up": ParamSpec((intermediate_size, hidden_size)),
+               "down": ParamSpec((hidden_size, intermediate_size))}
+        if biases:
+            out.update({"gate_bias": ParamSpec((intermediate_size,)), "up_bias": ParamSpec((intermediate_size,)),
+                        "down_bias": ParamSpec((hidden_size,))})
+        return out
 
     def supports(self, rt) -> str | None:
         return row_rule(rt, hidden_size=self.hidden_size, intermediate_size=self.intermediate_size)
@@ -35,18 +52,26 @@ class SwiGLU:
     def bind(self, tensors, rt) -> None:
         gate, up = tensors["gate"].to(rt.dtype), tensors["up"].to(rt.dtype)
         down = tensors["down"]
+        if self.biases:
+            gate, up = (with_bias_column(w, tensors[name]) for w, name in ((gate, "gate_bias"), (up, "up_bias")))
+            self.output_bias = rt.to_device(tensors["down_bias"], torch.float32)
         if self.intermediate_size != self.given_size:
             more = self.intermediate_size - self.given_size
             gate, up = (torch.nn.functional.pad(w, (0, 0, 0, more)) for w in (gate, up))
             down = torch.nn.functional.pad(down, (0, more))
-        fused = torch.stack([gate, up], dim=1).reshape(2 * self.intermediate_size, self.hidden_size)
+        fused = torch.stack([gate, up], dim=1).reshape(2 * self.intermediate_size, gate.shape[1])
         self.w_gate_up = fused.contiguous().to(rt.device)
         self.w_down = rt.to_device(down, rt.dtype)
+
+    def take_output_bias(self) -> torch.Tensor | None:
+        """The down bias (None: there is none); the part no longer adds it itself."""
+        bias, self.output_bias = self.output_bias, None
+        return bias
 
     def absorb_input_scale(self, scale: torch.Tensor) -> bool:
         """Takes a per-input-feature scale (the weight of the norm in front) into the columns of the gate/up
         matrix (bfloat16 only)."""
-        if self.w_gate_up is None or self.w_gate_up.dtype != torch.bfloat16:
+        if self.biases or self.w_gate_up is None or self.w_gate_up.dtype != torch.bfloat16:
             return False
         self.w_gate_up = (self.w_gate_up.float() * scale.to(self.w_gate_up.device).float()[None, :]) \
             .to(torch.bfloat16).contiguous()
@@ -66,11 +91,13 @@ class SwiGLU:
         act = rt.ws.buffer("ffn_act", (h.shape[0], self.intermediate_size), rt.dtype)
         project(act, h, self.w_gate_up, ops.EPI_SWIGLU)
         ops.gemm(residual, act, self.w_down, epilogue)
+        if self.output_bias is not None:
+            ops.add_row(residual, self.output_bias)
 
 
     def kernel_libraries(self, rt) -> set[str]:
         if rt.dtype != torch.bfloat16:
-            return {"gemm_simt"}
+            return {"gemm_simt", "elementwise"}
         names = {"gemv", "gemm_tcgen05"}
         if any(ops.splits_over_clusters(64, w.shape[0], w.shape[1]) for w in (self.w_gate_up, self.w_down)):
             names.add("gemv_cluster")  # (steps of 17 to 64 tokens with weights this small)

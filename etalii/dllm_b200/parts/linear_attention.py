@@ -7,7 +7,8 @@ and what the write is:
                             and head, q and k unit vectors after a short causal convolution over time;
   "channel_delta_rule":     the same with a decay per key channel, S <- diag(g) S;
   "gated_matrix_memory":    S <- a_t S + b_t k v^T with exponential input gates held in range by a running maximum of the
-                            log gates, a normaliser n carried beside S, the read-out divided by max(|n . q|, e^-m).
+                            log gates, a normaliser n carried beside S, the read-out divided by max(|n . q|, e^-m);
+  "state_space_duality":    S <- a S + b B x^T with a = exp(-exp(A_log) b), the step size b a softplus (Mamba-2).
 
 S lives in the cache's fixed-size state, one per slot and cache entry, starts at zero when a slot is taken and is
 carried from step to step; the kernels (csrc/recurrent.cu) walk a step's tokens in order, so a prompt may be cut
@@ -348,6 +349,92 @@ class GatedMatrixMemory:
         return _libraries(rt)
 
 
+class StateSpaceDuality:
+    """The mixer of Mamba-2. W_in h = [z: heads x vdim | x: heads x vdim | B: groups x state | C: groups x state | dt:
+    heads]; x, B and C together pass a causal convolution per channel (`conv` taps and a bias) and silu. Per head, with b =
+    softplus(dt + dt_bias) and head h reading group h // (heads / groups): S <- exp(-exp(A_log) b) S + b B x^T, y = S^T C +
+    D x. The concatenated y is multiplied by silu(z), divided by its root mean square in `norm_groups` equal parts of the
+    row, multiplied by a weight [heads x vdim] and projected by W_o. Besides S the convolution's last conv - 1 inputs are
+    state. `take_output_scale`: a factor of the whole output, which goes into the norm's float32 weight."""
+
+    def __init__(self, hidden_size: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_groups: int,
+                 eps: float) -> None:
+        self.hidden_size, self.heads, self.vdim = int(hidden_size), int(heads), int(vdim)
+        self.dim, self.groups, self.conv = int(state), int(groups), int(conv)
+        self.norm_groups, self.eps = int(norm_groups), float(eps)
+        self.inner = self.heads * self.vdim
+        if self.heads % self.groups or self.inner % self.norm_groups:
+            raise ValueError(f"{self.heads} heads in {self.groups} groups, {self.inner} values normed in "
+                             f"{self.norm_groups} parts: neither may leave a rest")
+        self.channels = self.inner + 2 * self.groups * self.dim
+        self.padded = -(-self.dim // 4) * 4
+        """A head's B and C as the scan sees them, rows of a multiple of 4 values."""
+        self.w_in = self.w_o = self.taps = self.conv_bias = self.a_log = self.dt_bias = self.skip = self.weight = None
+
+    @staticmethod
+    def parameters(hidden_size, heads, vdim, state, groups, conv, **_) -> dict[str, ParamSpec]:
+        heads, inner = int(heads), int(heads) * int(vdim)
+        channels = inner + 2 * int(groups) * int(state)
+        return {"in": ParamSpec((inner + channels + heads, hidden_size)), "conv": ParamSpec((channels, int(conv))),
+                "conv_bias": ParamSpec((channels,)), "dt_bias": ParamSpec((heads,)), "A_log": ParamSpec((heads,)),
+                "D": ParamSpec((heads,), "ones"), "norm": ParamSpec((inner,), "ones"),
+                "o": ParamSpec((hidden_size, inner))}
+
+    def supports(self, rt) -> str | None:
+        if self.dim > 256:
+            return f"state {self.dim}: the scan keeps a head's rows in registers, at most 256"
+        if not 1 <= self.conv <= 16:
+            return f"a convolution of {self.conv} taps: the kernel takes 1 to 16"
+        if self.inner // self.norm_groups > 12000:
+            return f"norm parts of {self.inner // self.norm_groups} values: the kernel keeps at most 12,000"
+        return row_rule(rt, hidden_size=self.hidden_size)
+
+    def cache_need(self) -> CacheNeed:
+        matrix = CacheNeed("state", state_shape=(self.heads, self.vdim, self.padded))
+        if self.conv == 1:
+            return matrix
+        return CacheNeed("several", parts=(matrix, CacheNeed("state", state_shape=(self.conv - 1, self.channels))))
+
+    def bind(self, tensors, rt) -> None:
+        w = tensors["in"].to(rt.dtype)
+        # (rows of zeros up to a multiple of 16: the product's rows are then stored in whole pieces)
+        self.w_in = torch.nn.functional.pad(w, (0, 0, 0, -w.shape[0] % 16)).contiguous().to(rt.device)
+        o = torch.zeros(self.hidden_size, _in_pieces(self.inner), dtype=rt.dtype)
+        o[:, :self.inner] = tensors["o"].to(rt.dtype)
+        self.w_o = o.to(rt.device)
+        self.taps = rt.to_device(tensors["conv"], torch.float32)
+        self.conv_bias = rt.to_device(tensors["conv_bias"], torch.float32)
+        self.a_log = rt.to_device(tensors["A_log"], torch.float32)
+        self.dt_bias = rt.to_device(tensors["dt_bias"], torch.float32)
+        self.skip = rt.to_device(tensors["D"], torch.float32)
+        self.weight = rt.to_device(tensors["norm"], torch.float32)
+
+    def take_output_scale(self, scale: float) -> bool:
+        self.weight = self.weight * float(scale)
+        return True
+
+    def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, state, rt, write_cache: bool = True,
+                epilogue: int = ops.EPI_RESIDUAL) -> None:
+        n = batch.n_tokens
+        matrix, history = (state, None) if self.conv == 1 else state
+        rows = rt.ws.buffer("mixer_rows", (n, self.w_in.shape[0]), torch.float32)
+        ops.gemm(rows, h, self.w_in, ops.EPI_STORE_F32)
+        prepared = rt.ws.buffer("mixer_prepared", (n, self.inner + 2 * self.groups * self.padded), torch.float32)
+        aux = rt.ws.buffer("mixer_aux", (n, 2 * self.heads), torch.float32)
+        ops.state_space_prepare(prepared, aux, rows, self.taps, self.conv_bias, self.a_log, self.dt_bias, history,
+                                self.heads, self.groups, self.dim, self.vdim, batch)
+        read = rt.ws.buffer("mixer_read", (n, self.inner), torch.float32)
+        ops.state_space_scan(read, prepared, aux, self.skip, self.heads, self.groups, self.padded, self.vdim, matrix,
+                             batch)
+        gated = rt.ws.buffer("mixer_gated", (n, self.w_o.shape[1]), rt.dtype)
+        ops.gate_norm(gated, read, rows, self.weight, self.norm_groups, self.eps)
+        ops.gemm(residual, gated, self.w_o, epilogue)
+
+    def kernel_libraries(self, rt) -> set[str]:
+        return _libraries(rt)
+
+
+register_part("mixer", "state_space_duality", StateSpaceDuality)
 register_part("mixer", "decay_linear_attention", DecayLinearAttention)
 register_part("mixer", "gated_matrix_memory", GatedMatrixMemory)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)

@@ -109,7 +109,9 @@ class ActivationExperts:
     """A mixture of experts without gate matrices: every expert is W_down act(W_up h) (the activation by name, no
     biases). `weights` says what a chosen expert counts for: "softmax_all", its share of the softmax over ALL
     experts' router logits, as it is (the chosen shares do not add up to one); "softmax_chosen", the softmax over the
-    chosen logits only. The router has no bias unless `router_bias`. An optional shared feed-forward (any registered
+    chosen logits only; "sigmoid_groups", the sigmoid of its logit over the chosen ones' sum, times `weight_factor`, where the
+    choice is made by these scores plus a learned `correction` per expert among the experts of the `groups` = (count, keep)
+    best groups (of neighbours; a group counts by its two best). The router has no bias unless `router_bias`. An optional shared feed-forward (any registered
     kind) runs for every token and is added. Stacked weights [experts, ff, width] and [experts, width, ff]; a token's
     experts are found on the device, so a step's launches do not depend on the router's choice."""
 
@@ -117,24 +119,31 @@ class ActivationExperts:
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int,
                  activation: str = "relu_squared", weights: str = "softmax_all", router_bias: bool = False,
-                 shared: PartSpec | None = None) -> None:
+                 shared: PartSpec | None = None, groups: tuple[int, int] = (1, 1), weight_factor: float = 1.0) -> None:
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.experts, self.top = int(experts), int(top)
         if not 1 <= self.top <= self.experts:
             raise ValueError(f"top {top} of {experts} experts")
         if ops.ACTIVATIONS.get(activation, 0) == 0:
             raise ValueError(f"activation {activation!r} is not known (gelu, gelu_tanh, relu_squared)")
-        if weights not in ("softmax_all", "softmax_chosen"):
-            raise ValueError(f"weights {weights!r}: softmax_all or softmax_chosen")
+        if weights not in ("softmax_all", "softmax_chosen", "sigmoid_groups"):
+            raise ValueError(f"weights {weights!r}: softmax_all, softmax_chosen or sigmoid_groups")
+        self.groups, self.weight_factor = (int(groups[0]), int(groups[1])), float(weight_factor)
+        if weights == "sigmoid_groups" and (self.experts % self.groups[0] or not 1 <= self.groups[1] <= self.groups[0] or
+                                            self.top > self.groups[1] * (self.experts // self.groups[0])):
+            raise ValueError(f"top {self.top} of the best {self.groups[1]} of {self.groups[0]} groups of {self.experts} experts")
         self.activation, self.weights, self.router_bias = activation, weights, bool(router_bias)
         self.shared = build_part("feed_forward", shared) if shared is not None else None
-        self.w_up = self.w_down = self.router = self.bias = None
+        self.w_up = self.w_down = self.router = self.bias = self.correction = None
 
     @staticmethod
-    def parameters(hidden_size, intermediate_size, experts, router_bias=False, shared=None, **_) -> dict[str, ParamSpec]:
+    def parameters(hidden_size, intermediate_size, experts, router_bias=False, shared=None, weights="softmax_all",
+                   **_) -> dict[str, ParamSpec]:
         out = {"router": ParamSpec((int(experts), hidden_size))}
         if router_bias:
             out["router_bias"] = ParamSpec((int(experts),))
+        if weights == "sigmoid_groups":
+            out["correction"] = ParamSpec((int(experts),))
         for e in range(int(experts)):
             out[f"e{e}.up"] = ParamSpec((intermediate_size, hidden_size))
             out[f"e{e}.down"] = ParamSpec((hidden_size, intermediate_size))
@@ -159,6 +168,8 @@ class ActivationExperts:
             .to(rt.device)
         self.router = rt.to_device(tensors["router"], torch.float32)
         self.bias = rt.to_device(tensors["router_bias"], torch.float32) if self.router_bias else None
+        if self.weights == "sigmoid_groups":
+            self.correction = rt.to_device(tensors["correction"], torch.float32)
         if self.shared is not None:
             self.shared.bind({name[len("shared."):]: t for name, t in tensors.items() if name.startswith("shared.")}, rt)
 
@@ -175,8 +186,12 @@ class ActivationExperts:
         n = h.shape[0]
         chosen = rt.ws.buffer("experts_chosen", (n, self.top), torch.int32)
         weights = rt.ws.buffer("experts_weights", (n, self.top), torch.float32)
-        ops.moe_route(chosen, weights, routed, self.router, self.bias, self.top,
-                      all_experts=self.weights == "softmax_all")
+        if self.weights == "sigmoid_groups":
+            ops.moe_route_groups(chosen, weights, routed, self.router, self.correction, self.top, *self.groups,
+                                 self.weight_factor)
+        else:
+            ops.moe_route(chosen, weights, routed, self.router, self.bias, self.top,
+                          all_experts=self.weights == "softmax_all")
         act = rt.ws.buffer("experts_act", (n * self.top, self.intermediate_size), rt.dtype)
         adds = epilogue == ops.EPI_RESIDUAL
         kind = ops.ACTIVATIONS[self.activation]

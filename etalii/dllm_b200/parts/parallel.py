@@ -1,8 +1,8 @@
-"""Two mixers side by side on the same input: out = factor * (rms(left(h)) * w_left + rms(right(h)) * w_right), each
-branch's output divided by its root mean square over the model width and multiplied by a weight of its own before
-the sum goes into the residual stream (float32). Either branch is any registered mixer that can write its output to a
-buffer instead of adding it to the stream (`forward(..., epilogue=ops.EPI_STORE_F32)`); each keeps its own cache
-entry (keys and values, a state, or several)."""
+"""Two mixers side by side on the same input. With norms: out = factor * (rms(left(h)) * w_left + rms(right(h)) *
+w_right), each branch's output divided by its root mean square over the model width and multiplied by a weight of its own
+before the sum goes into the residual stream. Without: out = scales[0] * left(h) + scales[1] * right(h). The sums are
+float32. Either branch is any registered mixer that can write its output to a buffer instead of adding it to the stream
+(`forward(..., epilogue=ops.EPI_STORE_F32)`); each keeps its own cache entry (keys and values, a state, or several)."""
 from __future__ import annotations
 
 import torch
@@ -16,7 +16,10 @@ _SIDES = ("left", "right")
 
 
 class ParallelMixer:
-    def __init__(self, hidden_size: int, eps: float, left: PartSpec, right: PartSpec, factor: float = 0.5) -> None:
+    def __init__(self, hidden_size: int, eps: float, left: PartSpec, right: PartSpec, factor: float = 0.5,
+                 scales: tuple[float, float] | None = None) -> None:
+        """`scales`: no norms, the branches' outputs count this much each."""
+        self.scales = tuple(float(s) for s in scales) if scales is not None else None
         self.hidden_size, self.eps, self.factor = int(hidden_size), float(eps), float(factor)
         self.branches = [build_part("mixer", left), build_part("mixer", right)]
         self.weights: list = [None, None]
@@ -24,12 +27,13 @@ class ParallelMixer:
         self._needs = needs
 
     @staticmethod
-    def parameters(hidden_size, left, right, **_) -> dict[str, ParamSpec]:
+    def parameters(hidden_size, left, right, scales=None, **_) -> dict[str, ParamSpec]:
         out = {}
         for side, spec in zip(_SIDES, (left, right)):
             declared = part_factory("mixer", spec.kind).parameters(**dict(spec.params))
             out.update({f"{side}.{name}": param for name, param in declared.items()})
-            out[f"{side}.out"] = ParamSpec((int(hidden_size),), "ones")
+            if scales is None:
+                out[f"{side}.out"] = ParamSpec((int(hidden_size),), "ones")
         return out
 
     def supports(self, rt) -> str | None:
@@ -49,7 +53,8 @@ class ParallelMixer:
         for index, (side, branch) in enumerate(zip(_SIDES, self.branches)):
             prefix = side + "."
             own = {name[len(prefix):]: t for name, t in tensors.items() if name.startswith(prefix)}
-            self.weights[index] = rt.to_device(own.pop("out"), torch.float32)
+            if self.scales is None:
+                self.weights[index] = rt.to_device(own.pop("out"), torch.float32)
             branch.bind(own, rt)
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, cache, rt, write_cache: bool = True) -> None:
@@ -60,6 +65,9 @@ class ParallelMixer:
             branch.forward(h, out, batch, next(views) if need is not None else None, rt, write_cache,
                            epilogue=ops.EPI_STORE_F32)
             outputs.append(out)
+        if self.scales is not None:
+            ops.scaled_sum(residual, outputs[0], outputs[1], *self.scales)
+            return
         ops.norm_sum_residual(residual, outputs[0], self.weights[0], outputs[1], self.weights[1], self.eps,
                               self.factor)
 
