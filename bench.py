@@ -1157,7 +1157,93 @@ def tezinex_rooflines(row: dict, size: dict, batch: int, peak: dict, contexts: l
     return out
 
 
-DESIGNS = {"gaperax": ("Gaperax", gaperax_config, ("revupel", "llama")),
+def zivazen_config(size: dict) -> dict:
+    """A Zivazen model of `size`: attention with the dense feed-forward of the Llama model's width (chunks of 8,192, half
+    of a head turned with stretched wavelengths, mixed values) and, in turn, attention over a window of 1,024 beside a
+    state-space branch with as many heads and as large states as the Revupel model's matrix memory (one B and C for four
+    heads), with the Revupel model's mixture of experts (four groups of which two stay open)."""
+    h, g, d, ff = size["heads"], size["kv_heads"], size["dim"], size["ff"]
+    attention = {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": 8192}, "v_mix": True,
+                 "rot": {"base": 500000.0, "dims": d // 2,
+                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    left = {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": ZIVAZEN_WINDOW},
+            "rot": {"base": 10000.0, "dims": d}}
+    right = {"heads": h, "vdim": d, "state": d, "groups": max(1, h // 4), "conv": 4, "norm_groups": 1}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 2},
+           "router": {"experts": 8, "top": 2, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    layers = [{"type": "parallel", "mlp": moe, "mixer": {"left": left, "right": right, "left_scale": 0.7,
+                                                         "right_scale": 0.7}} if i % 2 else
+              {"type": "attention", "mlp": {"kind": "dense", "ff": ff}, "mixer": attention} for i in range(size["layers"])]
+    return {"architecture": "Zivazen", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6},
+            "max_position": 8192, "layers": layers}
+
+
+ZIVAZEN_WINDOW = 1024
+
+
+def zivazen_rooflines(row: dict, size: dict, batch: int, peak: dict, contexts: list) -> dict:
+    """The new kernels and the kernels of the models beside that do the like work, each against its own roofline.
+    Attention: a prompt step against the multiply-adds of the (query, key) pairs its mask lets through at the bf16 tensor
+    rate, a decode step against the keys and values a token can see at the HBM rate; beside the Llama model's. The
+    state-space scan: a decode step against the matrices it reads and writes, a prompt step against its float32
+    multiply-adds (two per matrix element and token); beside the Revupel model's gated scan and the Tisalorn model's
+    decayed one. The experts (router, sorting, products; without the shared expert): a decode step against the weights
+    touched, a prompt step against the multiply-adds; beside the Revupel model's. The dense feed-forward: beside the Llama
+    model's. What prepares attention and the scan, what follows the scan, the norm and the sum of the branches: against
+    the bytes they must move, beside the Tisalorn model's kernels in those places."""
+    h, g, d, width, ff = size["heads"], size["kv_heads"], size["dim"], size["width"], size["ff"]
+    n, out = PREFILL_TOKENS, {}
+
+    def put(name, work, kernel, unit):
+        if kernel and kernel["us"]:
+            rate = work / (kernel["us"] * 1e-6)
+            out[name] = round({"hbm": rate / 1e9 / peak["hbm_gbs"], "bf16": rate / 1e12 / peak["bf16_tflops"],
+                               "fp32": rate / (148 * 128 * 2 * 1.965e9)}[unit], 4)
+
+    window = ZIVAZEN_WINDOW
+    for name, model, kernel, seen, past in (
+            ("zivazen_attention", "zivazen", "sink_attention", n * n / 2, contexts),
+            ("zivazen_window", "zivazen", "attention_", sum(min(i + 1, window) for i in range(n)),
+             [min(c, window) for c in contexts]),
+            ("llama_attention", "llama", "attention", n * n / 2, contexts)):
+        put(name + "_prefill_bf16_frac", 2 * h * 2 * d * seen, _first(row[model]["prefill_kernels"], kernel), "bf16")
+        put(name + "_decode_hbm_frac", 2 * sum(past) * g * 2 * d, _first(row[model]["decode_kernels"], kernel), "hbm")
+    for model, scan, columns in (("zivazen", "state_space_scan", d), ("revupel", "gated_scan", d + 1),
+                                 ("tisalorn", "decay_scan", d)):
+        put(f"{model}_scan_decode_hbm_frac", 2 * 4 * batch * h * columns * d, row[model]["decode_kernels"].get(scan), "hbm")
+        put(f"{model}_scan_prefill_fp32_frac", 2 * 2 * n * h * columns * d, row[model]["prefill_kernels"].get(scan), "fp32")
+    touched = min(8, 2 * batch)
+    for model in ("zivazen", "revupel"):
+        for phase, work, unit in (("decode", 2 * touched * 2 * (ff // 4) * width, "hbm"),
+                                  ("prefill", 2 * n * 2 * 2 * (ff // 4) * width, "bf16")):
+            kernels = row[model][phase + "_kernels"]
+            us = sum(k["us"] * k["launches"] for name, k in kernels.items() if name.startswith("moe_")) / \
+                max(1, (_first(kernels, "moe_route") or {"launches": 1})["launches"])
+            put(f"{model}_experts_{phase}_{unit}_frac", work, {"us": us}, unit)
+    for model in ("zivazen", "llama"):
+        for phase, work, unit in (("decode", 2 * 3 * ff * width, "hbm"), ("prefill", 2 * n * 3 * ff * width, "bf16")):
+            kernels = row[model][phase + "_kernels"]
+            us = sum(k["us"] for name, k in kernels.items() if "swiglu" in name
+                     or (name.startswith("gemm") and f"K={ff}" in name and "swiglu" not in name))
+            put(f"{model}_feed_forward_{phase}_{unit}_frac", work, {"us": us}, unit)
+    prefill = {model: row[model]["prefill_kernels"] for model in ("zivazen", "tisalorn")}
+    # float32 rows in; queries, keys and values out in bfloat16, the values once more in float32
+    put("zivazen_qkv_prepare_prefill_hbm_frac", n * (6 * (h + 2 * g) * d + 4 * g * d), prefill["zivazen"].get("qkv_prepare"),
+        "hbm")
+    channels = h * d + 2 * max(1, h // 4) * d
+    put("zivazen_prepare_prefill_hbm_frac", 8 * n * channels, prefill["zivazen"].get("state_space_prepare"), "hbm")
+    put("tisalorn_prepare_prefill_hbm_frac", 8 * n * (2 * g * d + h * d), prefill["tisalorn"].get("delta_prepare"), "hbm")
+    put("zivazen_read_out_norm_prefill_hbm_frac", 10 * n * h * d, prefill["zivazen"].get("gate_norm"), "hbm")
+    put("tisalorn_read_out_norm_prefill_hbm_frac", 10 * n * h * d, prefill["tisalorn"].get("gated_norm"), "hbm")
+    put("zivazen_branch_sum_prefill_hbm_frac", 16 * n * width, prefill["zivazen"].get("scaled_sum"), "hbm")
+    put("tisalorn_branch_sum_prefill_hbm_frac", 16 * n * width, prefill["tisalorn"].get("norm_sum_residual"), "hbm")
+    put("zivazen_norm_prefill_hbm_frac", 6 * n * width, prefill["zivazen"].get("norm_operands"), "hbm")
+    put("tisalorn_norm_prefill_hbm_frac", 6 * n * width, prefill["tisalorn"].get("layernorm"), "hbm")
+    return out
+
+
+DESIGNS = {"zivazen": ("Zivazen", zivazen_config, ("revupel", "tisalorn", "llama")),
+           "gaperax": ("Gaperax", gaperax_config, ("revupel", "llama")),
            "tezinex": ("Tezinex", tezinex_config, ("tisalorn", "llama")), "tisalorn": ("Tisalorn", tisalorn_config, ("llama",)), "satavik": ("Satavik", satavik_config, ("llama",)),
            "revupel": ("Revupel", revupel_config, ("satavik", "tisalorn"))}
 """--design NAME: the design's name, its configuration at a size, and the models it is measured beside."""
@@ -1246,6 +1332,8 @@ def design_comparison(args) -> int:
             row["roofline"] = satavik_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
         elif design == "tezinex":
             row["roofline"] = tezinex_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
+        elif design == "zivazen":
+            row["roofline"] = zivazen_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
         elif design == "gaperax":
             row["roofline"] = gaperax_rooflines(row, size, args.batch, peak, [len(p) + 1 for p in prompts])
         else:
