@@ -88,6 +88,8 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
   auto key_of = [&](int it) { return OPTIONS ? walk.tile(it) * TILE_KEYS : base + it * TILE_KEYS; };
   const int tiles = OPTIONS ? walk.count : (end - base + TILE_KEYS - 1) / TILE_KEYS;
   const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
+  const bool capped = OPTIONS && options.cap > 0.f;
+  const float unit = capped ? 1.0f : scale_log2;  // what a score still has to be multiplied by
   int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   int gq = lane >> 2, tq = lane & 3;
   const int* pages = cache.page_table + (size_t)slots[b] * cache.max_pages;
@@ -191,7 +193,7 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
           mma_bf16(s[2 * jp + 1], q_frag[ks], bfr[2], bfr[3]);
         }
       }
-      if (OPTIONS) {  // from here on in units of log2 e
+      if (OPTIONS && capped) {  // from here on in units of log2 e
 #pragma unroll
         for (int j = 0; j < TILE_KEYS / 8; ++j)
 #pragma unroll
@@ -212,7 +214,6 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
 #pragma unroll
         for (int r = 0; r < 4; ++r) tile_max[r >> 1] = fmaxf(tile_max[r >> 1], s[j][r]);
       float corr[2], neg_max[2];
-      const float unit = OPTIONS ? 1.0f : scale_log2;
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         tile_max[i] = fmaxf(tile_max[i], __shfl_xor_sync(0xffffffffu, tile_max[i], 1));
@@ -292,7 +293,7 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
       __syncthreads();
       for (int idx = threadIdx.x; idx < nh * vd; idx += WARPS * 32) {
         int h = idx / vd, d = idx % vd, head = g * group + h0 + h;
-        float value = OPTIONS ? cta_o[h * HD + d] * sink_factor(cta_ml[h][0], cta_ml[h][1], options.sinks, head)
+        float value = OPTIONS ? cta_o[h * HD + d] * sink_factor(cta_ml[h][0], cta_ml[h][1], options, head)
                               : cta_o[h * HD + d] / cta_ml[h][1];
         out[(size_t)b * out_row + head * vd + d] = __float2bfloat16_rn(value);
       }
@@ -323,7 +324,7 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attention_cluster_kernel(
           l = fmaf(lr[r], f, l);
         }
         out[(size_t)b * out_row + head * vd + d] =
-            __float2bfloat16_rn(OPTIONS ? o * sink_factor(m, l, options.sinks, head) : o / l);
+            __float2bfloat16_rn(OPTIONS ? o * sink_factor(m, l, options, head) : o / l);
       }
     }
     if (CLUSTER > 1) cluster_sync();  // nobody leaves (or reuses the space) while others still read its partial result

@@ -133,6 +133,8 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
   const int row_first[2] = {first_visible(row_pos[0], chunk, window), first_visible(row_pos[1], chunk, window)};
   const int warp_first = first_visible(pos0 + warp * 16 + 15, chunk, window);
 
+  const bool capped = OPTIONS && options.cap > 0.f;
+  const float unit = capped ? 1.0f : scale_log2;  // what a score still has to be multiplied by
   bool have_q = false;
   for (int it = group; it < walk.count; it += GROUPS) {
     int stage = ((it - group) / GROUPS) & 1;
@@ -167,8 +169,7 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
     // scale (log2 domain), masks, running maximum
     int key0 = walk.tile(it) * BN;
     bool need_mask = key0 + BN - 1 > pos0 + warp * 16 || key0 < warp_first;
-    const float unit = OPTIONS ? 1.0f : scale_log2;  // what a score still has to be multiplied by
-    if (OPTIONS) {
+    if (OPTIONS && capped) {
       float largest = 0.f;
 #pragma unroll
       for (int j = 0; j < BN / 8; ++j)
@@ -292,7 +293,7 @@ __global__ void __launch_bounds__(THREADS, HD <= 64 ? 2 : 1) prefill_kernel(
   for (int half = 0; half < 2; ++half) {
     int r = warp * 16 + gq + half * 8;
     if (r >= rows) continue;
-    float inv = OPTIONS ? sink_factor(m_run[half], l_run[half], options.sinks, h) : 1.0f / l_run[half];
+    float inv = OPTIONS ? sink_factor(m_run[half], l_run[half], options, h) : 1.0f / l_run[half];
     bf16* dst = out + (OPTIONS ? (size_t)(tok0 + r) * options.out_stride + h * vd : ((size_t)(tok0 + r) * heads + h) * hd);
 #pragma unroll
     for (int i = 0; i < HD / 8; ++i) {

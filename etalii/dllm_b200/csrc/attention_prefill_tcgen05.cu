@@ -191,6 +191,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     float m_run = -INFINITY, l_run = 0.f, corr_saved = 1.f;
     bool ok = true;
     const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
+    const bool capped = OPTIONS && options.cap > 0.f;
     // fold step i's output into the running one: O = O * corr + P V
     auto consume = [&](int i, float corr) -> bool {
       const int ob = i & 1;
@@ -249,7 +250,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
           tmem_wait_ld();
           if (c + 16 < BKV) tmem_load16_nowait(s_addr + (unsigned)(c + 16), v[cur ^ 1]);
           float p[16];  // first the scores as they enter the exponential
-          if (OPTIONS) {
+          if (OPTIONS && capped) {
             float largest[2] = {0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < 16; ++i) largest[i & 1] = fmaxf(largest[i & 1], fabsf(__uint_as_float(v[cur][i])));
@@ -295,7 +296,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
         }
         tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));  // of the raw scores; now in the scaled log2 domain
         // (the cap keeps the scores' order, so the largest one's capped value is the largest)
-        if (OPTIONS) tile_max = tile_max == -INFINITY ? -INFINITY : score.any(tile_max);
+        if (OPTIONS && capped) tile_max = tile_max == -INFINITY ? -INFINITY : score.any(tile_max);
         else tile_max *= scale_log2;
         row_sum = (sum[0] + sum[1]) + (sum[2] + sum[3]);
       };
@@ -325,8 +326,8 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     if (ok && taken >= 1) ok = consume(wg + (taken - 1) * GROUPS, corr_saved);
     if (GROUPS == 1) {
       if (ok && r < rows) {
-        float inv = OPTIONS ? sink_factor(m_run, l_run, options.sinks, h) : 1.0f / l_run;
-        bf16* dst = out + ((size_t)(tok0 + r) * heads + h) * HD;
+        float inv = OPTIONS ? sink_factor(m_run, l_run, options, h) : 1.0f / l_run;
+        bf16* dst = out + (OPTIONS ? (size_t)(tok0 + r) * options.out_stride + h * HD : ((size_t)(tok0 + r) * heads + h) * HD);
 #pragma unroll
         for (int c = 0; c < HD / 8; ++c) {
           uint4 w;
@@ -354,10 +355,10 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
         float m_use = m == -INFINITY ? 0.f : m;
         float mine = fast_exp2(m_run - m_use), theirs = fast_exp2(m_other - m_use);
         float l = l_run * mine + l_other * theirs;
-        float inv = OPTIONS ? sink_factor(m_use, l, options.sinks, h) : 1.0f / l;
+        float inv = OPTIONS ? sink_factor(m_use, l, options, h) : 1.0f / l;
         mine *= inv;
         theirs *= inv;
-        bf16* dst = out + ((size_t)(tok0 + r) * heads + h) * HD;
+        bf16* dst = out + (OPTIONS ? (size_t)(tok0 + r) * options.out_stride + h * HD : ((size_t)(tok0 + r) * heads + h) * HD);
 #pragma unroll
         for (int c = 0; c < HD / 8; ++c) {
           uint4 w;

@@ -1,7 +1,7 @@
 // A mixture of gated feed-forward experts, token by token: every token goes to the `top` experts with the largest router
 // logits, weighted by the softmax over those logits only.
 //
-//   moe_route:  a block per token: logits = W_r x + b in float32 from the float32 stream, `top` rounds of arg-max (the
+//   moe_route:  a block per token (or four, in a step of many): logits = W_r x + b in float32 from the float32 stream, `top` rounds of arg-max (the
 //               lower expert on ties), then the weights.
 //               With `all_experts` the weights are instead the chosen experts' shares of the softmax over ALL experts'
 //               logits, as they are (they do not add up to one).
@@ -27,22 +27,6 @@ constexpr int MAX_TOP = 16;
 template <typename T> struct Vec;
 template <> struct Vec<float> { static constexpr int N = 4; };
 template <> struct Vec<__nv_bfloat16> { static constexpr int N = 8; };
-
-__device__ __forceinline__ float piece(const float* a, const float* b) {
-  float4 x = *(const float4*)a, y = *(const float4*)b;
-  return fmaf(x.w, y.w, fmaf(x.z, y.z, fmaf(x.y, y.y, x.x * y.x)));
-}
-// This lane's share of a . b over n values (the warp's shares add up to the dot product).
-template <typename T>
-__device__ __forceinline__ float lane_dot(const T* a, const T* b, int n, int lane) {
-  float s = 0.f;
-  if (n % Vec<T>::N == 0 && (((uintptr_t)a | (uintptr_t)b) & 15) == 0) {
-    for (int d = lane * Vec<T>::N; d < n; d += 32 * Vec<T>::N) s += piece(a + d, b + d);
-  } else {
-    for (int d = lane; d < n; d += 32) s = fmaf(to_float(a[d]), to_float(b[d]), s);
-  }
-  return s;
-}
 
 // This lane's shares of R dot products at once: rows w, w + stride, ... against the same b. The R rows' pieces are
 // asked for together (and b's piece once), so a warp keeps R loads in flight where one row after another keeps one.
@@ -73,35 +57,97 @@ __device__ __forceinline__ void lane_dots(const T* w, size_t stride, const T* b,
   }
 }
 
-// The router's weights are float32 whatever the activations are.
-template <typename X>
-__device__ __forceinline__ float lane_dot_router(const float* w, const X* x, int n, int lane) {
-  float s = 0.f;
-  for (int d = lane; d < n; d += 32) s = fmaf(w[d], to_float(x[d]), s);
-  return s;
+// Sixteen bytes of activations as float32.
+__device__ __forceinline__ void load_piece(const float* x, float* out) {
+  float4 v = *reinterpret_cast<const float4*>(x);
+  out[0] = v.x; out[1] = v.y; out[2] = v.z; out[3] = v.w;
 }
-template <>
-__device__ __forceinline__ float lane_dot_router<float>(const float* w, const float* x, int n, int lane) {
-  return lane_dot(w, x, n, lane);
+__device__ __forceinline__ void load_piece(const __nv_bfloat16* x, float* out) {
+  uint4 raw = *reinterpret_cast<const uint4*>(x);
+  const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    float2 f = __bfloat1622float2(p[i]);
+    out[2 * i] = f.x;
+    out[2 * i + 1] = f.y;
+  }
 }
 
-template <typename X>
+// logits[t][e] = w[e] . x[t] (+ bias[e]) for a block's tokens (TOKENS of them, `here` of which exist): the block's warps
+// share the experts out, two at a time, and a warp reads a piece of an expert's row once for all tokens. The router's
+// weights are float32 whatever the activations are. A token's sum does not depend on how many tokens the block has.
+template <int TOKENS, typename X>
+__device__ __forceinline__ void router_logits(float (*logits)[MAX_EXPERTS], const X* x, int here, int width,
+                                              const float* w, const float* bias, int experts, int warp, int lane) {
+  constexpr int N = Vec<X>::N, R = 2;
+  const bool pieces = width % N == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
+  for (int e0 = warp; e0 < experts; e0 += WARPS * R) {
+    float sum[R][TOKENS];
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+      for (int t = 0; t < TOKENS; ++t) sum[r][t] = 0.f;
+    const bool second = e0 + WARPS < experts;
+    const float* w0 = w + (size_t)e0 * width;
+    const float* w1 = second ? w0 + (size_t)WARPS * width : w0;
+    if (pieces) {
+#pragma unroll (TOKENS == 1 ? 4 : 1)
+      for (int d = lane * N; d < width; d += 32 * N) {
+        float wv[R][N], xv[N];
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+          load_piece(w0 + d + i, wv[0] + i);
+          load_piece(w1 + d + i, wv[1] + i);
+        }
+#pragma unroll
+        for (int t = 0; t < TOKENS; ++t) {
+          if (t >= here) break;
+          load_piece(x + (size_t)t * width + d, xv);
+#pragma unroll
+          for (int i = 0; i < N; ++i) {
+            sum[0][t] = fmaf(wv[0][i], xv[i], sum[0][t]);
+            sum[1][t] = fmaf(wv[1][i], xv[i], sum[1][t]);
+          }
+        }
+      }
+    } else {
+      for (int d = lane; d < width; d += 32)
+#pragma unroll
+        for (int t = 0; t < TOKENS; ++t) {
+          if (t >= here) break;
+          float xv = to_float(x[(size_t)t * width + d]);
+          sum[0][t] = fmaf(w0[d], xv, sum[0][t]);
+          sum[1][t] = fmaf(w1[d], xv, sum[1][t]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < TOKENS; ++t) {
+      float a = warp_sum(sum[0][t]), b = warp_sum(sum[1][t]);
+      if (lane == 0 && t < here) {
+        logits[t][e0] = a + (bias != nullptr ? bias[e0] : 0.f);
+        if (second) logits[t][e0 + WARPS] = b + (bias != nullptr ? bias[e0 + WARPS] : 0.f);
+      }
+    }
+  }
+}
+
+constexpr int ROUTE_TOKENS = 4;  // tokens a block takes in a step of many
+
+template <int TOKENS, typename X>
 __global__ void __launch_bounds__(WARPS * 32) moe_route_kernel(
     const X* __restrict__ x, int width, const float* __restrict__ w, const float* __restrict__ bias, int experts,
     int top, int tokens, int* __restrict__ chosen, float* __restrict__ weights, int all_experts) {
-  // a block per token: its warps share the experts' logits out, warp 0 then chooses
-  __shared__ float logits[MAX_EXPERTS];
+  // the block's warps share the experts' logits out, then warp i chooses for the block's token i
+  __shared__ float all_logits[TOKENS][MAX_EXPERTS];
   pdl_launch_dependents();
   pdl_wait();
   int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  int t = blockIdx.x;
-  const X* row = x + (size_t)t * width;
-  for (int e = warp; e < experts; e += WARPS) {
-    float s = warp_sum(lane_dot_router(w + (size_t)e * width, row, width, lane));
-    if (lane == 0) logits[e] = s + (bias != nullptr ? bias[e] : 0.f);
-  }
+  const int t0 = blockIdx.x * TOKENS, here = min(TOKENS, tokens - t0);
+  router_logits<TOKENS>(all_logits, x + (size_t)t0 * width, here, width, w, bias, experts, warp, lane);
   __syncthreads();
-  if (warp != 0) return;
+  if (warp >= here) return;
+  const int t = t0 + warp;
+  float* logits = all_logits[warp];
   float kept[MAX_TOP];
   float largest = 0.f, total = 0.f, everyone = 0.f;
   if (all_experts) {  // the softmax's denominator over every expert, before the chosen logits are struck out
@@ -141,25 +187,26 @@ __global__ void __launch_bounds__(WARPS * 32) moe_route_kernel(
 // The `top` experts of a token by sigmoid scores s: the choice is made by c = s + correction, among the experts of the
 // `keep` groups (of `group` neighbours each) whose two largest c add up to the most; a closed expert counts as minus
 // infinity. Weights: s over the chosen experts' sum (+ 1e-20), times `factor`. Lower experts and groups win ties.
-template <typename X>
+template <int TOKENS, typename X>
 __global__ void __launch_bounds__(WARPS * 32) moe_route_groups_kernel(
     const X* __restrict__ x, int width, const float* __restrict__ w, const float* __restrict__ correction, int experts,
     int group, int keep, float factor, int top, int tokens, int* __restrict__ chosen, float* __restrict__ weights) {
-  __shared__ float scores[MAX_EXPERTS], choice[MAX_EXPERTS], totals[MAX_EXPERTS];
+  __shared__ float all_scores[TOKENS][MAX_EXPERTS], all_choices[TOKENS][MAX_EXPERTS], all_totals[TOKENS][MAX_EXPERTS];
   pdl_launch_dependents();
   pdl_wait();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
-  const X* row = x + (size_t)t * width;
-  for (int e = warp; e < experts; e += WARPS) {
-    float z = warp_sum(lane_dot_router(w + (size_t)e * width, row, width, lane));
-    if (lane == 0) {
-      float s = 1.0f / (1.0f + expf(-z));
-      scores[e] = s;
-      choice[e] = s + (correction != nullptr ? correction[e] : 0.f);
-    }
-  }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = blockIdx.x * TOKENS, here = min(TOKENS, tokens - t0);
+  router_logits<TOKENS>(all_scores, x + (size_t)t0 * width, here, width, w, nullptr, experts, warp, lane);
   __syncthreads();
-  if (warp != 0) return;
+  if (warp >= here) return;
+  const int t = t0 + warp;
+  float *scores = all_scores[warp], *choice = all_choices[warp], *totals = all_totals[warp];
+  for (int e = lane; e < experts; e += 32) {
+    float s = 1.0f / (1.0f + expf(-scores[e]));
+    scores[e] = s;
+    choice[e] = s + (correction != nullptr ? correction[e] : 0.f);
+  }
+  __syncwarp();
   const int groups = experts / group;
   if (keep < groups) {
     for (int g = lane; g < groups; g += 32) {
@@ -332,13 +379,18 @@ DLLM_EXPORT int dllm_moe_route(const void* x, int width, const float* w, const f
   if (experts <= 0 || experts > MAX_EXPERTS || top <= 0 || top > MAX_TOP || top > experts || width <= 0)
     return DLLM_UNSUPPORTED_SIZE;
   if (x == nullptr || w == nullptr || chosen == nullptr || weights == nullptr) return DLLM_BAD_ARGUMENT;
-  dim3 grid(tokens), block(WARPS * 32);
+  const bool many = tokens >= 256;
+  const int per = many ? ROUTE_TOKENS : 1;
+  dim3 grid((tokens + per - 1) / per), block(WARPS * 32);
+  auto go = [&](auto kernel, auto* rows) {
+    return dllm_launch_pdl(kernel, grid, block, 0, stream, rows, width, w, bias, experts, top, tokens, chosen, weights,
+                           all_experts);
+  };
   if (dtype == DLLM_F32)
-    return dllm_launch_pdl(moe_route_kernel<float>, grid, block, 0, stream, (const float*)x, width, w, bias, experts,
-                           top, tokens, chosen, weights, all_experts);
+    return many ? go(moe_route_kernel<ROUTE_TOKENS, float>, (const float*)x) : go(moe_route_kernel<1, float>, (const float*)x);
   if (dtype == DLLM_BF16)
-    return dllm_launch_pdl(moe_route_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)x, width, w,
-                           bias, experts, top, tokens, chosen, weights, all_experts);
+    return many ? go(moe_route_kernel<ROUTE_TOKENS, __nv_bfloat16>, (const __nv_bfloat16*)x)
+                : go(moe_route_kernel<1, __nv_bfloat16>, (const __nv_bfloat16*)x);
   return DLLM_BAD_ARGUMENT;
 }
 
@@ -350,13 +402,19 @@ DLLM_EXPORT int dllm_moe_route_groups(const void* x, int width, const float* w, 
       experts % groups || keep <= 0 || keep > groups || top > keep * (experts / groups))
     return DLLM_UNSUPPORTED_SIZE;
   if (x == nullptr || w == nullptr || chosen == nullptr || weights == nullptr) return DLLM_BAD_ARGUMENT;
-  dim3 grid(tokens), block(WARPS * 32);
+  const bool many = tokens >= 256;
+  const int per = many ? ROUTE_TOKENS : 1;
+  dim3 grid((tokens + per - 1) / per), block(WARPS * 32);
+  auto go = [&](auto kernel, auto* rows) {
+    return dllm_launch_pdl(kernel, grid, block, 0, stream, rows, width, w, correction, experts, experts / groups, keep,
+                           factor, top, tokens, chosen, weights);
+  };
   if (dtype == DLLM_F32)
-    return dllm_launch_pdl(moe_route_groups_kernel<float>, grid, block, 0, stream, (const float*)x, width, w, correction,
-                           experts, experts / groups, keep, factor, top, tokens, chosen, weights);
+    return many ? go(moe_route_groups_kernel<ROUTE_TOKENS, float>, (const float*)x)
+                : go(moe_route_groups_kernel<1, float>, (const float*)x);
   if (dtype == DLLM_BF16)
-    return dllm_launch_pdl(moe_route_groups_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)x, width,
-                           w, correction, experts, experts / groups, keep, factor, top, tokens, chosen, weights);
+    return many ? go(moe_route_groups_kernel<ROUTE_TOKENS, __nv_bfloat16>, (const __nv_bfloat16*)x)
+                : go(moe_route_groups_kernel<1, __nv_bfloat16>, (const __nv_bfloat16*)x);
   return DLLM_BAD_ARGUMENT;
 }
 

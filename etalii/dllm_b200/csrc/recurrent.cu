@@ -937,6 +937,77 @@ __global__ void __launch_bounds__(256) state_space_prepare_kernel(StateSpacePrep
   prepared[i] = silu_exact(sum);
 }
 
+// The same for steps of many tokens whose sizes are multiples of four: a thread owns four channels of PREPARE_TILE
+// consecutive tokens, so an input is read once for all its taps. The sums run in the order of the kernel above. The last
+// blocks along y make the decays and step sizes.
+constexpr int PREPARE_TILE = 8;
+
+template <int TAPS>
+__global__ void __launch_bounds__(128) state_space_prepare_tile_kernel(StateSpacePrepareArgs a, int tokens) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * PREPARE_TILE, here = min(PREPARE_TILE, tokens - t0);
+  const int inner = a.heads * a.vdim, channels = inner + 2 * a.groups * a.dim;
+  constexpr int HISTORY = TAPS - 1;
+  const int channel_blocks = (channels / 4 + 127) / 128;
+  if ((int)blockIdx.y >= channel_blocks) {
+    const int i = (blockIdx.y - channel_blocks) * 128 + threadIdx.x;
+    if (i >= here * a.heads) return;
+    const int t = t0 + i / a.heads, h = i % a.heads;
+    const float dt = softplus(a.proj[(size_t)t * a.stride + inner + channels + h] + a.dt_bias[h]);
+    float* aux = a.aux + (size_t)t * 2 * a.heads;
+    aux[h] = expf(-expf(a.a_log[h]) * dt);
+    aux[a.heads + h] = dt;
+    return;
+  }
+  const int ch = 4 * (blockIdx.y * 128 + threadIdx.x);
+  if (ch >= channels) return;
+  const float* rows = a.proj + inner + ch;
+  float4 now[PREPARE_TILE];
+#pragma unroll
+  for (int i = 0; i < PREPARE_TILE; ++i)
+    now[i] = *reinterpret_cast<const float4*>(rows + (size_t)(t0 + min(i, here - 1)) * a.stride);
+  float tap[4 * TAPS];  // channel c's tap j at c TAPS + j
+#pragma unroll
+  for (int i = 0; i < TAPS; ++i) {
+    float4 v = *reinterpret_cast<const float4*>(a.taps + (size_t)ch * TAPS + 4 * i);
+    tap[4 * i] = v.x; tap[4 * i + 1] = v.y; tap[4 * i + 2] = v.z; tap[4 * i + 3] = v.w;
+  }
+  const float4 bias = a.bias != nullptr ? *reinterpret_cast<const float4*>(a.bias + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 past[HISTORY > 0 ? HISTORY : 1];
+  int seq_before = -1;
+#pragma unroll
+  for (int i = 0; i < PREPARE_TILE; ++i) {
+    if (i >= here) break;
+    const int t = t0 + i, seq = a.tok_seq[t];
+    if (HISTORY > 0 && seq != seq_before) {  // the tile's first token, or another sequence's
+      seq_before = seq;
+      const int local = t - a.cu_seqlens[seq];
+      const float* kept = a.conv_state + (size_t)a.slots[seq] * HISTORY * channels + ch;
+#pragma unroll
+      for (int j = 0; j < HISTORY; ++j) {
+        const int back = HISTORY - j;
+        past[j] = *reinterpret_cast<const float4*>(back <= local ? rows + (size_t)(t - back) * a.stride
+                                                                 : kept + (size_t)(HISTORY - (back - local)) * channels);
+      }
+    }
+    float4 sum = bias;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const float4 x = j < HISTORY ? past[j < HISTORY ? j : 0] : now[i];
+      sum.x = fmaf(tap[j], x.x, sum.x);
+      sum.y = fmaf(tap[TAPS + j], x.y, sum.y);
+      sum.z = fmaf(tap[2 * TAPS + j], x.z, sum.z);
+      sum.w = fmaf(tap[3 * TAPS + j], x.w, sum.w);
+    }
+    *reinterpret_cast<float4*>(a.prepared + (size_t)t * channels + ch) =
+        make_float4(silu_exact(sum.x), silu_exact(sum.y), silu_exact(sum.z), silu_exact(sum.w));
+#pragma unroll
+    for (int j = 0; j + 1 < HISTORY; ++j) past[j] = past[j + 1];
+    if (HISTORY > 0) past[HISTORY > 0 ? HISTORY - 1 : 0] = now[i];
+  }
+}
+
 // The convolution's history after a step of any lengths: a thread owns a channel and reads all it needs before it writes.
 __global__ void __launch_bounds__(256) state_space_history_kernel(StateSpacePrepareArgs a) {
   pdl_launch_dependents();
@@ -974,21 +1045,31 @@ DLLM_EXPORT int dllm_state_space_prepare(const float* proj, int stride, const fl
     return DLLM_BAD_ARGUMENT;
   StateSpacePrepareArgs a = {proj, stride, taps, bias, n_taps, a_log, dt_bias, conv_state, tok_seq, cu_seqlens, slots,
                              heads, groups, dim, padded, vdim, prepared, aux, single};
-  int places = heads * vdim + 2 * groups * padded + heads;
-  int status = dllm_launch_pdl(state_space_prepare_kernel, dim3(tokens, (places + 255) / 256), dim3(256), 0, stream, a);
+  int places = heads * vdim + 2 * groups * padded + heads, channels = heads * vdim + 2 * groups * dim, status;
+  const bool fours = !single && tokens >= 64 && dim % 4 == 0 && heads * vdim % 4 == 0 && stride % 4 == 0 && n_taps <= 4 &&
+                     (((uintptr_t)proj | (uintptr_t)taps | (uintptr_t)bias | (uintptr_t)conv_state | (uintptr_t)prepared) & 15) == 0;
+  if (fours) {
+    dim3 grid((tokens + PREPARE_TILE - 1) / PREPARE_TILE,
+              (channels / 4 + 127) / 128 + (PREPARE_TILE * heads + 127) / 128);
+    auto go = [&](auto kernel) { return dllm_launch_pdl(kernel, grid, dim3(128), 0, stream, a, tokens); };
+    status = n_taps == 1 ? go(state_space_prepare_tile_kernel<1>)
+             : n_taps == 2 ? go(state_space_prepare_tile_kernel<2>)
+             : n_taps == 3 ? go(state_space_prepare_tile_kernel<3>) : go(state_space_prepare_tile_kernel<4>);
+  } else {
+    status = dllm_launch_pdl(state_space_prepare_kernel, dim3(tokens, (places + 255) / 256), dim3(256), 0, stream, a);
+  }
   if (status != DLLM_OK || single || n_taps == 1) return status;
-  int channels = heads * vdim + 2 * groups * dim;
   return dllm_launch_pdl(state_space_history_kernel, dim3(sequences, (channels + 255) / 256), dim3(256), 0, stream, a);
 }
 
 // y [tokens, width] float32 times silu(z) (z the first `width` values of rows of `z_stride` floats), divided by its root mean
 // square in `parts` equal parts of the row (each by its own), times weight [width]; rounded once to the output type. Output
-// rows have `out_stride` values, up to 31 more than `width`, and zeros behind it. A block per token and part, whose gated
+// rows have `out_stride` values, `fill` (up to 31) zeros behind the `width`. A block per token and part, whose gated
 // values wait in shared memory for their sum of squares.
 template <typename T>
 __global__ void gate_norm_kernel(T* __restrict__ out, const float* __restrict__ y, const float* __restrict__ z,
                                  int z_stride, const float* __restrict__ weight, int width, int part, float eps,
-                                 int out_stride) {
+                                 int out_stride, int fill) {
   extern __shared__ __align__(16) float stage[];  // [part]
   __shared__ float scratch[32];
   pdl_launch_dependents();
@@ -1009,23 +1090,24 @@ __global__ void gate_norm_kernel(T* __restrict__ out, const float* __restrict__ 
   const float inv = 1.0f / sqrtf(warp_sum(total) / (float)part + eps);
   T* dst = out + (size_t)t * out_stride;
   for (int i = threadIdx.x; i < part; i += blockDim.x) dst[at + i] = from_float<T>(stage[i] * inv * weight[at + i]);
-  if (at + part == width && width + threadIdx.x < out_stride) dst[width + threadIdx.x] = from_float<T>(0.f);
+  if (at + part == width && (int)threadIdx.x < fill) dst[width + threadIdx.x] = from_float<T>(0.f);
 }
 
 DLLM_EXPORT int dllm_gate_norm(void* out, const float* y, const float* z, int z_stride, const float* weight, int tokens,
-                               int width, int parts, float eps, int out_stride, int out_dtype, cudaStream_t stream) {
+                               int width, int parts, float eps, int out_stride, int fill, int out_dtype,
+                               cudaStream_t stream) {
   if (tokens <= 0) return DLLM_OK;
   if (width <= 0 || parts <= 0 || width % parts || parts > 65535 || width / parts > 12000 || z_stride < width ||
-      out_stride < width || out_stride > width + 31)
+      fill < 0 || fill > 31 || out_stride < width + fill)
     return DLLM_UNSUPPORTED_SIZE;
   if (!out || !y || !z || !weight) return DLLM_BAD_ARGUMENT;
   const int part = width / parts, threads = part >= 2048 ? 512 : (part >= 512 ? 256 : (part >= 128 ? 128 : 64));
   if (out_dtype == DLLM_F32)
     return dllm_launch_pdl(gate_norm_kernel<float>, dim3(tokens, parts), dim3(threads), part * sizeof(float), stream,
-                           (float*)out, y, z, z_stride, weight, width, part, eps, out_stride);
+                           (float*)out, y, z, z_stride, weight, width, part, eps, out_stride, fill);
   if (out_dtype == DLLM_BF16)
     return dllm_launch_pdl(gate_norm_kernel<__nv_bfloat16>, dim3(tokens, parts), dim3(threads), part * sizeof(float),
-                           stream, (__nv_bfloat16*)out, y, z, z_stride, weight, width, part, eps, out_stride);
+                           stream, (__nv_bfloat16*)out, y, z, z_stride, weight, width, part, eps, out_stride, fill);
   return DLLM_BAD_ARGUMENT;
 }
 

@@ -1,5 +1,6 @@
 // What a softmax attention may have besides a scale and a window: a cap on the scores, a sink per head, first positions
-// that stay visible, chunks, values of another size than the keys, and longer output rows. The attention kernels take it as an
+// that stay visible, chunks, values of another size than the keys, a factor of
+// the output, and longer output rows. The attention kernels take it as an
 // argument that their plain instantiations ignore (OPTIONS = false) and that others read (OPTIONS = true).
 #pragma once
 #include "wide_kv.cuh"
@@ -11,6 +12,7 @@ struct ScoreOptions {
   int value_dim;
   int out_stride;      // elements of an output row
   int chunk;           // 0, or: a token sees the positions of its own chunk of this many only
+  float out_scale;     // what the outputs are multiplied by before they are rounded
 };
 
 constexpr float SCORE_LOG2E = 1.4426950408889634f;
@@ -57,10 +59,10 @@ struct ScoreCap {
 };
 
 // The last step of a softmax's sum under a sink: with the running maximum m (log2 units) and sum l, the factor that the
-// running weighted sum of values is multiplied by.
-__device__ __forceinline__ float sink_factor(float m, float l, const float* sinks, int head) {
-  if (sinks == nullptr) return 1.0f / l;
-  float sink = sinks[head] * SCORE_LOG2E, top = fmaxf(m, sink);
+// running weighted sum of values is multiplied by (the output's own factor in it).
+__device__ __forceinline__ float sink_factor(float m, float l, const ScoreOptions& options, int head) {
+  if (options.sinks == nullptr) return options.out_scale / l;
+  float sink = options.sinks[head] * SCORE_LOG2E, top = fmaxf(m, sink);
   float f = fast_exp2(m - top);
-  return f / fmaf(l, f, fast_exp2(sink - top));
+  return f * options.out_scale / fmaf(l, f, fast_exp2(sink - top));
 }

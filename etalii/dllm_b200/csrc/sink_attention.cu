@@ -20,15 +20,15 @@ constexpr int PLACES = MAX_DIM / 32;  // value places a lane owns
 
 struct SinkArgs {
   const void* q;       // [tokens, heads * dim] in the cache's type
-  void* out;           // [tokens, out_stride] in the cache's type; zeros behind heads * vdim
+  void* out;           // [tokens, out_stride] in the cache's type; `fill` zeros behind heads * vdim
   int out_stride;
   WideKv cache;
   const float* sinks;  // [heads] or null
   const int* tok_seq;
   const int* tok_pos;
   const int* slots;
-  int tokens, heads, window, keep, chunk;
-  float scale, cap;
+  int tokens, heads, fill, window, keep, chunk;
+  float scale, cap, out_scale;
 };
 
 __device__ __forceinline__ float dot_piece(const float* q, const float* k) {
@@ -105,13 +105,13 @@ __device__ __forceinline__ void finish(Running& r, const SinkArgs& a, int t, int
     factor = expf(r.m - m);
     r.l = r.l * factor + expf(sink - m);
   }
-  factor /= r.l;
+  factor *= a.out_scale / r.l;
   T* row = (T*)a.out + (size_t)t * a.out_stride;
 #pragma unroll
   for (int i = 0; i < PLACES; ++i)
     if (lane + 32 * i < vdim) row[(size_t)h * vdim + lane + 32 * i] = from_float<T>(r.acc[i] * factor);
   if (h == a.heads - 1)
-    for (int i = a.heads * vdim + lane; i < a.out_stride; i += 32) row[i] = from_float<T>(0.f);
+    for (int i = lane; i < a.fill; i += 32) row[a.heads * vdim + i] = from_float<T>(0.f);
 }
 
 template <typename T>
@@ -187,20 +187,21 @@ int launch(const SinkArgs& a, int split, cudaStream_t stream) {
 }  // namespace
 
 // q [tokens, heads * dim] and out [tokens, out_stride] in the cache's type; sinks [heads] float32 or null; window 0 and
-// chunk 0: all positions; cap 0: scores as they are. `split` != 0: a block of sixteen warps per (token, head) instead of a warp.
+// chunk 0: all positions; cap 0: scores as they are; the outputs are multiplied by out_scale, `fill` zeros
+// follow a row's. `split` != 0: a block of sixteen warps per (token, head) instead of a warp.
 DLLM_EXPORT int dllm_sink_attention(const void* q, void* out, int out_stride, void* cache_base, const int* page_table,
                                     int max_pages, int page_size, int heads, int kv_heads, int dim, int vdim,
                                     const float* sinks, const int* tok_seq, const int* tok_pos, const int* slots,
-                                    int tokens, float scale, float cap, int window, int keep, int chunk, int split,
-                                    int dtype,
-                                    cudaStream_t stream) {
+                                    int tokens, float scale, float cap, int window, int keep, int chunk, float out_scale,
+                                    int fill, int split, int dtype, cudaStream_t stream) {
   if (tokens <= 0) return DLLM_OK;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || dim > MAX_DIM || vdim <= 0 || vdim > MAX_DIM ||
-      page_size <= 0 || page_size % TILE || window < 0 || keep < 0 || chunk < 0 || out_stride < heads * vdim)
+      page_size <= 0 || page_size % TILE || window < 0 || keep < 0 || chunk < 0 || fill < 0 ||
+      out_stride < heads * vdim + fill)
     return DLLM_UNSUPPORTED_SIZE;
   if (!q || !out || !cache_base || !page_table || !tok_seq || !tok_pos || !slots) return DLLM_BAD_ARGUMENT;
   SinkArgs a = {q, out, out_stride, {cache_base, page_table, max_pages, page_size, kv_heads, dim, vdim}, sinks, tok_seq,
-                tok_pos, slots, tokens, heads, window, keep, chunk, scale, cap};
+                tok_pos, slots, tokens, heads, fill, window, keep, chunk, scale, cap, out_scale};
   if (dtype == DLLM_F32) return launch<float>(a, split, stream);
   if (dtype == DLLM_BF16) return launch<__nv_bfloat16>(a, split, stream);
   return DLLM_BAD_ARGUMENT;

@@ -60,17 +60,19 @@ _prototypes = {
                                                     c_void_p],
     ("sink_attention", "dllm_sink_attention"): [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                                c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                                c_float, c_float, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
+                                                c_void_p],
     ("sink_attention_prefill", "dllm_sink_attention_prefill"): [
         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
+        c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_float,
+        c_void_p],
     ("sink_attention_decode", "dllm_sink_attention_decode"): [
         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-        c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
     ("sink_attention_tcgen05", "dllm_sink_attention_tcgen05"): [
-        c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p,
-        c_void_p],
+        c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
+        c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_int, c_int, c_float,
+        c_void_p, c_void_p],
     ("qkv_prepare", "dllm_qkv_prepare"): [
         c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
         c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
@@ -87,7 +89,7 @@ _prototypes = {
                                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                 c_int, c_void_p, c_void_p, c_int, c_void_p],
     ("recurrent", "dllm_gate_norm"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int,
-                                      c_int, c_void_p],
+                                      c_int, c_int, c_void_p],
     ("moe", "dllm_moe_route_groups"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int,
                                        c_void_p, c_void_p, c_int, c_void_p],
     ("elementwise", "dllm_norm_sum_residual"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
@@ -633,25 +635,29 @@ def sigmoid_attention_tiled(out: torch.Tensor, q: torch.Tensor, cache, heads: in
 
 def sink_attention(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
                    sinks: torch.Tensor | None, window: int, keep: int, batch, split: bool | None = None,
-                   chunk: int = 0) -> None:
+                   chunk: int = 0, out_scale: float = 1.0, out_at: int | None = None) -> None:
     """Softmax attention of every token over its own sequence's cache: scores q . k * scale, then softcap * tanh(score /
     softcap) if softcap > 0, of the keys j <= i with i - j < window (0: all), or with `chunk` those of the token's own chunk of that many positions, or j < keep; the
     denominator also holds
     exp(sinks[h]) where `sinks` float32 [heads] is given. q [tokens, heads x dim] and out [tokens, heads x value_dim, or
-    longer rows: zeros behind] in the cache's type. The general kernel: float32 arithmetic, every size up to 256.
+    longer rows: zeros behind; or with `out_at` a stretch of longer rows from that column on] in the cache's type; the
+    outputs count `out_scale` times. The general kernel: float32 arithmetic, every size up to 256.
     `split`: a block of sixteen warps per (token, head) instead of a warp (default: for steps of few tokens)."""
     _cuda(out, q, sinks)
     dim, vdim, tokens = cache.head_dim, cache.value_dim, batch.n_tokens
     assert q.dtype == cache.dtype and out.dtype == cache.dtype and not cache.keys_only
-    assert q.shape[1] == heads * dim and out.shape[1] >= heads * vdim
+    at = int(out_at or 0)
+    fill = out.shape[1] - heads * vdim if out_at is None else 0
+    assert q.shape[1] == heads * dim and out.shape[1] >= at + heads * vdim
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
     if split is None:
         split = tokens * heads <= 4 * _multiprocessors()
     _check(_fn("sink_attention", "dllm_sink_attention")(
-        q.data_ptr(), out.data_ptr(), out.shape[1], cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
-        cache.page_size, heads, cache.kv_heads, dim, vdim, sinks.data_ptr() if sinks is not None else None,
+        q.data_ptr(), out.data_ptr() + at * out.element_size(), out.shape[1], cache.base_ptr,
+        cache.page_table.data_ptr(), cache.max_pages, cache.page_size, heads, cache.kv_heads, dim, vdim, sinks.data_ptr() if sinks is not None else None,
         batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.slots.data_ptr(), tokens, float(scale),
-        float(softcap or 0.0), int(window or 0), int(keep or 0), int(chunk or 0), 1 if split else 0, _code(cache.dtype), _stream()),
+        float(softcap or 0.0), int(window or 0), int(keep or 0), int(chunk or 0), float(out_scale), fill,
+        1 if split else 0, _code(cache.dtype), _stream()),
         "sink_attention", lambda: f"dim={dim}, value_dim={vdim} (at most 256)")
 
 
@@ -661,21 +667,24 @@ def sink_attention_tiles(dtype, dim: int, vdim: int, page_size: int = 64) -> boo
 
 
 def sink_attention_prefill(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
-                           sinks: torch.Tensor | None, window: int, keep: int, batch, chunk: int = 0) -> None:
+                           sinks: torch.Tensor | None, window: int, keep: int, batch, chunk: int = 0,
+                           out_scale: float = 1.0, out_at: int | None = None) -> None:
     """`sink_attention` for portions of prompts (bfloat16, mma.sync, tiles of 64 queries; sizes:
     `sink_attention_tiles`)."""
     _cuda(out, q, sinks)
     dim, vdim = cache.head_dim, cache.value_dim
     assert sink_attention_tiles(cache.dtype, dim, vdim, cache.page_size) and not cache.keys_only
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
-    assert q.shape[1] == heads * dim and out.shape[1] == heads * vdim
+    at = int(out_at or 0)
+    assert q.shape[1] == heads * dim and out.shape[1] >= at + heads * vdim
+    assert out_at is not None or out.shape[1] == heads * vdim
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
     _check(_fn("sink_attention_prefill", "dllm_sink_attention_prefill")(
-        out.data_ptr(), out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
-        cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(),
+        out.data_ptr() + 2 * at, out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(),
+        cache.max_pages, cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(),
         batch.cu_seqlens.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), batch.n_tiles, float(scale),
         float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0),
-        int(chunk or 0), _stream()), "sink_attention_prefill")
+        int(chunk or 0), float(out_scale), _stream()), "sink_attention_prefill")
 
 
 def sink_attention_tcgen05_supported(cache) -> bool:
@@ -683,39 +692,45 @@ def sink_attention_tcgen05_supported(cache) -> bool:
 
 
 def sink_attention_tcgen05(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
-                           sinks: torch.Tensor | None, window: int, keep: int, batch, chunk: int = 0) -> None:
+                           sinks: torch.Tensor | None, window: int, keep: int, batch, chunk: int = 0,
+                           out_scale: float = 1.0, out_at: int | None = None) -> None:
     """`sink_attention` for portions of prompts on the 5th-generation tensor cores (bfloat16, keys and values of 64 or
     128 values)."""
     _cuda(out, q, sinks)
     assert sink_attention_tcgen05_supported(cache) and not cache.keys_only
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
-    assert q.shape[1] == heads * cache.head_dim and out.shape[1] == q.shape[1]
+    at = int(out_at or 0)
+    assert q.shape[1] == heads * cache.head_dim and out.shape[1] >= at + q.shape[1] and at % 8 == 0
+    assert out_at is not None or out.shape[1] == q.shape[1]
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
     _check(_fn("sink_attention_tcgen05", "dllm_sink_attention_tcgen05")(
-        out.data_ptr(), q.data_ptr(), batch.n_tokens, cache.base_ptr, cache.storage.shape[0],
+        out.data_ptr() + 2 * at, out.shape[1], q.data_ptr(), batch.n_tokens, cache.base_ptr, cache.storage.shape[0],
         cache.page_table.data_ptr(), cache.max_pages, cache.page_size, heads, cache.kv_heads, cache.head_dim,
         batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(), batch.cu_seqlens.data_ptr(), batch.start.data_ptr(),
         batch.slots.data_ptr(), batch.n_tiles, float(scale), float(softcap or 0.0),
         sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0), int(chunk or 0),
-        _status_word().data_ptr(), _stream()), "sink_attention_tcgen05")
+        float(out_scale), _status_word().data_ptr(), _stream()), "sink_attention_tcgen05")
 
 
 def sink_attention_decode(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
                           sinks: torch.Tensor | None, window: int, keep: int, batch, shape: int = -1,
-                          chunk: int = 0) -> None:
+                          chunk: int = 0, out_scale: float = 1.0, out_at: int | None = None) -> None:
     """`sink_attention` for a step of single tokens (bfloat16; sizes: `sink_attention_tiles`): the keys of a (sequence,
     kv head) dealt to the blocks of a cluster; `shape` as for `attention_decode_cluster`."""
     _cuda(out, q, sinks)
     dim, vdim = cache.head_dim, cache.value_dim
     assert sink_attention_tiles(cache.dtype, dim, vdim, cache.page_size) and not cache.keys_only
     assert batch.n_tokens == batch.n_seqs and q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
-    assert q.shape[1] == heads * dim and out.shape[1] == heads * vdim
+    at = int(out_at or 0)
+    assert q.shape[1] == heads * dim and out.shape[1] >= at + heads * vdim
+    assert out_at is not None or out.shape[1] == heads * vdim
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
     _check(_fn("sink_attention_decode", "dllm_sink_attention_decode")(
-        out.data_ptr(), out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(), cache.max_pages,
-        cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tok_pos.data_ptr(), batch.slots.data_ptr(),
+        out.data_ptr() + 2 * at, out.shape[1], q.data_ptr(), cache.base_ptr, cache.page_table.data_ptr(),
+        cache.max_pages, cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tok_pos.data_ptr(), batch.slots.data_ptr(),
         batch.n_seqs, float(scale), float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None,
-        int(window or 0), int(keep or 0), int(chunk or 0), int(shape), _stream()), "sink_attention_decode")
+        int(window or 0), int(keep or 0), int(chunk or 0), float(out_scale), int(shape), _stream()),
+        "sink_attention_decode")
 
 
 def glu_clamped_fuses(rows: int, outputs: int, inner: int) -> bool:
@@ -1481,16 +1496,19 @@ def state_space_scan(out: torch.Tensor, prepared: torch.Tensor, aux: torch.Tenso
 
 
 def gate_norm(out: torch.Tensor, y: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, parts: int,
-              eps: float) -> None:
+              eps: float, out_at: int | None = None, fill: int | None = None) -> None:
     """out = v / rms(v over each of `parts` equal parts of the row) * weight with v = y * silu(z), z the first values of
-    `rows` float32. y float32 [tokens, width]; out may have up to 31 columns more, which get zeros."""
+    `rows` float32. y float32 [tokens, width]; out may have up to 31 columns more, which get zeros; or
+    with `out_at` the result is a stretch of its longer rows from that column on, with `fill` zeros behind."""
     _cuda(out, y, rows, weight)
     tokens, width = y.shape
     assert y.dtype == rows.dtype == weight.dtype == torch.float32 and weight.numel() == width
-    assert out.shape[0] == tokens and rows.shape[0] >= tokens
+    at = int(out_at or 0)
+    fill = int(fill or 0) if out_at is not None else out.shape[1] - width
+    assert out.shape[0] == tokens and rows.shape[0] >= tokens and out.shape[1] >= at + width + fill
     _check(_fn("recurrent", "dllm_gate_norm")(
-        out.data_ptr(), y.data_ptr(), rows.data_ptr(), rows.shape[1], weight.data_ptr(), tokens, width, int(parts),
-        float(eps), out.shape[1], _code(out.dtype), _stream()), "gate_norm",
+        out.data_ptr() + at * out.element_size(), y.data_ptr(), rows.data_ptr(), rows.shape[1], weight.data_ptr(), tokens, width, int(parts),
+        float(eps), out.shape[1], fill, _code(out.dtype), _stream()), "gate_norm",
         lambda: f"width={width} in {parts} parts (of at most 12,000 values)")
 
 

@@ -51,6 +51,7 @@ class Attention:
         self.window = int(window) if window else None
         self.position = build_part("position", position) if position is not None else None
         self.w_qkv = self.w_o = None
+        self.output_scale = 1.0
 
     @staticmethod
     def parameters(hidden_size, num_heads, num_kv_heads, head_dim, values="projected", **_) -> dict[str, ParamSpec]:
@@ -107,10 +108,11 @@ class Attention:
         return True
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, cache, rt, write_cache: bool = True,
-                epilogue: int = ops.EPI_RESIDUAL) -> None:
+                epilogue: int = ops.EPI_RESIDUAL, operand=None) -> None:
         """h: normed activations [tokens, hidden]; adds the attention output to `residual` (float32) in place. A
         mixer that runs this one as a branch passes `epilogue=ops.EPI_STORE_F32`: `residual` is then its buffer for
-        the branch's output and is overwritten."""
+        the branch's output and is overwritten. One that has taken the output matrix (`give_output_matrix`) passes
+        `operand` = (rows, column): what that matrix multiplies goes there."""
         n = batch.n_tokens
         q_size = self.num_heads * self.head_dim
         q = rt.ws.buffer("q", (n, q_size), rt.dtype)
@@ -144,6 +146,15 @@ class Attention:
             qkv = rt.ws.buffer("qkv", (n, q_size + 2 * self.num_kv_heads * self.head_dim), torch.float32)
             project(qkv, h, self.w_qkv, ops.EPI_STORE_F32)
             ops.rope_cache_write(qkv, q, cache, table, rotary_dim, self.num_heads, batch, write_cache)
+        if operand is not None:
+            attended, at = operand
+            attend = ops.sink_attention_decode
+            if not batch.is_decode:
+                attend = ops.sink_attention_tcgen05 if ops.attention_prefill_tcgen05_supported(cache) and \
+                    batch.max_context > TCGEN05_ATTENTION_FROM.get(self.head_dim, 512) else ops.sink_attention_prefill
+            attend(attended, q, cache, self.num_heads, self.scale, 0.0, None, self.window or 0, 0, batch,
+                   out_scale=self.output_scale, out_at=at)
+            return
         attended = rt.ws.buffer("attended", (n, q_size), rt.dtype)
         if batch.is_decode and rt.dtype == torch.bfloat16 and ops.attention_decode_cluster_supported(cache):
             ops.attention_decode_cluster(attended, q, cache, self.num_heads, self.scale, self.window or 0, batch)
@@ -166,6 +177,14 @@ class Attention:
             ops.attention_general(attended, q, cache, self.num_heads, self.scale, self.window or 0, batch)
         ops.gemm(residual, attended, self.w_o, epilogue)
 
+    def give_output_matrix(self, rt, scale: float) -> torch.Tensor | None:
+        """The output matrix, for a mixer that multiplies several branches' operands by theirs in one product (None: the
+        kernels that can write into longer rows do not run these sizes). From then on the operand counts `scale` times and
+        goes where `forward` is told."""
+        if not ops.sink_attention_tiles(rt.dtype, self.head_dim, self.head_dim):
+            return None
+        w, self.w_o, self.output_scale = self.w_o, None, float(scale)
+        return w
 
     def kernel_libraries(self, rt) -> set[str]:
         """The kernel libraries this part's steps call (built together when the model loads)."""
@@ -173,8 +192,11 @@ class Attention:
             return {"gemm_simt", "elementwise", "attention"}
         hd = self.head_dim
         names = {"gemv", "gemm_tcgen05", "elementwise"}
-        if any(ops.splits_over_clusters(64, w.shape[0], w.shape[1]) for w in (self.w_qkv, self.w_o)):
+        if any(ops.splits_over_clusters(64, w.shape[0], w.shape[1]) for w in (self.w_qkv, self.w_o) if w is not None):
             names.add("gemv_cluster")  # (steps of 17 to 64 tokens with weights this small)
+        if self.w_o is None:  # (given away)
+            names |= {"sink_attention_decode", "sink_attention_prefill"}
+            return names | ({"sink_attention_tcgen05"} if hd in TCGEN05_ATTENTION_FROM else set())
         names.add("attention_decode_cluster" if hd % 16 == 0 and hd <= 128 else "attention_decode")
         if hd in (64, 128):
             names.add("attention_prefill_tcgen05")  # (long prompts; short ones take the mma.sync kernel)

@@ -355,7 +355,7 @@ class StateSpaceDuality:
     softplus(dt + dt_bias) and head h reading group h // (heads / groups): S <- exp(-exp(A_log) b) S + b B x^T, y = S^T C +
     D x. The concatenated y is multiplied by silu(z), divided by its root mean square in `norm_groups` equal parts of the
     row, multiplied by a weight [heads x vdim] and projected by W_o. Besides S the convolution's last conv - 1 inputs are
-    state. `take_output_scale`: a factor of the whole output, which goes into the norm's float32 weight."""
+    state. A factor of the whole output (`give_output_matrix`) goes into the norm's float32 weight."""
 
     def __init__(self, hidden_size: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_groups: int,
                  eps: float) -> None:
@@ -409,12 +409,17 @@ class StateSpaceDuality:
         self.skip = rt.to_device(tensors["D"], torch.float32)
         self.weight = rt.to_device(tensors["norm"], torch.float32)
 
-    def take_output_scale(self, scale: float) -> bool:
+    def give_output_matrix(self, rt, scale: float) -> torch.Tensor | None:
+        """The output matrix, for a mixer that multiplies several branches' operands by theirs in one product. From then on
+        the operand counts `scale` times and goes where `forward` is told."""
+        w, self.w_o = self.w_o, None
         self.weight = self.weight * float(scale)
-        return True
+        return w
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, state, rt, write_cache: bool = True,
-                epilogue: int = ops.EPI_RESIDUAL) -> None:
+                epilogue: int = ops.EPI_RESIDUAL, operand=None) -> None:
+        """Adds the output to `residual` (float32), or with `epilogue=ops.EPI_STORE_F32` writes it there, or with `operand` =
+        (rows, column) leaves what the output matrix multiplies there."""
         n = batch.n_tokens
         matrix, history = (state, None) if self.conv == 1 else state
         rows = rt.ws.buffer("mixer_rows", (n, self.w_in.shape[0]), torch.float32)
@@ -426,6 +431,10 @@ class StateSpaceDuality:
         read = rt.ws.buffer("mixer_read", (n, self.inner), torch.float32)
         ops.state_space_scan(read, prepared, aux, self.skip, self.heads, self.groups, self.padded, self.vdim, matrix,
                              batch)
+        if operand is not None:
+            ops.gate_norm(operand[0], read, rows, self.weight, self.norm_groups, self.eps, out_at=operand[1],
+                          fill=_in_pieces(self.inner) - self.inner)
+            return
         gated = rt.ws.buffer("mixer_gated", (n, self.w_o.shape[1]), rt.dtype)
         ops.gate_norm(gated, read, rows, self.weight, self.norm_groups, self.eps)
         ops.gemm(residual, gated, self.w_o, epilogue)

@@ -1,7 +1,8 @@
 """Two mixers side by side on the same input. With norms: out = factor * (rms(left(h)) * w_left + rms(right(h)) *
 w_right), each branch's output divided by its root mean square over the model width and multiplied by a weight of its own
 before the sum goes into the residual stream. Without: out = scales[0] * left(h) + scales[1] * right(h). The sums are
-float32. Either branch is any registered mixer that can write its output to a buffer instead of adding it to the stream
+float32, and where both branches can give their output matrix away (`give_output_matrix(rt, scale)`) the sum is one product:
+their operands lie side by side in one row, with the scales in them. Either branch is any registered mixer that can write its output to a buffer instead of adding it to the stream
 (`forward(..., epilogue=ops.EPI_STORE_F32)`); each keeps its own cache entry (keys and values, a state, or several)."""
 from __future__ import annotations
 
@@ -23,6 +24,9 @@ class ParallelMixer:
         self.hidden_size, self.eps, self.factor = int(hidden_size), float(eps), float(factor)
         self.branches = [build_part("mixer", left), build_part("mixer", right)]
         self.weights: list = [None, None]
+        self.w_out = None
+        """Both branches' output matrices side by side, where they gave them away."""
+        self.columns = (0, 0)
         needs = [b.cache_need() if hasattr(b, "cache_need") else None for b in self.branches]
         self._needs = needs
 
@@ -56,9 +60,31 @@ class ParallelMixer:
             if self.scales is None:
                 self.weights[index] = rt.to_device(own.pop("out"), torch.float32)
             branch.bind(own, rt)
+        if self.scales is not None:
+            self._join(rt)
+
+    def _join(self, rt) -> None:
+        if rt.dtype != torch.bfloat16 or not all(hasattr(branch, "give_output_matrix") for branch in self.branches):
+            return
+        left, right = self.branches
+        first = left.give_output_matrix(rt, self.scales[0])
+        if first is None:
+            return
+        second = right.give_output_matrix(rt, self.scales[1])
+        if second is None:
+            raise ValueError(f"the right branch ({type(right).__name__}) keeps its output matrix")
+        self.columns = (0, first.shape[1])
+        self.w_out = torch.cat([first, second], dim=1).contiguous()
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, cache, rt, write_cache: bool = True) -> None:
         views = iter(cache if isinstance(cache, (tuple, list)) else (cache,))
+        if self.w_out is not None:
+            joined = rt.ws.buffer("branches", (batch.n_tokens, self.w_out.shape[1]), rt.dtype)
+            for branch, need, column in zip(self.branches, self._needs, self.columns):
+                branch.forward(h, None, batch, next(views) if need is not None else None, rt, write_cache,
+                               operand=(joined, column))
+            ops.gemm(residual, joined, self.w_out, ops.EPI_RESIDUAL)
+            return
         outputs = []
         for index, (branch, need) in enumerate(zip(self.branches, self._needs)):
             out = rt.ws.buffer(f"branch_{index}", (batch.n_tokens, self.hidden_size), torch.float32)

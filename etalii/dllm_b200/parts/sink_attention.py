@@ -62,6 +62,7 @@ class SinkAttention:
         self.cache_keep = max(int(keep) for _, keep in readers) if bounded else 0
         self.padded = -(-self.num_heads * self.vdim // 8) * 8
         """The output product's rows: heads x vdim filled up with zeros to 16-byte pieces."""
+        self.output_scale = 1.0
         self.w_in = self.w_o = self.bias_rows = self.sinks = self.norm_weights = self.output_bias = None
 
     @staticmethod
@@ -124,15 +125,23 @@ class SinkAttention:
         if self.position is not None:
             self.position.bind({}, rt)
 
+    def give_output_matrix(self, rt, scale: float) -> torch.Tensor | None:
+        """As `Attention.give_output_matrix` (None also for an output that has a bias or ends between 16-byte pieces)."""
+        if self.has_output_bias or self.padded != self.num_heads * self.vdim:
+            return None
+        w, self.w_o, self.output_scale = self.w_o, None, float(scale)
+        return w
+
     def take_output_bias(self) -> torch.Tensor | None:
         """The output bias (None: there is none); the part no longer adds it itself."""
         bias, self.output_bias = self.output_bias, None
         return bias
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, batch, cache, rt, write_cache: bool = True,
-                epilogue: int = ops.EPI_RESIDUAL) -> None:
+                epilogue: int = ops.EPI_RESIDUAL, operand=None) -> None:
         """h: the mixer's input [tokens, hidden] in the activation type. Adds the output to `residual` (float32), or
-        with `epilogue=ops.EPI_STORE_F32` writes it there."""
+        with `epilogue=ops.EPI_STORE_F32` writes it there, or with `operand` = (rows, column) leaves what the output
+        matrix multiplies there (`give_output_matrix`)."""
         n = batch.n_tokens
         heads, groups, dim, vdim = self.num_heads, self.num_kv_heads, self.dim, self.vdim
         rows = rt.ws.buffer("mixer_rows", (n, self.w_in.shape[0]), torch.float32)
@@ -148,7 +157,7 @@ class SinkAttention:
                         eps=self.qk_eps or 0.0, table=table,
                         rotary_dim=self.position.rotary_dim if self.position is not None else 0, first=first,
                         share=self.share)
-        attended = rt.ws.buffer("attended", (n, self.padded), rt.dtype)
+        attended, at = operand or (rt.ws.buffer("attended", (n, self.padded), rt.dtype), None)
         attend = ops.sink_attention
         if ops.sink_attention_tiles(rt.dtype, dim, vdim, cache.page_size):
             reach = batch.max_context
@@ -161,7 +170,11 @@ class SinkAttention:
             else:
                 attend = ops.sink_attention_prefill
         more = {"chunk": self.chunk} if self.chunk else {}
+        if operand is not None:
+            more.update(out_scale=self.output_scale, out_at=at)
         attend(attended, q, cache, heads, self.scale, self.softcap, self.sinks, self.window, self.keep_first, batch, **more)
+        if operand is not None:
+            return
         ops.gemm(residual, attended, self.w_o, epilogue)
         if self.output_bias is not None:
             ops.add_row(residual, self.output_bias)

@@ -678,9 +678,6 @@ def test_state_space_part_in_pieces(name, dtype, shape):
     got = _feed(PartHarness(part.cache_need(), dtype, 3), _mixer_call(part, rt), sequences, SCHEDULE, width)
     for rows, h in zip(got, sequences):
         assert rel_error(rows, _plain_state_space(weights, m, h)) <= PART_TOL[dtype]
-    assert part.take_output_scale(0.3)  # a factor of the whole output, in the norm's weight
-    got = _feed(PartHarness(part.cache_need(), dtype, 1), _mixer_call(part, rt), sequences[:1], [[(0, 75)]], width)
-    assert rel_error(got[0], 0.3 * _plain_state_space(weights, m, sequences[0])) <= PART_TOL[dtype]
 
 
 @pytest.mark.parametrize("name,dtype", DTYPES)
@@ -745,6 +742,72 @@ def test_the_convolution_reaches_back_by_its_taps_and_no_further(name, dtype, co
         got, moved = run(other), np.abs(run(other) - run(h)).max(axis=1)
         assert rel_error(got, _plain_state_space(weights, m, other, 1e-2)) <= PART_TOL[dtype]
         assert [i for i in range(55) if moved[i] > 1e-3] == list(range(marked, min(55, marked + conv)))
+
+
+# ---- both branches side by side -------------------------------------------------------------------------------------------------
+
+
+class NestedHarness(PartHarness):
+    """A harness for a mixer whose branches keep several things each."""
+
+    def __init__(self, need, dtype, sequences, **more):
+        flat = []
+
+        def collect(n):
+            if n.kind == "several":
+                return tuple(collect(p) for p in n.parts)
+            flat.append(n)
+            return len(flat) - 1
+
+        shape = collect(need)
+        from etalii.dllm_b200.cache.paged import CacheNeed
+
+        super().__init__(CacheNeed("several", parts=tuple(flat)), dtype, sequences, **more)
+        views = self.view
+        view_of = lambda at: tuple(view_of(a) for a in at) if isinstance(at, tuple) else views[at]  # noqa: E731
+        self.view = view_of(shape)
+
+
+PARALLEL_SHAPES = {
+    "tiles": C.parallel(4, 1, 64, 64, 100, 64, 0.12, (6, 32, 32, 2, 4, 3)),
+    "half_turned": C.parallel(6, 3, 128, 128, 50, 64, 0.08, (6, 32, 32, 1, 3, 1), 0.8, 0.5),
+    "values_of_their_own": C.parallel(4, 2, 24, 40, 33, 8, 0.2, (4, 12, 10, 2, 3, 2), 1.0, 2.0),
+    "rows_that_end_anywhere": C.parallel(3, 1, 10, 14, 9, 4, 0.3, (6, 7, 9, 3, 1, 1)),
+    "odd_inner": C.parallel(2, 2, 32, 32, 40, 32, 0.2, (3, 7, 9, 1, 2, 3), 0.3, -0.9),
+}
+
+
+@pytest.mark.parametrize("name,dtype", DTYPES)
+@pytest.mark.parametrize("shape", sorted(PARALLEL_SHAPES))
+def test_both_branches_in_pieces(name, dtype, shape):
+    """The weighted sum of the branches, added to what is there: as one product over both operands side by side where their
+    sizes allow it, else as two and a sum."""
+    from etalii.dllm_b200.architectures.zivazen import mixer_spec
+
+    rt = _runtime(dtype)
+    layer, width = PARALLEL_SHAPES[shape], 72
+    m = layer["mixer"]
+    weights = {f"left.{k}": v for k, v in _window_weights(len(shape), width, m["left"]).items()}
+    weights.update({f"right.{k}": v for k, v in _state_space_weights(len(shape), width, m["right"]).items()})
+    spec = mixer_spec(width, 1e-5, layer, "", None)
+    part = _part("mixer", spec.kind, **spec.params)
+    part.bind({k: v for k, v in weights.items()}, rt)
+    joined = dtype == torch.bfloat16 and m["left"]["heads"] * m["left"]["vdim"] % 8 == 0
+    assert (part.w_out is not None) == joined
+    sequences = _inputs(dtype, width, 3)
+
+    def call(h, out, batch, view):
+        out.fill_(0.5)
+        part.forward(h.to(rt.dtype), out, batch, view, rt)
+
+    got = _feed(NestedHarness(part.cache_need(), dtype, 3), call, sequences, SCHEDULE, width)
+    named = _np(weights, (("conv_bias", "conv.b"),))
+    for rows, h in zip(got, sequences):
+        want = P.parallel(named, m, h.double().numpy(), None, 0, 1e-5)[0]
+        assert rel_error(rows - 0.5, want) <= PART_TOL[dtype]
+    long = _inputs(dtype, width, 4, [430])  # prompts that take the kernels for long contexts
+    got = _feed(NestedHarness(part.cache_need(), dtype, 1), call, long, [[(0, 300)], [(0, 127)]] + [[(0, 1)]] * 3, width)[0]
+    assert rel_error(got - 0.5, P.parallel(named, m, long[0].double().numpy(), None, 0, 1e-5)[0]) <= PART_TOL[dtype]
 
 
 # ---- whole models through the engine -------------------------------------------------------------------------------------------
