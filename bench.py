@@ -1201,13 +1201,15 @@ def zivazen_rooflines(row: dict, size: dict, batch: int, peak: dict, contexts: l
                                "fp32": rate / (148 * 128 * 2 * 1.965e9)}[unit], 4)
 
     window = ZIVAZEN_WINDOW
-    for name, model, kernel, seen, past in (
-            ("zivazen_attention", "zivazen", "sink_attention", n * n / 2, contexts),
-            ("zivazen_window", "zivazen", "attention_", sum(min(i + 1, window) for i in range(n)),
+    for name, model, mask, seen, past in (
+            ("zivazen_attention", "zivazen", " chunk=", n * n / 2, contexts),
+            ("zivazen_window", "zivazen", " window=", sum(min(i + 1, window) for i in range(n)),
              [min(c, window) for c in contexts]),
-            ("llama_attention", "llama", "attention", n * n / 2, contexts)):
-        put(name + "_prefill_bf16_frac", 2 * h * 2 * d * seen, _first(row[model]["prefill_kernels"], kernel), "bf16")
-        put(name + "_decode_hbm_frac", 2 * sum(past) * g * 2 * d, _first(row[model]["decode_kernels"], kernel), "hbm")
+            ("llama_attention", "llama", "", n * n / 2, contexts)):
+        prompt, single = (next((k for label, k in row[model][phase + "_kernels"].items()
+                                if "attention" in label and mask in label), None) for phase in ("prefill", "decode"))
+        put(name + "_prefill_bf16_frac", 2 * h * 2 * d * seen, prompt, "bf16")
+        put(name + "_decode_hbm_frac", 2 * sum(past) * g * 2 * d, single, "hbm")
     for model, scan, columns in (("zivazen", "state_space_scan", d), ("revupel", "gated_scan", d + 1),
                                  ("tisalorn", "decay_scan", d)):
         put(f"{model}_scan_decode_hbm_frac", 2 * 4 * batch * h * columns * d, row[model]["decode_kernels"].get(scan), "hbm")

@@ -91,6 +91,7 @@ __global__ void __launch_bounds__(256) embed_normed_kernel(float* __restrict__ o
                                                            const int* __restrict__ tokens,
                                                            const float* __restrict__ weight, int hidden, int vocab,
                                                            float scale, float eps, int* __restrict__ status) {
+  constexpr int PLACES = 16;
   __shared__ float partial[8];
   int row = blockIdx.x;
   pdl_launch_dependents();
@@ -102,10 +103,17 @@ __global__ void __launch_bounds__(256) embed_normed_kernel(float* __restrict__ o
     return;
   }
   const T* src = table + (size_t)token * hidden;
-  float sum = 0.f;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-    float v = to_float(src[i]) * scale;
-    sum = fmaf(v, v, sum);
+  float sum = 0.f, v[PLACES];  // (the first PLACES values of a thread wait in registers for the sum)
+#pragma unroll
+  for (int p = 0; p < PLACES; ++p) {
+    int i = threadIdx.x + p * blockDim.x;
+    v[p] = i < hidden ? to_float(src[i]) * scale : 0.f;
+  }
+#pragma unroll
+  for (int p = 0; p < PLACES; ++p) sum = fmaf(v[p], v[p], sum);
+  for (int i = threadIdx.x + PLACES * blockDim.x; i < hidden; i += blockDim.x) {
+    float u = to_float(src[i]) * scale;
+    sum = fmaf(u, u, sum);
   }
   sum = warp_sum(sum);
   if ((threadIdx.x & 31) == 0) partial[threadIdx.x >> 5] = sum;
@@ -113,7 +121,12 @@ __global__ void __launch_bounds__(256) embed_normed_kernel(float* __restrict__ o
   float total = 0.f;
   for (int w = 0; w < (int)(blockDim.x >> 5); ++w) total += partial[w];
   const float inv = 1.0f / sqrtf(total / (float)hidden + eps);
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x)
+#pragma unroll
+  for (int p = 0; p < PLACES; ++p) {
+    int i = threadIdx.x + p * blockDim.x;
+    if (i < hidden) out[(size_t)row * hidden + i] = v[p] * inv * weight[i];
+  }
+  for (int i = threadIdx.x + PLACES * blockDim.x; i < hidden; i += blockDim.x)
     out[(size_t)row * hidden + i] = to_float(src[i]) * scale * inv * weight[i];
 }
 

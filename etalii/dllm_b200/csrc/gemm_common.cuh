@@ -29,6 +29,8 @@
 // W's rows interleave gate and up; C in the activation type [M,N/2] = gelu(gate) * up with the tanh form of gelu,
 // 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))), in float32. Where EPI_GLU_CLAMPED is: the weight-streaming kernels.
 #define EPI_GLU_GELU_TANH 11
+// C in the activation type [M,N] = max(product, 0)^2, in float32. Where EPI_GLU_CLAMPED is, without a norm in front.
+#define EPI_RELU_SQUARED 12
 
 // What the q/k/v epilogue needs: where queries go, where the cache is, the rotation table, who the tokens are.
 struct RopeArgs {
@@ -123,6 +125,12 @@ __device__ __forceinline__ void epilogue_pair(void* __restrict__ c, int m, int n
     T* dst = (T*)c + (size_t)m * N + n;
     dst[0] = from_float<T>(v0);
     if (second) dst[1] = from_float<T>(v1);
+  } else if (EPI == EPI_RELU_SQUARED) {
+    T* dst = (T*)c + (size_t)m * N + n;
+    v0 = fmaxf(v0, 0.f);
+    v1 = fmaxf(v1, 0.f);
+    dst[0] = from_float<T>(v0 * v0);
+    if (second) dst[1] = from_float<T>(v1 * v1);
   } else if (EPI == EPI_RESIDUAL) {
     float* dst = (float*)c + (size_t)m * N + n;
     dst[0] += v0;

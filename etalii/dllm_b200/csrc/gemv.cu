@@ -375,6 +375,9 @@ int dispatch(void* c, const void* a, const float* norm_w, float eps, const bf16*
     case EPI_ARGMAX: return launch<EPI_ARGMAX, NORM>(c, a, norm_w, eps, w, M, N, K, rope, pf, stream);
     case EPI_GLU_CLAMPED: return launch<EPI_GLU_CLAMPED, NORM>(c, a, norm_w, eps, w, M, N, K, rope, pf, stream);
     case EPI_GLU_GELU_TANH: return launch<EPI_GLU_GELU_TANH, NORM>(c, a, norm_w, eps, w, M, N, K, rope, pf, stream);
+    case EPI_RELU_SQUARED:
+      if (!NORM) return launch<EPI_RELU_SQUARED, false>(c, a, nullptr, eps, w, M, N, K, rope, pf, stream);
+      return DLLM_BAD_ARGUMENT;
     default: return DLLM_BAD_ARGUMENT;
   }
 }
@@ -390,8 +393,8 @@ DLLM_EXPORT int dllm_gemv_bf16(void* c, const void* a, const float* norm_w, floa
   bool gated = epilogue == EPI_SWIGLU || epilogue == EPI_GLU_CLAMPED || epilogue == EPI_GLU_GELU_TANH;
   if (M > 64 || K <= 0 || (K & 7) || ((N & 1) && gated) || epilogue < 0 ||
       (epilogue > EPI_SWIGLU && epilogue != EPI_ARGMAX && epilogue != EPI_GLU_CLAMPED &&
-       epilogue != EPI_GLU_GELU_TANH) ||
-      (epilogue == EPI_GLU_CLAMPED && norm_w != nullptr))
+       epilogue != EPI_GLU_GELU_TANH && epilogue != EPI_RELU_SQUARED) ||
+      ((epilogue == EPI_GLU_CLAMPED || epilogue == EPI_RELU_SQUARED) && norm_w != nullptr))
     return DLLM_UNSUPPORTED_SIZE;
   RopeArgs rope{};
   Prefetch pf{(const char*)prefetch_ptr, prefetch_ptr ? (size_t)prefetch_bytes : 0};

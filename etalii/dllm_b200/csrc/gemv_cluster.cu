@@ -389,6 +389,9 @@ int dispatch(void* c, const void* a, const float* norm_w, float eps, const bf16*
     case EPI_QKV_ROPE: return launch<EPI_QKV_ROPE, NORM>(c, a, norm_w, eps, w, M, N, K, rope, pf, blocks, stream);
     case EPI_GLU_CLAMPED: return launch<EPI_GLU_CLAMPED, NORM>(c, a, norm_w, eps, w, M, N, K, rope, pf, blocks, stream);
     case EPI_GLU_GELU_TANH: return launch<EPI_GLU_GELU_TANH, NORM>(c, a, norm_w, eps, w, M, N, K, rope, pf, blocks, stream);
+    case EPI_RELU_SQUARED:
+      if (!NORM) return launch<EPI_RELU_SQUARED, false>(c, a, nullptr, eps, w, M, N, K, rope, pf, blocks, stream);
+      return DLLM_BAD_ARGUMENT;
     default: return DLLM_BAD_ARGUMENT;
   }
 }
@@ -404,8 +407,9 @@ DLLM_EXPORT int dllm_gemv_cluster(void* c, const void* a, const float* norm_w, f
   if (M <= 0 || N <= 0) return DLLM_OK;
   bool gated = epilogue == EPI_SWIGLU || epilogue == EPI_GLU_CLAMPED || epilogue == EPI_GLU_GELU_TANH;
   if (M > 64 || K <= 0 || (K & 7) || ((N & 1) && gated) || epilogue < 0 ||
-      (epilogue > EPI_SWIGLU && epilogue != EPI_GLU_CLAMPED && epilogue != EPI_GLU_GELU_TANH) ||
-      (epilogue == EPI_GLU_CLAMPED && norm_w != nullptr))
+      (epilogue > EPI_SWIGLU && epilogue != EPI_GLU_CLAMPED && epilogue != EPI_GLU_GELU_TANH &&
+       epilogue != EPI_RELU_SQUARED) ||
+      ((epilogue == EPI_GLU_CLAMPED || epilogue == EPI_RELU_SQUARED) && norm_w != nullptr))
     return DLLM_UNSUPPORTED_SIZE;
   if (cluster < 0) return DLLM_BAD_ARGUMENT;
   int blocks = cluster;

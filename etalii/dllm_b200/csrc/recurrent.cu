@@ -6,7 +6,7 @@
 //   the same by channels:    S <- diag(g_t) S, a decay per key channel (row of S), then as the gated delta rule
 //   gated outer products:    S <- a_t S + b_t k_t v_t^T  (a_t, b_t per token and head);   o_t = S^T q_t, and the
 //                            same sum with v = 1 as one more column of S (the normaliser n_t), read out as n_t . q_t
-//   state-space duality:     the same without a normaliser, heads sharing k and q, and o_t = S^T q_t + skip v_t
+//   state-space duality:     (whose prompts may run in segments side by side) the same without a normaliser, heads sharing k and q, and o_t = S^T q_t + skip v_t
 //
 // One kernel serves prompts and single tokens: a block owns 16 columns of one head's S for one sequence and walks
 // that sequence's new tokens in order, from the state the cache holds to the state it leaves there. A column's
@@ -73,6 +73,12 @@ struct ScanArgs {
   int decay_stride;
   // state-space duality: the read-out gets skip[head] times the token's own v
   const float* skip;
+  // segments of a prompt side by side (0: none): a sequence's tokens in stretches of `segment`, at most `segments` of them;
+  // segment_state [sequences][segments][heads][vdim][dim] holds what each leaves of a zero state, then what each starts
+  // from; segment_decay [sequences][segments][heads] the product of its tokens' factors
+  int segment, segments;
+  float* segment_state;
+  float* segment_decay;
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -82,7 +88,7 @@ __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
 
 // MODE 0: decayed outer products; MODE 1: gated delta rule; MODE 2: gated outer products; MODE 3: the delta rule with a
 // decay per row of S (whose stage rows hold the decays between q and v); MODE 4: gated outer products without a normaliser,
-// whose read-out gets a share of v. TOKENS: tokens a stage. LPC lanes share a column (8 or
+// whose read-out gets a share of v; MODE 5: the same without a read-out (what a segment leaves of a zero state). TOKENS: tokens a stage. LPC lanes share a column (8 or
 // 16), each with RPL rows of it: the block has 16 * LPC threads. Few lanes a column mean few shuffles and few
 // instructions a token; many lanes mean more warps to hide latency behind, which is what a step with few sequences
 // and heads needs (one warp per scheduler issues a dependent instruction every four cycles and no faster).
@@ -91,12 +97,16 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   constexpr int DIMP = RPL * LPC;  // rows a stage holds per token (the head's dim rounded up)
   constexpr int CPW = 32 / LPC;    // columns a warp owns
   constexpr int SCAN_THREADS = SCAN_COLS * LPC;
-  constexpr int V_AT = (MODE == 3 ? 3 : 2) * DIMP;  // where the values start in a stage row
+  constexpr int VECTORS = MODE == 3 ? 3 : MODE == 5 ? 1 : 2;
+  constexpr int V_AT = VECTORS * DIMP;  // where the values start in a stage row
   constexpr int PER_TOKEN = V_AT + SCAN_COLS + 4;
   constexpr int PIECES = PER_TOKEN / 4;  // 16-byte pieces of a token's stage row
   extern __shared__ __align__(16) float stage[];  // [STAGES][TOKENS][PER_TOKEN]: k | q | (decays) | v (16 columns) | g, beta, k.q, -
   pdl_launch_dependents();
-  const int head = blockIdx.y, seq = blockIdx.z, col0 = blockIdx.x * SCAN_COLS;
+  constexpr bool SEGMENTS = MODE >= 4;
+  const bool segmented = SEGMENTS && a.segment > 0;
+  const int head = blockIdx.y, col0 = blockIdx.x * SCAN_COLS;
+  const int seq = segmented ? blockIdx.z / a.segments : blockIdx.z, part = segmented ? blockIdx.z % a.segments : 0;
   const int qk_head = head / (a.heads / a.qk_heads);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rg = lane / CPW, cc = lane % CPW;
@@ -104,15 +114,27 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   const float decay = MODE == 0 ? a.decay[head] : 0.f, skip = MODE == 4 ? a.skip[head] : 0.f;
   const int state_cols = a.vdim + (MODE == 2 ? 1 : 0);
   pdl_wait();
-  const int first = a.cu_seqlens[seq], count = a.cu_seqlens[seq + 1] - first;
+  int first = a.cu_seqlens[seq], count = a.cu_seqlens[seq + 1] - first;
   const int slot = a.slots[seq];
   float* my_state = a.state + (((size_t)slot * a.heads + head) * state_cols + col) * (size_t)a.dim + rg * 4;
+  const float* start = my_state;  // where this block's state comes from, and
+  bool leaves = true;             // whether it goes to `my_state`
+  if (segmented) {
+    float* kept = a.segment_state + (((size_t)blockIdx.z * a.heads + head) * a.vdim + col) * (size_t)a.dim + rg * 4;
+    const int behind = count - (part + 1) * a.segment;  // tokens behind this segment
+    if (behind + a.segment <= 0 || (MODE == 5 && behind <= 0)) return;
+    if (MODE == 5) my_state = kept;
+    else if (count > a.segment) start = kept;
+    leaves = MODE == 5 || behind <= 0;
+    first += part * a.segment;
+    count = min(a.segment, count - part * a.segment);
+  }
 
   float S[RPL];  // (dim is a multiple of 4 and so is a lane's first row: a piece of 4 rows is inside the head or not)
 #pragma unroll
   for (int j = 0; j < RPL; j += 4) {
-    float4 s4 = (col < state_cols && j * LPC + rg * 4 < a.dim) ? *reinterpret_cast<const float4*>(my_state + j * LPC)
-                                                             : make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 s4 = (MODE != 5 && col < state_cols && j * LPC + rg * 4 < a.dim)
+                    ? *reinterpret_cast<const float4*>(start + j * LPC) : make_float4(0.f, 0.f, 0.f, 0.f);
     S[j] = s4.x; S[j + 1] = s4.y; S[j + 2] = s4.z; S[j + 3] = s4.w;
   }
 
@@ -133,7 +155,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
         const float* src = nullptr;
         if (e < DIMP) {
           if (e < a.dim) src = k0 + row + e;
-        } else if (e < 2 * DIMP) {
+        } else if (MODE != 5 && e < 2 * DIMP) {
           if (e - DIMP < a.dim) src = q0 + row + (e - DIMP);
         } else if (MODE == 3 && e < 3 * DIMP) {
           if (e - 2 * DIMP < a.dim) src = d0 + t * a.decay_stride + (e - 2 * DIMP);
@@ -143,7 +165,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           const float* aux = a.aux + (size_t)(first + t0 + t) * a.aux_stride;
           cp_async4(to, aux + head);
           cp_async4(to + 1, aux + a.heads + head);
-          if (MODE != 4) cp_async4(to + 2, aux + 2 * a.heads + qk_head);
+          if (MODE < 4) cp_async4(to + 2, aux + 2 * a.heads + qk_head);
           continue;
         }
         if (src != nullptr) cp_async16(to, src);
@@ -156,7 +178,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
         const float* src = nullptr;
         if (e < DIMP) {
           if (e < a.dim) src = a.k + token * a.stride + qk_head * a.dim + e;
-        } else if (e < 2 * DIMP) {
+        } else if (MODE != 5 && e < 2 * DIMP) {
           if (e - DIMP < a.dim) src = a.q + token * a.stride + qk_head * a.dim + (e - DIMP);
         } else if (MODE == 3 && e < 3 * DIMP) {
           if (e - 2 * DIMP < a.dim) src = a.decays + token * a.decay_stride + head * a.dim + (e - 2 * DIMP);
@@ -167,7 +189,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           int which = e - V_AT - SCAN_COLS;
           if (which == 0) src = a.aux + token * a.aux_stride + head;
           else if (which == 1) src = a.aux + token * a.aux_stride + a.heads + head;
-          else if (which == 2 && MODE != 4) src = a.aux + token * a.aux_stride + 2 * a.heads + qk_head;
+          else if (which == 2 && MODE < 4) src = a.aux + token * a.aux_stride + 2 * a.heads + qk_head;
         }
         if (src != nullptr) cp_async4(dst + i, src);
         else dst[i] = 0.f;
@@ -176,24 +198,27 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
     cp_async_commit();
   };
 
+  float product = 1.f;  // MODE 5: the product of the tokens' factors
   // one token of the decayed sum: the state moves on, the lane's part of S^T q comes back. Two rows an instruction
   // (the packed float32 multiply-add of sm_100: the same roundings as two single ones, half the issue slots).
   auto decayed = [&](const float* row) -> float {
-    float v = row[2 * DIMP + warp * CPW + cc];
+    float v = row[V_AT + warp * CPW + cc];
     float keep = decay;
-    if (MODE == 2 || MODE == 4) {  // this token's own factors; the column behind the values is written with v = 1
-      keep = row[2 * DIMP + SCAN_COLS];
-      v = (MODE == 2 && col == a.vdim ? 1.0f : v) * row[2 * DIMP + SCAN_COLS + 1];
+    if (MODE == 2 || MODE >= 4) {  // this token's own factors; the column behind the values is written with v = 1
+      keep = row[V_AT + SCAN_COLS];
+      v = (MODE == 2 && col == a.vdim ? 1.0f : v) * row[V_AT + SCAN_COLS + 1];
     }
+    if (MODE == 5) product *= keep;
     const float2 vv = make_float2(v, v), dd = make_float2(keep, keep);
     float2 p = make_float2(0.f, 0.f);
 #pragma unroll
     for (int j = 0; j < RPL; j += 4) {
       float4 k4 = *reinterpret_cast<const float4*>(row + j * LPC + rg * 4);
-      float4 q4 = *reinterpret_cast<const float4*>(row + DIMP + j * LPC + rg * 4);
       float2 s01 = __ffma2_rn(dd, make_float2(S[j], S[j + 1]), __fmul2_rn(make_float2(k4.x, k4.y), vv));
       float2 s23 = __ffma2_rn(dd, make_float2(S[j + 2], S[j + 3]), __fmul2_rn(make_float2(k4.z, k4.w), vv));
       S[j] = s01.x; S[j + 1] = s01.y; S[j + 2] = s23.x; S[j + 3] = s23.y;
+      if (MODE == 5) continue;
+      float4 q4 = *reinterpret_cast<const float4*>(row + DIMP + j * LPC + rg * 4);
       p = __ffma2_rn(s01, make_float2(q4.x, q4.y), p);
       p = __ffma2_rn(s23, make_float2(q4.z, q4.w), p);
     }
@@ -220,7 +245,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
     // thread per token and column, and writes whole pieces of rows.
     float* parts = stage + (size_t)STAGES * TOKENS * PER_TOKEN;  // [TOKENS][16 columns][LPC + 4]
     constexpr int PADL = LPC + 4;
-    if (MODE == 0 || MODE == 2 || MODE == 4) {
+    if (MODE == 0 || MODE == 2 || MODE >= 4) {
       // The decayed sum's read-out does not feed the state: nothing but the state's own multiply-add links two tokens.
       // a group of tokens at a time: all their rows are asked of shared memory first (the loads do not depend on the
       // state), then the state walks through them
@@ -232,16 +257,17 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
 #pragma unroll
         for (int w = 0; w < GROUP; ++w) {
           const float* row = base + (u + w) * PER_TOKEN;
-          v[w] = row[2 * DIMP + warp * CPW + cc];
+          v[w] = row[V_AT + warp * CPW + cc];
           keep[w] = decay;
-          if (MODE == 2 || MODE == 4) {
-            keep[w] = row[2 * DIMP + SCAN_COLS];
-            v[w] = (MODE == 2 && col == a.vdim ? 1.0f : v[w]) * row[2 * DIMP + SCAN_COLS + 1];
+          if (MODE == 2 || MODE >= 4) {
+            keep[w] = row[V_AT + SCAN_COLS];
+            v[w] = (MODE == 2 && col == a.vdim ? 1.0f : v[w]) * row[V_AT + SCAN_COLS + 1];
           }
+          if (MODE == 5) product *= keep[w];
 #pragma unroll
           for (int j = 0; j < RPL; j += 4) {
             kq[w][j / 2] = *reinterpret_cast<const float4*>(row + j * LPC + rg * 4);
-            kq[w][j / 2 + 1] = *reinterpret_cast<const float4*>(row + DIMP + j * LPC + rg * 4);
+            if (MODE != 5) kq[w][j / 2 + 1] = *reinterpret_cast<const float4*>(row + DIMP + j * LPC + rg * 4);
           }
         }
 #pragma unroll
@@ -250,18 +276,22 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
           float2 p = make_float2(0.f, 0.f);
 #pragma unroll
           for (int j = 0; j < RPL; j += 4) {
-            float4 k4 = kq[w][j / 2], q4 = kq[w][j / 2 + 1];
+            float4 k4 = kq[w][j / 2];
             float2 s01 = __ffma2_rn(dd, make_float2(S[j], S[j + 1]), __fmul2_rn(make_float2(k4.x, k4.y), vv));
             float2 s23 = __ffma2_rn(dd, make_float2(S[j + 2], S[j + 3]), __fmul2_rn(make_float2(k4.z, k4.w), vv));
             S[j] = s01.x; S[j + 1] = s01.y; S[j + 2] = s23.x; S[j + 3] = s23.y;
+            if (MODE == 5) continue;
+            float4 q4 = kq[w][j / 2 + 1];
             p = __ffma2_rn(s01, make_float2(q4.x, q4.y), p);
             p = __ffma2_rn(s23, make_float2(q4.z, q4.w), p);
           }
-          parts[((u + w) * SCAN_COLS + warp * CPW + cc) * PADL + rg] = p.x + p.y;
+          if (MODE != 5) parts[((u + w) * SCAN_COLS + warp * CPW + cc) * PADL + rg] = p.x + p.y;
         }
       }
-      for (; u < here; ++u)
-        parts[(u * SCAN_COLS + warp * CPW + cc) * PADL + rg] = decayed(base + u * PER_TOKEN);
+      for (; u < here; ++u) {
+        const float p = decayed(base + u * PER_TOKEN);
+        if (MODE != 5) parts[(u * SCAN_COLS + warp * CPW + cc) * PADL + rg] = p;
+      }
     } else {
       // The delta rule: what the state answers to k feeds the write, so the sum S^T k is finished token by token (the
       // shuffles are most of the time from one token to the next); S^T q waits for the end of the chunk. A token's rows
@@ -323,7 +353,7 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
       }
     }
     __syncthreads();
-    for (int i = tid; i < here * SCAN_COLS; i += SCAN_THREADS) {
+    for (int i = tid; MODE != 5 && i < here * SCAN_COLS; i += SCAN_THREADS) {
       int u = i / SCAN_COLS, c = i % SCAN_COLS;
       const float4* mine = reinterpret_cast<const float4*>(parts + i * PADL);
       float sum = 0.f;
@@ -342,14 +372,15 @@ __global__ void __launch_bounds__(SCAN_COLS * LPC) scan_kernel(ScanArgs a) {
   }
 #pragma unroll
   for (int j = 0; j < RPL; j += 4)
-    if (col < state_cols && j * LPC + rg * 4 < a.dim)
+    if (leaves && col < state_cols && j * LPC + rg * 4 < a.dim)
       *reinterpret_cast<float4*>(my_state + j * LPC) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
+  if (MODE == 5 && col0 == 0 && tid == 0) a.segment_decay[(size_t)blockIdx.z * a.heads + head] = product;
 }
 
 template <int RPL, int LPC, int MODE, int TOKENS, int STAGES>
 static int launch_scan_case(const ScanArgs& a, dim3 grid, cudaStream_t stream) {
-  size_t bytes = (size_t)STAGES * TOKENS * ((MODE == 3 ? 3 : 2) * RPL * LPC + SCAN_COLS + 4) * sizeof(float);
-  bytes += (size_t)TOKENS * SCAN_COLS * (LPC + 4) * sizeof(float);  // the parts of the read-out
+  size_t bytes = (size_t)STAGES * TOKENS * ((MODE == 3 ? 3 : MODE == 5 ? 1 : 2) * RPL * LPC + SCAN_COLS + 4) * sizeof(float);
+  if (MODE != 5) bytes += (size_t)TOKENS * SCAN_COLS * (LPC + 4) * sizeof(float);  // the parts of the read-out
   static bool allowed = false;  // (more than 48 KB of dynamic shared memory has to be asked for once)
   if (bytes > 48 * 1024 && !allowed) {
     if (cudaFuncSetAttribute(scan_kernel<RPL, LPC, MODE, TOKENS, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -383,6 +414,42 @@ static int launch_scan(const ScanArgs& a, int sequences, int longest, cudaStream
   SCAN_CASE(32, 8, 8) SCAN_CASE(16, 16, 8)
 #undef SCAN_CASE
   return DLLM_UNSUPPORTED_SIZE;
+}
+
+// The same over segments of prompts side by side: few lanes a column (few instructions a token; there are blocks enough)
+// and few stages (several blocks a multiprocessor hide each other's latency).
+template <int MODE>
+static int launch_segments(const ScanArgs& a, int sequences, cudaStream_t stream) {
+  dim3 grid((a.vdim + SCAN_COLS - 1) / SCAN_COLS, a.heads, sequences * a.segments);
+  if (a.dim <= 32) return launch_scan_case<4, 8, MODE, 16, 2>(a, grid, stream);
+  if (a.dim <= 64) return launch_scan_case<8, 8, MODE, 16, 2>(a, grid, stream);
+  if (a.dim <= 128) return launch_scan_case<16, 8, MODE, 16, 2>(a, grid, stream);
+  return launch_scan_case<32, 8, MODE, 8, 2>(a, grid, stream);
+}
+
+// From what every segment leaves of a zero state to what it starts from: S = the cache's state; segment by segment, start =
+// S, S = decay S + left. A thread per four values of a head's matrix. Sequences of one segment are left out.
+__global__ void __launch_bounds__(256) segment_states_kernel(ScanArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int head = blockIdx.y, seq = blockIdx.z, count = a.cu_seqlens[seq + 1] - a.cu_seqlens[seq];
+  const int fours = a.vdim * a.dim / 4, i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= fours || count <= a.segment) return;
+  float4 s = reinterpret_cast<const float4*>(a.state + ((size_t)a.slots[seq] * a.heads + head) * a.vdim * a.dim)[i];
+  for (int part = 0; part * a.segment < count; ++part) {
+    const size_t at = ((size_t)seq * a.segments + part) * a.heads + head;
+    float4* kept = reinterpret_cast<float4*>(a.segment_state + at * a.vdim * a.dim) + i;
+    float4 left = make_float4(0.f, 0.f, 0.f, 0.f);
+    float decay = 0.f;
+    const bool last = (part + 1) * a.segment >= count;  // (nothing is known of what the last one leaves, nor needed)
+    if (!last) {
+      left = *kept;
+      decay = a.segment_decay[at];
+    }
+    *kept = s;
+    s.x = fmaf(decay, s.x, left.x); s.y = fmaf(decay, s.y, left.y);
+    s.z = fmaf(decay, s.z, left.z); s.w = fmaf(decay, s.w, left.w);
+  }
 }
 
 static bool scan_sizes_ok(int heads, int qk_heads, int dim, int vdim, int stride) {
@@ -468,9 +535,13 @@ DLLM_EXPORT int dllm_gated_scan(const float* q, const float* k, const float* v, 
 
 // State-space duality over the new tokens of every sequence: per head S <- a_t S + b_t k_t v_t^T, out = S^T q_t + skip v_t,
 // head h reading q/k head h / (heads / qk_heads). aux [tokens][aux_stride] holds a (heads) then b (heads); skip [heads].
+// With `segment` > 0 (a multiple of 16) the stretches of that many tokens of a sequence run side by side: first what each
+// leaves of a zero state, then from that what each starts from, then every stretch from there. segment_state and
+// segment_decay are scratch for `segments` = ceil(longest / segment) stretches a sequence (see ScanArgs).
 DLLM_EXPORT int dllm_state_space_scan(const float* q, const float* k, const float* v, int stride, int heads, int qk_heads,
                                       int dim, int vdim, const float* aux, int aux_stride, const float* skip,
                                       float* state, const int* cu_seqlens, const int* slots, int sequences, int longest,
+                                      int segment, int segments, float* segment_state, float* segment_decay,
                                       float* out, cudaStream_t stream) {
   if (sequences <= 0) return DLLM_OK;
   if (!scan_sizes_ok(heads, qk_heads, dim, vdim, stride) || sequences >= 65536 || aux_stride < 2 * heads)
@@ -480,7 +551,17 @@ DLLM_EXPORT int dllm_state_space_scan(const float* q, const float* k, const floa
   a.q = q; a.k = k; a.v = v; a.stride = stride; a.heads = heads; a.qk_heads = qk_heads; a.dim = dim; a.vdim = vdim;
   a.state = state; a.cu_seqlens = cu_seqlens; a.slots = slots; a.out = out; a.aux = aux; a.aux_stride = aux_stride;
   a.skip = skip; a.out_scale = 1.0f; a.vector = scan_vector(q, k, v, stride, dim, vdim);
-  return launch_scan<4>(a, sequences, longest, stream);
+  if (segment <= 0) return launch_scan<4>(a, sequences, longest, stream);
+  if (segment % 16 || (long long)segment * segments < longest || (long long)sequences * segments >= 65536)
+    return DLLM_UNSUPPORTED_SIZE;
+  if (!segment_state || !segment_decay) return DLLM_BAD_ARGUMENT;
+  a.segment = segment; a.segments = segments; a.segment_state = segment_state; a.segment_decay = segment_decay;
+  int status = launch_segments<5>(a, sequences, stream);
+  if (status != DLLM_OK) return status;
+  status = dllm_launch_pdl(segment_states_kernel, dim3((vdim * dim / 4 + 255) / 256, heads, sequences), dim3(256), 0, stream,
+                           a);
+  if (status != DLLM_OK) return status;
+  return launch_segments<4>(a, sequences, stream);
 }
 
 // ---- the gates of the gated outer products under a running maximum ------------------------------------------------

@@ -19,7 +19,10 @@ _STATUS = {-1: "bad argument", -2: "unsupported size", -3: "kernel launch failed
 EPI_GLU_GELU_TANH = 11
 """Gate and up rows interleaved as for SwiGLU: c[M, N/2] = gelu(gate) * up with the tanh form of gelu. Where
 EPI_GLU_CLAMPED is: the weight-streaming kernels (`glu_clamped_fuses`)."""
-_EPILOGUE_NAMES = {0: "store_f32", 1: "store", 2: "residual", 3: "swiglu", 10: "glu_clamped", 11: "glu_gelu_tanh"}
+EPI_RELU_SQUARED = 12
+"""c = max(product, 0)^2 in the weights' dtype. Where EPI_GLU_CLAMPED is."""
+_EPILOGUE_NAMES = {0: "store_f32", 1: "store", 2: "residual", 3: "swiglu", 10: "glu_clamped", 11: "glu_gelu_tanh",
+                   12: "relu_squared"}
 
 
 class KernelError(RuntimeError):
@@ -83,8 +86,8 @@ _prototypes = {
                                             c_float, c_int, c_void_p],
     ("elementwise", "dllm_scaled_sum"): [c_void_p, c_void_p, c_void_p, c_float, c_float, c_longlong, c_void_p],
     ("recurrent", "dllm_state_space_scan"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                                             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
-                                             c_void_p],
+                                             c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                             c_void_p, c_void_p, c_void_p, c_void_p],
     ("recurrent", "dllm_state_space_prepare"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                 c_int, c_void_p, c_void_p, c_int, c_void_p],
@@ -266,7 +269,7 @@ def _check(status: int, what: str, detail="") -> None:
     formatting a message costs a launch's worth of host time)."""
     global launches
     launches += 1
-    if callable(what):
+    if callable(what) and (trace is not None or status != 0):
         what = what()
     if trace is not None and status == 0:
         event = torch.cuda.Event(enable_timing=True)
@@ -661,6 +664,11 @@ def sink_attention(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale:
         "sink_attention", lambda: f"dim={dim}, value_dim={vdim} (at most 256)")
 
 
+def _mask_name(window, chunk) -> str:
+    """What tells a traced launch from one under another mask."""
+    return (f" window={int(window)}" if window else "") + (f" chunk={int(chunk)}" if chunk else "")
+
+
 def sink_attention_tiles(dtype, dim: int, vdim: int, page_size: int = 64) -> bool:
     """Whether the tensor-core kernels for tiles of queries and for single tokens run these sizes."""
     return dtype == torch.bfloat16 and page_size == 64 and dim % 8 == 0 and vdim % 8 == 0 and max(dim, vdim) <= 128
@@ -684,7 +692,7 @@ def sink_attention_prefill(out: torch.Tensor, q: torch.Tensor, cache, heads: int
         cache.max_pages, cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(),
         batch.cu_seqlens.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), batch.n_tiles, float(scale),
         float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0),
-        int(chunk or 0), float(out_scale), _stream()), "sink_attention_prefill")
+        int(chunk or 0), float(out_scale), _stream()), lambda: "sink_attention_prefill" + _mask_name(window, chunk))
 
 
 def sink_attention_tcgen05_supported(cache) -> bool:
@@ -709,7 +717,7 @@ def sink_attention_tcgen05(out: torch.Tensor, q: torch.Tensor, cache, heads: int
         batch.tile_seq.data_ptr(), batch.tile_first.data_ptr(), batch.cu_seqlens.data_ptr(), batch.start.data_ptr(),
         batch.slots.data_ptr(), batch.n_tiles, float(scale), float(softcap or 0.0),
         sinks.data_ptr() if sinks is not None else None, int(window or 0), int(keep or 0), int(chunk or 0),
-        float(out_scale), _status_word().data_ptr(), _stream()), "sink_attention_tcgen05")
+        float(out_scale), _status_word().data_ptr(), _stream()), lambda: "sink_attention_tcgen05" + _mask_name(window, chunk))
 
 
 def sink_attention_decode(out: torch.Tensor, q: torch.Tensor, cache, heads: int, scale: float, softcap: float,
@@ -730,12 +738,12 @@ def sink_attention_decode(out: torch.Tensor, q: torch.Tensor, cache, heads: int,
         cache.max_pages, cache.page_size, heads, cache.kv_heads, dim, vdim, batch.tok_pos.data_ptr(), batch.slots.data_ptr(),
         batch.n_seqs, float(scale), float(softcap or 0.0), sinks.data_ptr() if sinks is not None else None,
         int(window or 0), int(keep or 0), int(chunk or 0), float(out_scale), int(shape), _stream()),
-        "sink_attention_decode")
+        lambda: "sink_attention_decode" + _mask_name(window, chunk))
 
 
 def glu_clamped_fuses(rows: int, outputs: int, inner: int) -> bool:
     """Whether a bfloat16 product of these sizes runs in one of the two weight-streaming kernels that can end in the
-    clamped GLU (a block per 16 rows of W, or the reduction split over a cluster)."""
+    clamped GLU or the square of relu (a block per 16 rows of W, or the reduction split over a cluster)."""
     return streams(rows, outputs, inner) and not takes_weights_as_rows(rows, outputs, inner) and \
         not streams_through_shared_memory(rows, outputs, inner)
 
@@ -1480,19 +1488,40 @@ def state_space_prepare(prepared: torch.Tensor, aux: torch.Tensor, rows: torch.T
         "state_space_prepare", lambda: f"taps={n_taps} (at most 16), dim={dim} (at most 256)")
 
 
+def state_space_segment(batch, heads: int, vdim: int) -> int:
+    """Into stretches of how many tokens a step's prompts are cut for the state-space scan (0: not at all): where the step's
+    own blocks (16 columns of a head and sequence each) would leave the device waiting for one token after the other."""
+    if batch.max_new < 256 or batch.n_seqs * heads * -(-vdim // 16) >= 8 * _multiprocessors():
+        return 0
+    return SCAN_SEGMENT
+
+
+SCAN_SEGMENT = 256
+
+
 def state_space_scan(out: torch.Tensor, prepared: torch.Tensor, aux: torch.Tensor, skip: torch.Tensor, heads: int,
-                     groups: int, padded: int, vdim: int, state: torch.Tensor, batch) -> None:
+                     groups: int, padded: int, vdim: int, state: torch.Tensor, batch, segment: int = 0,
+                     segment_state: torch.Tensor | None = None, segment_decay: torch.Tensor | None = None) -> None:
     """Per sequence and head, over the step's tokens in order: S <- a S + b B x^T, out = S^T C + skip x, with x, B, C and the
-    factors a, b as `state_space_prepare` leaves them. state [slots, heads, vdim, padded] float32."""
-    _cuda(out, prepared, aux, skip, state)
+    factors a, b as `state_space_prepare` leaves them. state [slots, heads, vdim, padded] float32. With `segment` (a
+    multiple of 16) stretches of that many tokens run side by side (three kernels instead of one; scratch: float32,
+    sequences x ceil(longest / segment) x heads matrices [vdim, padded] and as many numbers)."""
+    _cuda(out, prepared, aux, skip, state, segment_state, segment_decay)
     assert all(t.dtype == torch.float32 for t in (out, prepared, aux, skip, state))
     assert tuple(state.shape[1:]) == (heads, vdim, padded) and out.shape[1] == heads * vdim and skip.numel() == heads
-    b_at = heads * vdim
+    b_at, segments = heads * vdim, 0
+    if segment:
+        segments = -(-batch.max_new // segment)
+        matrices = batch.n_seqs * segments * heads
+        assert segment_state.dtype == segment_decay.dtype == torch.float32
+        assert segment_state.numel() >= matrices * vdim * padded and segment_decay.numel() >= matrices
+    ptr = lambda tensor: tensor.data_ptr() if tensor is not None else None  # noqa: E731
     _check(_fn("recurrent", "dllm_state_space_scan")(
         _columns(prepared, b_at + groups * padded), _columns(prepared, b_at), prepared.data_ptr(), prepared.shape[1],
         heads, groups, padded, vdim, aux.data_ptr(), aux.shape[1], skip.data_ptr(), state.data_ptr(),
-        batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_seqs, int(batch.max_new), out.data_ptr(),
-        _stream()), "state_space_scan", lambda: f"dim={padded} (a multiple of 4, at most 256)")
+        batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_seqs, int(batch.max_new), int(segment), segments,
+        ptr(segment_state), ptr(segment_decay), out.data_ptr(), _stream()), "state_space_scan",
+        lambda: f"dim={padded} (a multiple of 4, at most 256), segments of {segment} (a multiple of 16)")
 
 
 def gate_norm(out: torch.Tensor, y: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, parts: int,
@@ -1715,7 +1744,7 @@ def gemm(c: torch.Tensor, a: torch.Tensor, w: torch.Tensor, epilogue: int = EPI_
     n = w.shape[0]
     assert w.shape[1] == k, (a.shape, w.shape)
     want_cols = n // 2 if epilogue in (EPI_SWIGLU, EPI_GLU_CLAMPED, EPI_GLU_GELU_TANH) else n
-    if epilogue in (EPI_GLU_CLAMPED, EPI_GLU_GELU_TANH):
+    if epilogue in (EPI_GLU_CLAMPED, EPI_GLU_GELU_TANH, EPI_RELU_SQUARED):
         assert w.dtype == torch.bfloat16 and kernel == 0 and norm_weight is None and glu_clamped_fuses(m, n, k)
     want_dtype = torch.float32 if epilogue in (EPI_STORE_F32, EPI_RESIDUAL) else w.dtype
     assert tuple(c.shape) == (m, want_cols) and c.dtype == want_dtype, (c.shape, c.dtype, m, want_cols, want_dtype)

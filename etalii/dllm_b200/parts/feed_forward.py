@@ -206,10 +206,14 @@ class ActivationMLP:
             h = h.tensor()
         rows = h.shape[0]
         ff = self.intermediate_size
-        pre = rt.ws.buffer("ffn_pre", (rows, self.w_up.shape[0]), torch.float32)
-        ops.gemm(pre, h, self.w_up, ops.EPI_STORE_F32)
         act = rt.ws.buffer("ffn_act", (rows, self.padded), rt.dtype)
-        ops.bias_act(act, pre, self.b_up, ops.ACTIVATIONS[self.activation], ff, self.token_gate)
+        if rt.dtype == torch.bfloat16 and self.activation == "relu_squared" and self.b_up is None and \
+                not self.token_gate and self.padded == ff and ops.glu_clamped_fuses(rows, *self.w_up.shape):
+            ops.gemm(act, h, self.w_up, ops.EPI_RELU_SQUARED)  # (a decode-sized product ends in the activation)
+        else:
+            pre = rt.ws.buffer("ffn_pre", (rows, self.w_up.shape[0]), torch.float32)
+            ops.gemm(pre, h, self.w_up, ops.EPI_STORE_F32)
+            ops.bias_act(act, pre, self.b_up, ops.ACTIVATIONS[self.activation], ff, self.token_gate)
         ops.gemm(residual, act, self.w_down, epilogue)
         if self.b_down is not None:
             ops.add_row(residual, self.b_down)

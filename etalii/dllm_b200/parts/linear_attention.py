@@ -429,8 +429,14 @@ class StateSpaceDuality:
         ops.state_space_prepare(prepared, aux, rows, self.taps, self.conv_bias, self.a_log, self.dt_bias, history,
                                 self.heads, self.groups, self.dim, self.vdim, batch)
         read = rt.ws.buffer("mixer_read", (n, self.inner), torch.float32)
+        segment = ops.state_space_segment(batch, self.heads, self.vdim)
+        left = decay = None
+        if segment:  # (a prompt's stretches side by side, each from what those before it leave)
+            matrices = batch.n_seqs * -(-batch.max_new // segment) * self.heads
+            left = rt.ws.buffer("segment_state", (matrices * self.vdim * self.padded,), torch.float32)
+            decay = rt.ws.buffer("segment_decay", (matrices,), torch.float32)
         ops.state_space_scan(read, prepared, aux, self.skip, self.heads, self.groups, self.padded, self.vdim, matrix,
-                             batch)
+                             batch, segment, left, decay)
         if operand is not None:
             ops.gate_norm(operand[0], read, rows, self.weight, self.norm_groups, self.eps, out_at=operand[1],
                           fill=_in_pieces(self.inner) - self.inner)

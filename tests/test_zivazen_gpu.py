@@ -681,11 +681,16 @@ def test_state_space_part_in_pieces(name, dtype, shape):
 
 
 @pytest.mark.parametrize("name,dtype", DTYPES)
-@pytest.mark.parametrize("count", [1, 3, 70])
-def test_state_space_of_long_portions(name, dtype, count):
-    """Prompts of hundreds of tokens, alone and many at once (other launch shapes), with portions whose ends fall anywhere."""
-    rt = _runtime(dtype)
-    m, width = _ssm(6, 20, 24, 2, 4, 1), 64
+@pytest.mark.parametrize("count,segment", [(1, 0), (1, None), (1, 16), (3, 48), (3, None), (3, 4096), (70, 0), (70, 64)])
+@pytest.mark.parametrize("m", [_ssm(6, 20, 24, 2, 4, 1), _ssm(2, 9, 130, 1, 2, 1)], ids=["narrow", "wide"])
+def test_state_space_of_long_portions(monkeypatch, name, dtype, count, segment, m):
+    """Prompts of hundreds of tokens, alone and many at once (other launch shapes), with portions whose ends fall anywhere;
+    token after token, or in segments side by side (of 16 tokens, as the part chooses, longer than any prompt)."""
+    from etalii.dllm_b200.kernels import ops
+
+    if segment is not None:
+        monkeypatch.setattr(ops, "state_space_segment", lambda *a: segment)
+    rt, width = _runtime(dtype), 64
     weights = _state_space_weights(8, width, m, a_log=(-2.0, 1.0))
     part = _state_space(width, m)
     part.bind(weights, rt)
@@ -742,6 +747,21 @@ def test_the_convolution_reaches_back_by_its_taps_and_no_further(name, dtype, co
         got, moved = run(other), np.abs(run(other) - run(h)).max(axis=1)
         assert rel_error(got, _plain_state_space(weights, m, other, 1e-2)) <= PART_TOL[dtype]
         assert [i for i in range(55) if moved[i] > 1e-3] == list(range(marked, min(55, marked + conv)))
+
+
+@pytest.mark.parametrize("rows", [1, 8, 16, 40, 64])
+@pytest.mark.parametrize("width,ff", [(96, 40), (512, 1024), (1024, 2048)])
+def test_squared_relu_inside_the_product(rows, width, ff):
+    from etalii.dllm_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(rows)
+    if not ops.glu_clamped_fuses(rows, ff, width):
+        pytest.skip("these sizes take another product kernel")
+    h, w = torch.randn(rows, width, generator=g).to(torch.bfloat16), _bf16(g, ff, width)
+    out = torch.empty(rows, ff, dtype=torch.bfloat16, device=DEV)
+    ops.gemm(out, _dev(h), _dev(w), ops.EPI_RELU_SQUARED)
+    want = np.maximum(h.double().numpy() @ w.double().numpy().T, 0) ** 2
+    assert rel_error(host(out), want) < 6e-3
 
 
 # ---- both branches side by side -------------------------------------------------------------------------------------------------
