@@ -1210,10 +1210,12 @@ def zivazen_rooflines(row: dict, size: dict, batch: int, peak: dict, contexts: l
                                 if "attention" in label and mask in label), None) for phase in ("prefill", "decode"))
         put(name + "_prefill_bf16_frac", 2 * h * 2 * d * seen, prompt, "bf16")
         put(name + "_decode_hbm_frac", 2 * sum(past) * g * 2 * d, single, "hbm")
-    for model, scan, columns in (("zivazen", "state_space_scan", d), ("revupel", "gated_scan", d + 1),
-                                 ("tisalorn", "decay_scan", d)):
-        put(f"{model}_scan_decode_hbm_frac", 2 * 4 * batch * h * columns * d, row[model]["decode_kernels"].get(scan), "hbm")
-        put(f"{model}_scan_prefill_fp32_frac", 2 * 2 * n * h * columns * d, row[model]["prefill_kernels"].get(scan), "fp32")
+    for model, scans, columns in (("zivazen", ("state_space_chunks", "state_space_scan"), d), ("revupel", ("gated_scan",), d + 1),
+                                  ("tisalorn", ("decay_scan",), d)):
+        put(f"{model}_scan_decode_hbm_frac", 2 * 4 * batch * h * columns * d, _first(row[model]["decode_kernels"], *scans),
+            "hbm")
+        put(f"{model}_scan_prefill_fp32_frac", 2 * 2 * n * h * columns * d, _first(row[model]["prefill_kernels"], *scans),
+            "fp32")
     touched = min(8, 2 * batch)
     for model in ("zivazen", "revupel"):
         for phase, work, unit in (("decode", 2 * touched * 2 * (ff // 4) * width, "hbm"),

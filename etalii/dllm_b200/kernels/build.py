@@ -36,6 +36,7 @@ SOURCES = {
     "attention_prefill_tcgen05": "attention_prefill_tcgen05.cu",
     "attention_decode_static": "attention_decode_static.cu",
     "recurrent": "recurrent.cu",
+    "state_space_chunks": "state_space_chunks.cu",
     "diff_attention": "diff_attention.cu",
     "diff_attention_prefill": "diff_attention_prefill.cu",
     "diff_attention_decode": "diff_attention_decode.cu",

@@ -88,6 +88,9 @@ _prototypes = {
     ("recurrent", "dllm_state_space_scan"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                              c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                              c_void_p, c_void_p, c_void_p, c_void_p],
+    ("state_space_chunks", "dllm_state_space_chunks"): [
+        c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+        c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     ("recurrent", "dllm_state_space_prepare"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                 c_int, c_void_p, c_void_p, c_int, c_void_p],
@@ -1490,8 +1493,9 @@ def state_space_prepare(prepared: torch.Tensor, aux: torch.Tensor, rows: torch.T
 
 def state_space_segment(batch, heads: int, vdim: int) -> int:
     """Into stretches of how many tokens a step's prompts are cut for the state-space scan (0: not at all): where the step's
-    own blocks (16 columns of a head and sequence each) would leave the device waiting for one token after the other."""
-    if batch.max_new < 256 or batch.n_seqs * heads * -(-vdim // 16) >= 8 * _multiprocessors():
+    own blocks (16 columns of a head and sequence each) are fewer than its multiprocessors. (Measured on a prompt of 2,048
+    tokens: 64 blocks 127 us against 235, 128 blocks 262 against 305, 256 blocks 482 against 392.)"""
+    if batch.max_new < 256 or batch.n_seqs * heads * -(-vdim // 16) > _multiprocessors():
         return 0
     return SCAN_SEGMENT
 
@@ -1522,6 +1526,39 @@ def state_space_scan(out: torch.Tensor, prepared: torch.Tensor, aux: torch.Tenso
         batch.cu_seqlens.data_ptr(), batch.slots.data_ptr(), batch.n_seqs, int(batch.max_new), int(segment), segments,
         ptr(segment_state), ptr(segment_decay), out.data_ptr(), _stream()), "state_space_scan",
         lambda: f"dim={padded} (a multiple of 4, at most 256), segments of {segment} (a multiple of 16)")
+
+
+STATE_SPACE_CHUNK = 64
+STATE_SPACE_CHUNKS_FROM = 96
+"""New tokens of a step's longest portion from which its state-space scan runs as products over chunks."""
+STATE_SPACE_SCRATCH = 256 << 20
+"""Most floats that the states in front of all chunks may take (a step of many long prompts has scan blocks enough)."""
+
+
+def state_space_chunks_supported(dtype, padded: int, vdim: int, heads: int, batch) -> bool:
+    """Whether a step's state-space scan runs as tensor-core products over chunks (bfloat16 models)."""
+    chunks = batch.n_seqs * -(-batch.max_new // STATE_SPACE_CHUNK)
+    return dtype == torch.bfloat16 and padded <= 128 and vdim % 4 == 0 and batch.max_new >= STATE_SPACE_CHUNKS_FROM and \
+        chunks <= 65535 and chunks * heads * vdim * padded <= STATE_SPACE_SCRATCH
+
+
+def state_space_chunks(out: torch.Tensor, prepared: torch.Tensor, aux: torch.Tensor, a_log: torch.Tensor,
+                       skip: torch.Tensor, heads: int, groups: int, padded: int, vdim: int, state: torch.Tensor, batch,
+                       starts: torch.Tensor, decays: torch.Tensor) -> None:
+    """`state_space_scan` as products over chunks of 64 tokens (sizes: `state_space_chunks_supported`): the step sizes come
+    from aux, the decays from them and a_log. starts, decays: float32 scratch of sequences x ceil(longest / 64) x heads
+    matrices [vdim, padded] and as many numbers."""
+    _cuda(out, prepared, aux, a_log, skip, state, starts, decays)
+    assert all(t.dtype == torch.float32 for t in (out, prepared, aux, a_log, skip, state, starts, decays))
+    assert tuple(state.shape[1:]) == (heads, vdim, padded) and out.shape[1] == heads * vdim and skip.numel() == heads
+    assert prepared.shape[1] == heads * vdim + 2 * groups * padded and aux.shape[1] == 2 * heads and a_log.numel() == heads
+    matrices = batch.n_seqs * -(-batch.max_new // STATE_SPACE_CHUNK) * heads
+    assert starts.numel() >= matrices * vdim * padded and decays.numel() >= matrices
+    _check(_fn("state_space_chunks", "dllm_state_space_chunks")(
+        prepared.data_ptr(), prepared.shape[1], aux.data_ptr(), aux.shape[1], a_log.data_ptr(), skip.data_ptr(), heads,
+        groups, padded, vdim, state.data_ptr(), starts.data_ptr(), decays.data_ptr(), batch.cu_seqlens.data_ptr(),
+        batch.slots.data_ptr(), batch.n_seqs, int(batch.max_new), out.data_ptr(), _stream()), "state_space_chunks",
+        lambda: f"dim={padded} (a multiple of 4, at most 128), vdim={vdim} (a multiple of 4)")
 
 
 def gate_norm(out: torch.Tensor, y: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, parts: int,

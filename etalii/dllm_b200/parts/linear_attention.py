@@ -429,14 +429,19 @@ class StateSpaceDuality:
         ops.state_space_prepare(prepared, aux, rows, self.taps, self.conv_bias, self.a_log, self.dt_bias, history,
                                 self.heads, self.groups, self.dim, self.vdim, batch)
         read = rt.ws.buffer("mixer_read", (n, self.inner), torch.float32)
-        segment = ops.state_space_segment(batch, self.heads, self.vdim)
-        left = decay = None
-        if segment:  # (a prompt's stretches side by side, each from what those before it leave)
-            matrices = batch.n_seqs * -(-batch.max_new // segment) * self.heads
-            left = rt.ws.buffer("segment_state", (matrices * self.vdim * self.padded,), torch.float32)
-            decay = rt.ws.buffer("segment_decay", (matrices,), torch.float32)
-        ops.state_space_scan(read, prepared, aux, self.skip, self.heads, self.groups, self.padded, self.vdim, matrix,
-                             batch, segment, left, decay)
+        chunks = ops.state_space_chunks_supported(rt.dtype, self.padded, self.vdim, self.heads, batch)
+        stretch = ops.STATE_SPACE_CHUNK if chunks else ops.state_space_segment(batch, self.heads, self.vdim)
+        starts = decay = None
+        if stretch:  # (a prompt's stretches side by side, each from what those before it leave)
+            matrices = batch.n_seqs * -(-batch.max_new // stretch) * self.heads
+            starts = rt.ws.buffer("stretch_starts", (matrices * self.vdim * self.padded,), torch.float32)
+            decay = rt.ws.buffer("stretch_decays", (matrices,), torch.float32)
+        if chunks:
+            ops.state_space_chunks(read, prepared, aux, self.a_log, self.skip, self.heads, self.groups, self.padded,
+                                   self.vdim, matrix, batch, starts, decay)
+        else:
+            ops.state_space_scan(read, prepared, aux, self.skip, self.heads, self.groups, self.padded, self.vdim, matrix,
+                                 batch, stretch, starts, decay)
         if operand is not None:
             ops.gate_norm(operand[0], read, rows, self.weight, self.norm_groups, self.eps, out_at=operand[1],
                           fill=_in_pieces(self.inner) - self.inner)
@@ -446,7 +451,7 @@ class StateSpaceDuality:
         ops.gemm(residual, gated, self.w_o, epilogue)
 
     def kernel_libraries(self, rt) -> set[str]:
-        return _libraries(rt)
+        return _libraries(rt) | ({"state_space_chunks"} if rt.dtype == torch.bfloat16 else set())
 
 
 register_part("mixer", "state_space_duality", StateSpaceDuality)

@@ -690,6 +690,7 @@ def test_state_space_of_long_portions(monkeypatch, name, dtype, count, segment, 
 
     if segment is not None:
         monkeypatch.setattr(ops, "state_space_segment", lambda *a: segment)
+        monkeypatch.setattr(ops, "STATE_SPACE_CHUNKS_FROM", 1 << 30)
     rt, width = _runtime(dtype), 64
     weights = _state_space_weights(8, width, m, a_log=(-2.0, 1.0))
     part = _state_space(width, m)
@@ -701,6 +702,54 @@ def test_state_space_of_long_portions(monkeypatch, name, dtype, count, segment, 
     got = _feed(PartHarness(part.cache_need(), dtype, count), _mixer_call(part, rt), sequences, schedule, width)
     for i in range(0, count, 9):
         assert rel_error(got[i], _plain_state_space(weights, m, sequences[i])) <= PART_TOL[dtype]
+
+
+CHUNK_SHAPES = {
+    "one_tile": _ssm(4, 32, 32, 2, 3, 1),
+    "two_tiles": _ssm(6, 68, 64, 3, 4, 2),
+    "real": _ssm(2, 128, 128, 1, 4, 1),
+    "uneven": _ssm(3, 100, 76, 1, 2, 3),
+    "narrow": _ssm(5, 4, 5, 5, 1, 1),
+}
+
+
+@pytest.mark.parametrize("shape", sorted(CHUNK_SHAPES))
+@pytest.mark.parametrize("lengths", [[1], [64], [65, 1, 63, 128], [500, 130, 2]])
+@pytest.mark.parametrize("a_log,dt_bias", [((-1.0, 1.2), (-1.5, 1.0)), ((-7.0, 0.1), (-1.0, 0.3)), ((2.5, 0.5), (2.0, 1.0))],
+                         ids=["mixed", "slow", "fast"])
+def test_chunks_as_products_give_what_the_scan_gives(shape, lengths, a_log, dt_bias):
+    """The tensor-core form beside the token-by-token form from the same prepared rows and the same non-zero state: outputs
+    and final states, with decays that keep nearly all, nearly nothing and anything between, closer than one bfloat16
+    rounding would allow; slots that are not of the step stay as they are."""
+    from etalii.dllm_b200.engine.batch import BatchBuffers
+    from etalii.dllm_b200.kernels import ops
+
+    m = CHUNK_SHAPES[shape]
+    heads, groups, vdim, padded = m["heads"], m["groups"], m["vdim"], -(-m["state"] // 4) * 4
+    g = torch.Generator().manual_seed(len(shape) + sum(lengths))
+    slots = [3, 0, 4, 1][:len(lengths)]
+    batch = BatchBuffers(DEV).fill(slots, [[0] * n for n in lengths], [0] * len(lengths), [[] for _ in lengths])
+    n = sum(lengths)
+    rand = lambda *size: torch.randn(*size, generator=g)  # noqa: E731
+    prepared = _dev(rand(n, heads * vdim + 2 * groups * padded))
+    log = a_log[0] + a_log[1] * rand(heads)
+    steps = torch.nn.functional.softplus(dt_bias[0] + dt_bias[1] * rand(n, heads))
+    aux = _dev(torch.cat([torch.exp(-torch.exp(log) * steps), steps], dim=1))
+    skip, before = _dev(rand(heads)), rand(5, heads, vdim, padded)
+    states, outs = [], []
+    for chunks in (False, True):
+        state, out = _dev(before), torch.full((n, heads * vdim), 9.0, device=DEV)
+        if chunks:
+            matrices = len(lengths) * -(-max(lengths) // 64) * heads
+            ops.state_space_chunks(out, prepared, aux, _dev(log), skip, heads, groups, padded, vdim, state, batch,
+                                   torch.empty(matrices * vdim * padded, device=DEV), torch.empty(matrices, device=DEV))
+        else:
+            ops.state_space_scan(out, prepared, aux, skip, heads, groups, padded, vdim, state, batch)
+        states.append(host(state))
+        outs.append(host(out))
+    assert rel_error(outs[1], outs[0]) < 4e-5 and rel_error(states[1], states[0]) < 4e-5
+    untouched = [i for i in range(5) if i not in slots]
+    assert (states[1][untouched] == before.numpy()[untouched]).all()
 
 
 @pytest.mark.parametrize("name,dtype", DTYPES)
