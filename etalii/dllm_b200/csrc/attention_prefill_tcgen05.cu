@@ -54,7 +54,7 @@ struct Barriers {
   uint64_t s_full[2], s_empty[2], p_full[2], o_full[2], o_empty[2];
 };
 
-template <int HD, bool OPTIONS>
+template <int HD, bool OPTIONS, bool CAPPED>
 __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, bf16* __restrict__ out,
     KvLayout cache, const int* __restrict__ tile_seq, const int* __restrict__ tile_first,
@@ -190,8 +190,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
     for (int d = 0; d < HD; ++d) o[d] = 0.f;
     float m_run = -INFINITY, l_run = 0.f, corr_saved = 1.f;
     bool ok = true;
-    const ScoreCap score(scale_log2 / SCORE_LOG2E, OPTIONS ? options.cap : 0.f);
-    const bool capped = OPTIONS && options.cap > 0.f;
+    const ScoreCap score(scale_log2 / SCORE_LOG2E, CAPPED ? options.cap : 0.f);
     // fold step i's output into the running one: O = O * corr + P V
     auto consume = [&](int i, float corr) -> bool {
       const int ob = i & 1;
@@ -250,7 +249,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
           tmem_wait_ld();
           if (c + 16 < BKV) tmem_load16_nowait(s_addr + (unsigned)(c + 16), v[cur ^ 1]);
           float p[16];  // first the scores as they enter the exponential
-          if (OPTIONS && capped) {
+          if (CAPPED) {
             float largest[2] = {0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < 16; ++i) largest[i & 1] = fmaxf(largest[i & 1], fabsf(__uint_as_float(v[cur][i])));
@@ -296,7 +295,7 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
         }
         tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));  // of the raw scores; now in the scaled log2 domain
         // (the cap keeps the scores' order, so the largest one's capped value is the largest)
-        if (OPTIONS && capped) tile_max = tile_max == -INFINITY ? -INFINITY : score.any(tile_max);
+        if (CAPPED) tile_max = tile_max == -INFINITY ? -INFINITY : score.any(tile_max);
         else tile_max *= scale_log2;
         row_sum = (sum[0] + sum[1]) + (sum[2] + sum[3]);
       };
@@ -379,19 +378,19 @@ __global__ void __launch_bounds__(Shape<HD>::THREADS, 1) prefill_tcgen05_kernel(
   if (warp == SOFT_WARPS + 1) tmem_dealloc(tmem_base, TMEM_COLS);
 }
 
-template <int HD, bool OPTIONS>
+template <int HD, bool OPTIONS, bool CAPPED>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, void* out, const KvLayout& cache, const int* tile_seq,
            const int* tile_first, const int* cu_seqlens, const int* start, const int* slots, int tiles, int heads,
            float scale, int window, int* status, const ScoreOptions& options, cudaStream_t stream) {
   typedef Shape<HD> S;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(prefill_tcgen05_kernel<HD, OPTIONS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(prefill_tcgen05_kernel<HD, OPTIONS, CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)S::SMEM) != cudaSuccess)
       return DLLM_LAUNCH_FAILED;
     configured = true;
   }
-  return dllm_launch_pdl(prefill_tcgen05_kernel<HD, OPTIONS>, dim3(tiles, heads), dim3(S::THREADS), S::SMEM, stream, map_q,
+  return dllm_launch_pdl(prefill_tcgen05_kernel<HD, OPTIONS, CAPPED>, dim3(tiles, heads), dim3(S::THREADS), S::SMEM, stream, map_q,
                          map_kv, (bf16*)out, cache, tile_seq, tile_first, cu_seqlens, start, slots, heads,
                          scale * SCORE_LOG2E, window, status, options);
 }
@@ -413,11 +412,13 @@ int run(void* out, const void* q, int tokens, void* cache_base, long long cache_
       !make_map(&map_kv, cache_base, cache_pages * 2 * kv_heads * BKV, head_dim, BKV))
     return DLLM_LAUNCH_FAILED;
   KvLayout cache{cache_base, page_table, max_pages, page_size, kv_heads, head_dim};
-  if (head_dim == 64)
-    return launch<64, OPTIONS>(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale,
-                      window, status, options, stream);
-  return launch<128, OPTIONS>(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale,
-                     window, status, options, stream);
+  auto go = [&](auto run_one) {
+    return run_one(map_q, map_kv, out, cache, tile_seq, tile_first, cu_seqlens, start, slots, tiles, heads, scale, window,
+                   status, options, stream);
+  };
+  const bool capped = OPTIONS && options.cap > 0.f;  // (a kernel of its own: without a cap a score is one multiply-add)
+  if (head_dim == 64) return capped ? go(launch<64, OPTIONS, OPTIONS>) : go(launch<64, OPTIONS, false>);
+  return capped ? go(launch<128, OPTIONS, OPTIONS>) : go(launch<128, OPTIONS, false>);
 }
 }  // namespace
 

@@ -17,7 +17,7 @@
 // A warp owns a few output values: its lanes split the reduction in 16-byte pieces (the rows' loads asked for together),
 // sums in float32. These kernels read an
 // expert's weights once per token that chose it, which is what a step of few tokens needs.
-#include "common.cuh"
+#include "expert_unit.cuh"
 
 namespace {
 constexpr int WARPS = 8;
@@ -279,17 +279,9 @@ __global__ void __launch_bounds__(WARPS * 32) moe_up_kernel(
 #pragma unroll
   for (int r = 0; r < 2 * UP_PER_WARP; ++r) sums[r] = warp_sum(sums[r]);
   if (lane < UP_PER_WARP && f + lane < ff) {
-    float g = fminf(lane == 0 ? sums[0] : sums[2], limit);
-    float u = fminf(fmaxf(lane == 0 ? sums[1] : sums[3], -limit), limit);
-    act[(size_t)a * ff + f + lane] = from_float<T>(g / (1.0f + expf(-alpha * g)) * (u + shift));
+    act[(size_t)a * ff + f + lane] = from_float<T>(gated_unit(lane == 0 ? sums[0] : sums[2], lane == 0 ? sums[1] : sums[3],
+                                                              limit, alpha, shift));
   }
-}
-
-__device__ __forceinline__ float plain_activation(float z, int kind) {
-  if (kind == 1) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
-  if (kind == 2) return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
-  float r = fmaxf(z, 0.f);
-  return r * r;
 }
 
 constexpr int PLAIN_PER_WARP = 4;  // activated values a warp of moe_up_plain owns

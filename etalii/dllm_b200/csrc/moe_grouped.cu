@@ -10,7 +10,7 @@
 // (tiles past the last expert's rows return at once: the grid is sized for the worst case). Operands go through three
 // cp.async stages of 64 reduction values; eight warps of 64 x 32 outputs each. A pair's result does not depend on its
 // place or on its tile mates, so the arbitrary order inside an expert's list changes no bit.
-#include "common.cuh"
+#include "expert_unit.cuh"
 
 namespace {
 typedef __nv_bfloat16 bf16;
@@ -77,13 +77,6 @@ struct GroupedArgs {
   float limit, alpha, shift;
   int kind;               // EPI_ACT: 1 gelu (erf), 2 gelu (tanh form), 3 the square of relu
 };
-
-__device__ __forceinline__ float plain_activation(float z, int kind) {
-  if (kind == 1) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
-  if (kind == 2) return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
-  float r = fmaxf(z, 0.f);
-  return r * r;
-}
 
 template <int EPI>
 __global__ void __launch_bounds__(THREADS) grouped_kernel(GroupedArgs g) {
@@ -186,9 +179,8 @@ __global__ void __launch_bounds__(THREADS) grouped_kernel(GroupedArgs g) {
         for (int nj = 0; nj < 4; ++nj) {
           int n = n0 + warp_n * 32 + nj * 8 + tq * 2;  // (even: gate at n, up at n + 1)
           if (n + 1 < g.n) {
-            float gate = fminf(acc[mi][nj][half * 2], g.limit);
-            float up = fminf(fmaxf(acc[mi][nj][half * 2 + 1], -g.limit), g.limit);
-            dst[n / 2] = __float2bfloat16_rn(gate / (1.0f + expf(-g.alpha * gate)) * (up + g.shift));
+            dst[n / 2] = __float2bfloat16_rn(gated_unit(acc[mi][nj][half * 2], acc[mi][nj][half * 2 + 1], g.limit, g.alpha,
+                                                        g.shift));
           }
         }
       } else if (EPI == EPI_ACT) {
@@ -225,6 +217,27 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(float* __restrict__ ou
     for (int k = 0; k < top; ++k) sum = fmaf(weights[t * top + k], y[(t * top + k) * width + n], sum);
     out[i] = accumulate ? out[i] + sum : sum;
   }
+}
+
+// (width a multiple of 4: 16 bytes a thread)
+__global__ void __launch_bounds__(256) moe_combine_fours_kernel(float4* __restrict__ out, const float4* __restrict__ y,
+                                                                const float* __restrict__ weights, int fours, int top,
+                                                                int accumulate) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, n = blockIdx.y * blockDim.x + threadIdx.x;
+  if (n >= fours) return;
+  const size_t at = (size_t)t * fours + n;
+  const float4 before = accumulate ? out[at] : make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const float w = weights[t * top + k];
+    const float4 v = y[((size_t)t * top + k) * fours + n];
+    sum.x = fmaf(w, v.x, sum.x); sum.y = fmaf(w, v.y, sum.y); sum.z = fmaf(w, v.z, sum.z); sum.w = fmaf(w, v.w, sum.w);
+  }
+  if (accumulate) { sum.x += before.x; sum.y += before.y; sum.z += before.z; sum.w += before.w; }
+  out[at] = sum;
 }
 
 template <int EPI>
@@ -291,6 +304,9 @@ DLLM_EXPORT int dllm_moe_combine(float* out, const float* y, const float* weight
                                  int accumulate, cudaStream_t stream) {
   if (tokens <= 0) return DLLM_OK;
   if (width <= 0 || top <= 0) return DLLM_UNSUPPORTED_SIZE;
+  if ((width & 3) == 0 && (((uintptr_t)out | (uintptr_t)y) & 15) == 0)
+    return dllm_launch_pdl(moe_combine_fours_kernel, dim3(tokens, (width / 4 + 255) / 256), dim3(256), 0, stream,
+                           (float4*)out, (const float4*)y, weights, width / 4, top, accumulate);
   long long total = (long long)tokens * width;
   int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
   return dllm_launch_pdl(moe_combine_kernel, dim3(blocks), dim3(256), 0, stream, out, y, weights, width, top, total,

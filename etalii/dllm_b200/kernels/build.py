@@ -46,6 +46,7 @@ SOURCES = {
     "sigmoid_attention_tiled": "sigmoid_attention_tiled.cu",
     "moe": "moe.cu",
     "moe_grouped": "moe_grouped.cu",
+    "moe_grouped_tcgen05": "moe_grouped_tcgen05.cu",
     "sink_attention": "sink_attention.cu",
     "sink_attention_prefill": "sink_attention_prefill.cu",
     "sink_attention_decode": "sink_attention_decode.cu",

@@ -162,6 +162,12 @@ _prototypes = {
                                                    c_void_p, c_void_p, c_int, c_void_p],
     ("moe_grouped", "dllm_moe_grouped_down"): [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                                c_void_p, c_void_p, c_void_p],
+    ("moe_grouped_tcgen05", "dllm_moe_gather"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    ("moe_grouped_tcgen05", "dllm_moe_grouped_tcgen05_up"): [
+        c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_float, c_float, c_float, c_void_p,
+        c_void_p],
+    ("moe_grouped_tcgen05", "dllm_moe_grouped_tcgen05_down"): [
+        c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     ("moe_grouped", "dllm_moe_combine"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     ("elementwise", "dllm_concat_restart"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     ("recurrent", "dllm_decay_scan"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
@@ -1260,14 +1266,45 @@ def moe_grouped_supported(tokens: int, dtype, width: int, ff: int) -> bool:
     return dtype == torch.bfloat16 and tokens > MOE_GROUPED_FROM and width % 8 == 0 and ff % 8 == 0
 
 
+MOE_TCGEN05_FROM = 1 << 17
+"""Values of an expert's matrix from which a grouped step's products run on the 5th-generation tensor cores: below, tiles of
+128 x 256 are mostly empty (the products of 2,048 tokens, two of eight experts of 4096 x 2752: 250 us against 689, of 1024 x
+704: 57 against 81; of 128 tokens and 2048 x 1408: 55 against 87; of 1,117 tokens and 320 x 64: 33 against 28)."""
+
+
+def moe_tcgen05_supported(width: int, ff: int) -> bool:
+    """Whether a grouped step's products run on the 5th-generation tensor cores."""
+    return width % 8 == 0 and ff % 8 == 0 and width * ff >= MOE_TCGEN05_FROM
+
+
+def _moe_products_tcgen05(y: torch.Tensor, rows: torch.Tensor, h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
+                          act: torch.Tensor, offsets: torch.Tensor, place_pair: torch.Tensor, top: int, kind: int,
+                          limit: float = 0.0, alpha: float = 0.0, shift: float = 0.0) -> None:
+    """The activations in expert order, then both products of every expert (`kind` 0: the gated unit, else an activation)."""
+    _cuda(rows)
+    tokens, width = h.shape
+    experts, ff, pairs = w_down.shape[0], w_down.shape[2], tokens * int(top)
+    assert rows.dtype == torch.bfloat16 and rows.numel() >= pairs * width
+    stream, status = _stream(), _status_word().data_ptr()
+    _check(_fn("moe_grouped_tcgen05", "dllm_moe_gather")(rows.data_ptr(), h.data_ptr(), place_pair.data_ptr(), width,
+                                                         int(top), pairs, stream), "moe_gather")
+    _check(_fn("moe_grouped_tcgen05", "dllm_moe_grouped_tcgen05_up")(
+        act.data_ptr(), rows.data_ptr(), width, w_up.data_ptr(), ff, experts, pairs, offsets.data_ptr(), kind, float(limit),
+        float(alpha), float(shift), status, stream), "moe_grouped_up", lambda: f"width={width} ff={ff} (multiples of 8)")
+    _check(_fn("moe_grouped_tcgen05", "dllm_moe_grouped_tcgen05_down")(
+        y.data_ptr(), act.data_ptr(), ff, w_down.data_ptr(), width, experts, pairs, offsets.data_ptr(),
+        place_pair.data_ptr(), status, stream), "moe_grouped_down", lambda: f"width={width} ff={ff} (multiples of 8)")
+
+
 def moe_experts_grouped(out: torch.Tensor, h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                         chosen: torch.Tensor, weights: torch.Tensor, top: int, limit: float, alpha: float, shift: float,
                         offsets: torch.Tensor, place_pair: torch.Tensor, act: torch.Tensor, y: torch.Tensor,
-                        accumulate: bool = False) -> None:
+                        accumulate: bool = False, sorted_rows: torch.Tensor | None = None) -> None:
     """What `moe_up` and `moe_down` compute, for many tokens (bfloat16): the (token, choice) pairs are put in expert
     order on the device, every expert's rows run as tile products on the tensor cores (gate/up with the gated unit in
     the epilogue, then down, scattered back by pair), and a last kernel forms each token's weighted sum. Four launches
-    whose shapes depend on the sizes only. Scratch: offsets [experts + 1] and place_pair [pairs] int32, act [pairs, ff]
+    whose shapes depend on the sizes only; with `sorted_rows` (bfloat16 [pairs, width]) the activations are first put in
+    expert order there and the products run on the 5th-generation tensor cores (`moe_tcgen05_supported`). Scratch: offsets [experts + 1] and place_pair [pairs] int32, act [pairs, ff]
     bfloat16, y [pairs, width] float32."""
     _cuda(out, h, w_gate_up, w_down, chosen, weights, offsets, place_pair, act, y)
     tokens, width = h.shape
@@ -1283,13 +1320,16 @@ def moe_experts_grouped(out: torch.Tensor, h: torch.Tensor, w_gate_up: torch.Ten
     _check(_fn("moe_grouped", "dllm_moe_sort")(chosen.data_ptr(), pairs, experts, offsets.data_ptr(),
                                                place_pair.data_ptr(), stream), "moe_sort",
            lambda: f"experts={experts} (at most 256)")
-    _check(_fn("moe_grouped", "dllm_moe_grouped_up")(
-        act.data_ptr(), h.data_ptr(), width, w_gate_up.data_ptr(), ff, experts, int(top), tokens, offsets.data_ptr(),
-        place_pair.data_ptr(), float(limit), float(alpha), float(shift), stream), "moe_grouped_up",
-        lambda: f"width={width} (a multiple of 8)")
-    _check(_fn("moe_grouped", "dllm_moe_grouped_down")(
-        y.data_ptr(), act.data_ptr(), ff, w_down.data_ptr(), width, experts, int(top), tokens, offsets.data_ptr(),
-        place_pair.data_ptr(), stream), "moe_grouped_down", lambda: f"ff={ff} (a multiple of 8)")
+    if sorted_rows is not None:
+        _moe_products_tcgen05(y, sorted_rows, h, w_gate_up, w_down, act, offsets, place_pair, top, 0, limit, alpha, shift)
+    else:
+        _check(_fn("moe_grouped", "dllm_moe_grouped_up")(
+            act.data_ptr(), h.data_ptr(), width, w_gate_up.data_ptr(), ff, experts, int(top), tokens, offsets.data_ptr(),
+            place_pair.data_ptr(), float(limit), float(alpha), float(shift), stream), "moe_grouped_up",
+            lambda: f"width={width} (a multiple of 8)")
+        _check(_fn("moe_grouped", "dllm_moe_grouped_down")(
+            y.data_ptr(), act.data_ptr(), ff, w_down.data_ptr(), width, experts, int(top), tokens, offsets.data_ptr(),
+            place_pair.data_ptr(), stream), "moe_grouped_down", lambda: f"ff={ff} (a multiple of 8)")
     _check(_fn("moe_grouped", "dllm_moe_combine")(out.data_ptr(), y.data_ptr(), weights.data_ptr(), width, int(top),
                                                   tokens, 1 if accumulate else 0, stream), "moe_combine")
 
@@ -1297,7 +1337,7 @@ def moe_experts_grouped(out: torch.Tensor, h: torch.Tensor, w_gate_up: torch.Ten
 def moe_plain_experts_grouped(out: torch.Tensor, h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor,
                               chosen: torch.Tensor, weights: torch.Tensor, top: int, kind: int, offsets: torch.Tensor,
                               place_pair: torch.Tensor, act: torch.Tensor, y: torch.Tensor,
-                              accumulate: bool = False) -> None:
+                              accumulate: bool = False, sorted_rows: torch.Tensor | None = None) -> None:
     """`moe_experts_grouped` for experts without a gate matrix: W_down act(W_up h) with the activation `kind` in the
     first product's epilogue. w_up [experts, ff, width], w_down [experts, width, ff]; the same scratch."""
     _cuda(out, h, w_up, w_down, chosen, weights, offsets, place_pair, act, y)
@@ -1314,13 +1354,16 @@ def moe_plain_experts_grouped(out: torch.Tensor, h: torch.Tensor, w_up: torch.Te
     _check(_fn("moe_grouped", "dllm_moe_sort")(chosen.data_ptr(), pairs, experts, offsets.data_ptr(),
                                                place_pair.data_ptr(), stream), "moe_sort",
            lambda: f"experts={experts} (at most 256)")
-    _check(_fn("moe_grouped", "dllm_moe_grouped_up_plain")(
-        act.data_ptr(), h.data_ptr(), width, w_up.data_ptr(), ff, experts, int(top), tokens, offsets.data_ptr(),
-        place_pair.data_ptr(), int(kind), stream), "moe_grouped_up",
-        lambda: f"width={width} (a multiple of 8) ff={ff} (even)")
-    _check(_fn("moe_grouped", "dllm_moe_grouped_down")(
-        y.data_ptr(), act.data_ptr(), ff, w_down.data_ptr(), width, experts, int(top), tokens, offsets.data_ptr(),
-        place_pair.data_ptr(), stream), "moe_grouped_down", lambda: f"ff={ff} (a multiple of 8)")
+    if sorted_rows is not None:
+        _moe_products_tcgen05(y, sorted_rows, h, w_up, w_down, act, offsets, place_pair, top, int(kind))
+    else:
+        _check(_fn("moe_grouped", "dllm_moe_grouped_up_plain")(
+            act.data_ptr(), h.data_ptr(), width, w_up.data_ptr(), ff, experts, int(top), tokens, offsets.data_ptr(),
+            place_pair.data_ptr(), int(kind), stream), "moe_grouped_up",
+            lambda: f"width={width} (a multiple of 8) ff={ff} (even)")
+        _check(_fn("moe_grouped", "dllm_moe_grouped_down")(
+            y.data_ptr(), act.data_ptr(), ff, w_down.data_ptr(), width, experts, int(top), tokens, offsets.data_ptr(),
+            place_pair.data_ptr(), stream), "moe_grouped_down", lambda: f"ff={ff} (a multiple of 8)")
     _check(_fn("moe_grouped", "dllm_moe_combine")(out.data_ptr(), y.data_ptr(), weights.data_ptr(), width, int(top),
                                                   tokens, 1 if accumulate else 0, stream), "moe_combine")
 
@@ -1612,7 +1655,8 @@ def _status_word() -> torch.Tensor:
 
 def raise_if_failed() -> None:
     """Raises if a kernel has set the status word since the last look: a bounded wait on an mbarrier ran out
-    (codes 2-5 the tile product, 12-21 the tcgen05 attention, 32-33 the product that streams through shared memory)
+    (codes 2-5 the tile product, 12-21 the tcgen05 attention, 32-33 the product that streams through shared memory, 42-45
+    the experts' tile products)
     or the embedding met a token outside its table (64). Results computed since are not valid. The word lives in
     pinned host memory, so the look costs no synchronisation; it is meaningful after the host has waited for the
     kernels in question (a `.tolist()`, a copy to the host, a synchronize)."""

@@ -17,6 +17,13 @@ from .registry import build_part, part_factory, register_part
 from .spec import ParamSpec, PartSpec
 
 
+def _sorted_rows(rt, pairs: int, width: int, ff: int) -> torch.Tensor | None:
+    """Room for a grouped step's activations in expert order, where its products want them so."""
+    if not ops.moe_tcgen05_supported(width, ff):
+        return None
+    return rt.ws.buffer("experts_rows", (pairs, width), torch.bfloat16)
+
+
 class ClampedGLUExperts:
     accepts_stream = True
 
@@ -89,7 +96,8 @@ class ClampedGLUExperts:
             places = rt.ws.buffer("experts_places", (n * self.top,), torch.int32)
             pairs_out = rt.ws.buffer("experts_out", (n * self.top, self.hidden_size), torch.float32)
             ops.moe_experts_grouped(residual, h, self.w_gate_up, self.w_down, chosen, weights, self.top, self.limit,
-                                    self.alpha, self.shift, offsets, places, act, pairs_out, accumulate=adds)
+                                    self.alpha, self.shift, offsets, places, act, pairs_out, accumulate=adds,
+                                    sorted_rows=_sorted_rows(rt, n * self.top, self.hidden_size, self.intermediate_size))
         else:
             ops.moe_up(act, h, self.w_gate_up, chosen, self.top, self.limit, self.alpha, self.shift)
             ops.moe_down(residual, act, self.w_down, chosen, weights, self.top, accumulate=adds)
@@ -100,6 +108,8 @@ class ClampedGLUExperts:
         names = {"moe", "elementwise"}
         if rt.dtype == torch.bfloat16 and self.hidden_size % 8 == 0 and self.intermediate_size % 8 == 0:
             names.add("moe_grouped")
+            if ops.moe_tcgen05_supported(self.hidden_size, self.intermediate_size):
+                names.add("moe_grouped_tcgen05")
         if self.shared is not None and hasattr(self.shared, "kernel_libraries"):
             names |= set(self.shared.kernel_libraries(rt))
         return names
@@ -201,7 +211,9 @@ class ActivationExperts:
             places = rt.ws.buffer("experts_places", (n * self.top,), torch.int32)
             pairs_out = rt.ws.buffer("experts_out", (n * self.top, self.hidden_size), torch.float32)
             ops.moe_plain_experts_grouped(residual, h, self.w_up, self.w_down, chosen, weights, self.top, kind, offsets,
-                                          places, act, pairs_out, accumulate=adds)
+                                          places, act, pairs_out, accumulate=adds,
+                                          sorted_rows=_sorted_rows(rt, n * self.top, self.hidden_size,
+                                                                   self.intermediate_size))
         else:
             ops.moe_up_plain(act, h, self.w_up, chosen, self.top, kind)
             ops.moe_down(residual, act, self.w_down, chosen, weights, self.top, accumulate=adds)
@@ -212,6 +224,8 @@ class ActivationExperts:
         names = {"moe", "elementwise"}
         if rt.dtype == torch.bfloat16 and self.hidden_size % 8 == 0 and self.intermediate_size % 8 == 0:
             names.add("moe_grouped")
+            if ops.moe_tcgen05_supported(self.hidden_size, self.intermediate_size):
+                names.add("moe_grouped_tcgen05")
         if self.shared is not None and hasattr(self.shared, "kernel_libraries"):
             names |= set(self.shared.kernel_libraries(rt))
         return names

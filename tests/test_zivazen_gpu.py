@@ -206,6 +206,52 @@ def test_mixture_of_experts(name, dtype, rows, width, ff, shared):
     assert np.sort(errors)[int(0.95 * (rows - 1))] <= PART_TOL[dtype]  # (a row with a close call may choose otherwise)
 
 
+@pytest.mark.parametrize("gated", [False, True])
+@pytest.mark.parametrize("tokens,width,ff,experts,top", [(65, 96, 24, 5, 2), (300, 72, 40, 16, 3), (500, 256, 264, 3, 1),
+                                                         (130, 64, 520, 256, 4), (1000, 512, 128, 8, 8)])
+def test_grouped_products_on_either_tensor_core_path(gated, tokens, width, ff, experts, top):
+    """The tcgen05 tiles and the mma.sync tiles: experts without a token and with hundreds, tiles that end inside an
+    expert's rows and columns, all tokens to one expert; equal bit by bit, and close to the plain products."""
+    from etalii.dllm_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(tokens + experts)
+    h, w_up = torch.randn(tokens, width, generator=g).to(torch.bfloat16), \
+        _bf16(g, experts * ff * (2 if gated else 1), width).view(experts, -1, width)
+    w_down = _bf16(g, experts * width, ff).view(experts, width, ff)
+    chosen = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(tokens)]).to(torch.int32)
+    if top == 1:
+        chosen[:] = 1
+    weights, before = torch.rand(tokens, top, generator=g), torch.randn(tokens, width, generator=g)
+    pairs, ints = tokens * top, lambda n: torch.empty(n, dtype=torch.int32, device=DEV)  # noqa: E731
+    outs = []
+    for rows in (None, torch.empty(pairs, width, dtype=torch.bfloat16, device=DEV)):
+        out = _dev(before)
+        scratch = (ints(experts + 1), ints(pairs), torch.empty(pairs, ff, dtype=torch.bfloat16, device=DEV),
+                   torch.empty(pairs, width, device=DEV))
+        common = (out, _dev(h), _dev(w_up), _dev(w_down), _dev(chosen), _dev(weights), top)
+        if gated:
+            ops.moe_experts_grouped(*common, 3.0, 1.5, 0.5, *scratch, accumulate=True, sorted_rows=rows)
+        else:
+            ops.moe_plain_experts_grouped(*common, ops.ACTIVATIONS["relu_squared"], *scratch, accumulate=True,
+                                          sorted_rows=rows)
+        outs.append(host(out))
+    ops.raise_if_failed()
+    assert (outs[0] == outs[1]).all()
+    want = before.double().numpy()
+    hn, up, down = h.double().numpy(), w_up.double().numpy(), w_down.double().numpy()
+    for t in range(0, tokens, 7):
+        for k in range(top):
+            e = int(chosen[t, k])
+            z = up[e] @ hn[t]
+            if gated:
+                gate, u = np.minimum(z[0::2], 3.0), np.clip(z[1::2], -3.0, 3.0)
+                z = gate * P.sigmoid(1.5 * gate) * (u + 0.5)
+            else:
+                z = np.maximum(z, 0) ** 2
+            want[t] += float(weights[t, k]) * (down[e] @ z)
+    assert rel_error(outs[1][::7], want[::7]) < 2e-2
+
+
 # ---- attention with chunks, norms, rotation, a sink of zero and mixed values ---------------------------------------------------
 
 
