@@ -22,7 +22,7 @@
 
 namespace {
 typedef __nv_bfloat16 bf16;
-constexpr int CHUNK = 64, COLS = 64, WARPS = 4, THREADS = WARPS * 32;
+constexpr int CHUNK = 64, COLS = 64, WARPS = 8, THREADS = WARPS * 32;  // (warps: four of sixteen rows, two halves of columns)
 constexpr int LDX = COLS + 8;
 
 struct ChunkArgs {
@@ -77,28 +77,37 @@ __device__ __forceinline__ void split2(float x, float y, unsigned& hi, unsigned&
   lo = *reinterpret_cast<unsigned*>(&l);
 }
 
-// `rows` rows of `cols` values (of a row of `stride` floats) as hi and lo tiles [64][PAD + 8], zeros elsewhere; row r times
-// factor[r] if given.
+// A tile of 64 rows x PAD values on its way from global memory: asked for (`rows` rows of `cols` values, zeros elsewhere),
+// then put into hi and lo tiles [64][PAD + 8]; row r times factor[r] if given.
 template <int PAD>
-__device__ __forceinline__ void load_split(bf16* hi, bf16* lo, const float* src, size_t stride, int rows, int cols,
-                                           const float* factor) {
-  constexpr int FOURS = PAD / 4, LD = PAD + 8;
-#pragma unroll 4
-  for (int i = threadIdx.x; i < 64 * FOURS; i += THREADS) {
-    const int r = i / FOURS, c = 4 * (i % FOURS);
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < rows && c < cols) v = *reinterpret_cast<const float4*>(src + (size_t)r * stride + c);
-    if (factor != nullptr) {
-      const float f = factor[r];
-      v.x *= f; v.y *= f; v.z *= f; v.w *= f;
+struct Tile {
+  static constexpr int FOURS = PAD / 4, LD = PAD + 8, PIECES = 64 * FOURS / THREADS;
+  float4 v[PIECES];
+  __device__ __forceinline__ void ask(const float* src, size_t stride, int rows, int cols) {
+#pragma unroll
+    for (int p = 0; p < PIECES; ++p) {
+      const int i = threadIdx.x + p * THREADS, r = i / FOURS, c = 4 * (i % FOURS);
+      v[p] = r < rows && c < cols ? *reinterpret_cast<const float4*>(src + (size_t)r * stride + c)
+                                  : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    uint2 h, l;
-    split2(v.x, v.y, h.x, l.x);
-    split2(v.z, v.w, h.y, l.y);
-    *reinterpret_cast<uint2*>(hi + r * LD + c) = h;
-    *reinterpret_cast<uint2*>(lo + r * LD + c) = l;
   }
-}
+  __device__ __forceinline__ void put(bf16* hi, bf16* lo, const float* factor = nullptr) {
+#pragma unroll
+    for (int p = 0; p < PIECES; ++p) {
+      const int i = threadIdx.x + p * THREADS, r = i / FOURS, c = 4 * (i % FOURS);
+      float4 x = v[p];
+      if (factor != nullptr) {
+        const float f = factor[r];
+        x.x *= f; x.y *= f; x.z *= f; x.w *= f;
+      }
+      uint2 h, l;
+      split2(x.x, x.y, h.x, l.x);
+      split2(x.z, x.w, h.y, l.y);
+      *reinterpret_cast<uint2*>(hi + r * LD + c) = h;
+      *reinterpret_cast<uint2*>(lo + r * LD + c) = l;
+    }
+  }
+};
 
 // The chunk's tokens: how many, the first one's row; their step sizes, and the running sums of log a (beyond the last
 // token the step size is zero and the sum stays).
@@ -150,17 +159,21 @@ __global__ void __launch_bounds__(THREADS) left_kernel(ChunkArgs a) {
   const int head = blockIdx.y, col0 = blockIdx.x * COLS, group = head / (a.heads / a.groups);
   const int inner = a.heads * a.vdim, cols = min(COLS, a.vdim - col0);
   const float* row = a.prepared + (size_t)chunk.first * a.stride;
+  Tile<N> b;
+  Tile<COLS> x;
+  b.ask(row + inner + group * a.dim, a.stride, chunk.count, a.dim);
+  x.ask(row + head * a.vdim + col0, a.stride, chunk.count, cols);
   sum_logs(a, chunk, head, sums, steps);
-  load_split<N>(b_hi, b_lo, row + inner + group * a.dim, a.stride, chunk.count, a.dim, nullptr);
+  b.put(b_hi, b_lo);
   __syncthreads();
   if (threadIdx.x < CHUNK) factor[threadIdx.x] = steps[threadIdx.x] * expf((float)(sums[CHUNK - 1] - sums[threadIdx.x]));
   __syncthreads();
-  load_split<COLS>(x_hi, x_lo, row + head * a.vdim + col0, a.stride, chunk.count, cols, factor);
+  x.put(x_hi, x_lo, factor);
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, mat = lane >> 3;
-  float acc[N / 8][4];
+  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, mat = lane >> 3, n0 = (threadIdx.x >> 7) * (N / 2);
+  float acc[N / 16][4];
 #pragma unroll
-  for (int i = 0; i < N / 8; ++i)
+  for (int i = 0; i < N / 16; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
 #pragma unroll
@@ -170,9 +183,9 @@ __global__ void __launch_bounds__(THREADS) left_kernel(ChunkArgs a) {
     ldmatrix_x4_trans(xh, x_hi + at);
     ldmatrix_x4_trans(xl, x_lo + at);
 #pragma unroll
-    for (int n = 0; n < N / 16; ++n) {
+    for (int n = 0; n < N / 32; ++n) {
       unsigned bh[4], bl[4];
-      const int from = (k * 16 + (mat & 1) * 8 + (lane & 7)) * LDN + n * 16 + (mat >> 1) * 8;
+      const int from = (k * 16 + (mat & 1) * 8 + (lane & 7)) * LDN + n0 + n * 16 + (mat >> 1) * 8;
       ldmatrix_x4_trans(bh, b_hi + from);
       ldmatrix_x4_trans(bl, b_lo + from);
       mma_split(acc[2 * n], acc[2 * n + 1], xh, xl, bh, bl);
@@ -184,8 +197,8 @@ __global__ void __launch_bounds__(THREADS) left_kernel(ChunkArgs a) {
     const int col = col0 + warp * 16 + (lane >> 2) + 8 * half;
     if (col >= a.vdim) continue;
 #pragma unroll
-    for (int i = 0; i < N / 8; ++i) {
-      const int n = i * 8 + (lane & 3) * 2;
+    for (int i = 0; i < N / 16; ++i) {
+      const int n = n0 + i * 8 + (lane & 3) * 2;
       if (n < a.dim) *reinterpret_cast<float2*>(dst + (size_t)col * a.dim + n) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
     }
   }
@@ -194,8 +207,8 @@ __global__ void __launch_bounds__(THREADS) left_kernel(ChunkArgs a) {
 
 // A thread per four elements of a head's matrix; the chunks' loads are asked for several ahead of the state that walks
 // through them.
-__global__ void __launch_bounds__(256) starts_kernel(ChunkArgs a) {
-  constexpr int AHEAD = 4;
+__global__ void __launch_bounds__(128) starts_kernel(ChunkArgs a) {
+  constexpr int AHEAD = 6;
   pdl_launch_dependents();
   pdl_wait();
   const int head = blockIdx.y, seq = blockIdx.z;
@@ -207,23 +220,32 @@ __global__ void __launch_bounds__(256) starts_kernel(ChunkArgs a) {
   float4* kept = reinterpret_cast<float4*>(a.starts + first * a.vdim * a.dim) + i;
   const size_t step = (size_t)a.heads * fours;
   const float* decays = a.decays + first;
-  float4 s = *whole;
-  for (int p0 = 0; p0 < parts; p0 += AHEAD) {
-    float4 left[AHEAD];
-    float decay[AHEAD];
+  float4 s = *whole, left[2][AHEAD];
+  float decay[2][AHEAD];
+  auto ask = [&](int p0, int buffer) {
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j)
       if (p0 + j < parts) {
-        left[j] = kept[(p0 + j) * step];
-        decay[j] = decays[(size_t)(p0 + j) * a.heads];
+        left[buffer][j] = kept[(p0 + j) * step];
+        decay[buffer][j] = decays[(size_t)(p0 + j) * a.heads];
       }
+  };
+  auto walk = [&](int p0, int buffer) {
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j)
       if (p0 + j < parts) {
         kept[(p0 + j) * step] = s;
-        s.x = fmaf(decay[j], s.x, left[j].x); s.y = fmaf(decay[j], s.y, left[j].y);
-        s.z = fmaf(decay[j], s.z, left[j].z); s.w = fmaf(decay[j], s.w, left[j].w);
+        const float4 l = left[buffer][j];
+        const float d = decay[buffer][j];
+        s.x = fmaf(d, s.x, l.x); s.y = fmaf(d, s.y, l.y); s.z = fmaf(d, s.z, l.z); s.w = fmaf(d, s.w, l.w);
       }
+  };
+  ask(0, 0);
+  for (int p0 = 0; p0 < parts; p0 += 2 * AHEAD) {
+    ask(p0 + AHEAD, 1);
+    walk(p0, 0);
+    ask(p0 + 2 * AHEAD, 0);
+    walk(p0 + AHEAD, 1);
   }
   *whole = s;
 }
@@ -248,18 +270,27 @@ __global__ void __launch_bounds__(THREADS) chunks_kernel(ChunkArgs a) {
   const int inner = a.heads * a.vdim, cols = min(COLS, a.vdim - col0);
   const float* row = a.prepared + (size_t)chunk.first * a.stride;
   const float* x = row + head * a.vdim + col0;
-  sum_logs(a, chunk, head, sums, steps);
-  load_split<N>(c_hi, c_lo, row + inner + (a.groups + group) * a.dim, a.stride, chunk.count, a.dim, nullptr);
-  load_split<N>(b_hi, b_lo, a.starts + (((size_t)blockIdx.z * a.heads + head) * a.vdim + col0) * a.dim, a.dim, cols, a.dim,
-                nullptr);
-  load_split<COLS>(x_hi, x_lo, x, a.stride, chunk.count, cols, nullptr);
+  Tile<N> b;
+  {
+    Tile<N> c;
+    Tile<COLS> xs;
+    c.ask(row + inner + (a.groups + group) * a.dim, a.stride, chunk.count, a.dim);
+    b.ask(a.starts + (((size_t)blockIdx.z * a.heads + head) * a.vdim + col0) * a.dim, a.dim, cols, a.dim);
+    xs.ask(x, a.stride, chunk.count, cols);
+    sum_logs(a, chunk, head, sums, steps);
+    c.put(c_hi, c_lo);
+    b.put(b_hi, b_lo);
+    xs.put(x_hi, x_lo);
+  }
+  b.ask(row + inner + group * a.dim, a.stride, chunk.count, a.dim);  // (on its way while the products with S run)
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, mat = lane >> 3, g = lane >> 2, t = lane & 3;
+  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, mat = lane >> 3, g = lane >> 2, t = lane & 3;
+  const int v0 = (threadIdx.x >> 7) * (COLS / 2);  // the warp's columns
   const int c_at = (warp * 16 + (lane & 15)) * LDN + (lane >> 4) * 8;       // the left operand's sixteen tokens
   const int b_at = ((mat >> 1) * 8 + (lane & 7)) * LDN + (mat & 1) * 8;     // sixteen rows of a right operand
-  float acc[COLS / 8][4];
+  float acc[COLS / 16][4];
 #pragma unroll
-  for (int i = 0; i < COLS / 8; ++i)
+  for (int i = 0; i < COLS / 16; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
   // what the state in front of the chunk answers
@@ -269,22 +300,22 @@ __global__ void __launch_bounds__(THREADS) chunks_kernel(ChunkArgs a) {
     ldmatrix_x4(ch, c_hi + c_at + k * 16);
     ldmatrix_x4(cl, c_lo + c_at + k * 16);
 #pragma unroll
-    for (int n = 0; n < COLS / 16; ++n) {
+    for (int n = 0; n < COLS / 32; ++n) {
       unsigned sh[4], sl[4];
-      ldmatrix_x4(sh, b_hi + b_at + n * 16 * LDN + k * 16);
-      ldmatrix_x4(sl, b_lo + b_at + n * 16 * LDN + k * 16);
+      ldmatrix_x4(sh, b_hi + b_at + (v0 + n * 16) * LDN + k * 16);
+      ldmatrix_x4(sl, b_lo + b_at + (v0 + n * 16) * LDN + k * 16);
       mma_split(acc[2 * n], acc[2 * n + 1], ch, cl, sh, sl);
     }
   }
   const double own[2] = {sums[warp * 16 + g], sums[warp * 16 + g + 8]};  // this thread's two tokens
   const float reach[2] = {expf((float)own[0]), expf((float)own[1])};
 #pragma unroll
-  for (int i = 0; i < COLS / 8; ++i) {
+  for (int i = 0; i < COLS / 16; ++i) {
     acc[i][0] *= reach[0]; acc[i][1] *= reach[0];
     acc[i][2] *= reach[1]; acc[i][3] *= reach[1];
   }
   __syncthreads();  // S has been read by all
-  load_split<N>(b_hi, b_lo, row + inner + group * a.dim, a.stride, chunk.count, a.dim, nullptr);
+  b.put(b_hi, b_lo);
   __syncthreads();
   // the chunk's own tokens, sixteen at a time and none behind the warp's last
 #pragma unroll
@@ -319,9 +350,9 @@ __global__ void __launch_bounds__(THREADS) chunks_kernel(ChunkArgs a) {
         split2(p[0], p[1], ph[2 * i + half], pl[2 * i + half]);
       }
 #pragma unroll
-    for (int n = 0; n < COLS / 16; ++n) {
+    for (int n = 0; n < COLS / 32; ++n) {
       unsigned xh[4], xl[4];
-      const int at = (j * 16 + (mat & 1) * 8 + (lane & 7)) * LDX + n * 16 + (mat >> 1) * 8;
+      const int at = (j * 16 + (mat & 1) * 8 + (lane & 7)) * LDX + v0 + n * 16 + (mat >> 1) * 8;
       ldmatrix_x4_trans(xh, x_hi + at);
       ldmatrix_x4_trans(xl, x_lo + at);
       mma_split(acc[2 * n], acc[2 * n + 1], ph, pl, xh, xl);
@@ -335,8 +366,8 @@ __global__ void __launch_bounds__(THREADS) chunks_kernel(ChunkArgs a) {
     float* dst = a.out + (size_t)(chunk.first + token) * inner + head * a.vdim + col0;
     const float* own_x = x + (size_t)token * a.stride;
 #pragma unroll
-    for (int i = 0; i < COLS / 8; ++i) {
-      const int c = i * 8 + t * 2;
+    for (int i = 0; i < COLS / 16; ++i) {
+      const int c = v0 + i * 8 + t * 2;
       if (c >= cols) continue;
       const float2 xv = *reinterpret_cast<const float2*>(own_x + c);
       *reinterpret_cast<float2*>(dst + c) = make_float2(fmaf(share, xv.x, acc[i][2 * half]),
@@ -359,7 +390,7 @@ int launch(const ChunkArgs& a, int sequences, cudaStream_t stream) {
   const dim3 grid((a.vdim + COLS - 1) / COLS, a.heads, sequences * a.chunks);
   int status = dllm_launch_pdl(left_kernel<N>, grid, dim3(THREADS), left_bytes, stream, a);
   if (status != DLLM_OK) return status;
-  status = dllm_launch_pdl(starts_kernel, dim3((a.vdim * a.dim / 4 + 255) / 256, a.heads, sequences), dim3(256), 0, stream,
+  status = dllm_launch_pdl(starts_kernel, dim3((a.vdim * a.dim / 4 + 127) / 128, a.heads, sequences), dim3(128), 0, stream,
                            a);
   if (status != DLLM_OK) return status;
   return dllm_launch_pdl(chunks_kernel<N>, grid, dim3(THREADS), chunk_bytes, stream, a);
