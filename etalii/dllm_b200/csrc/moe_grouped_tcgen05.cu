@@ -177,7 +177,8 @@ __global__ void __launch_bounds__(THREADS, 1) grouped_tcgen05_kernel(const __gri
             __nv_bfloat162* po = reinterpret_cast<__nv_bfloat162*>(&o);
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-              po[j] = __floats2bfloat162_rn(plain_activation(f[i + 2 * j], g.kind), plain_activation(f[i + 2 * j + 1], g.kind));
+              po[j] = __floats2bfloat162_rn(plain_activation(f[i + 2 * j], g.kind),
+                                            plain_activation(f[i + 2 * j + 1], g.kind));
             if (n + i + 8 <= g.n) *reinterpret_cast<uint4*>(dst + i) = o;
           }
         } else {  // (gate at even columns, up at odd ones; n is a multiple of 16)
@@ -213,7 +214,8 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(uint4* __restrict__ row
 template <int EPI>
 int launch(const void* a, const void* w, const GroupedArgs& g, int pairs, int* status, cudaStream_t stream) {
   if ((long long)g.experts * g.n > 0x7fffffffll) return DLLM_UNSUPPORTED_SIZE;
-  if (status == nullptr || (((uintptr_t)a | (uintptr_t)w | (uintptr_t)g.act | (uintptr_t)g.y) & 15)) return DLLM_BAD_ARGUMENT;
+  if (status == nullptr || (((uintptr_t)a | (uintptr_t)w | (uintptr_t)g.act | (uintptr_t)g.y) & 15))
+    return DLLM_BAD_ARGUMENT;
   alignas(64) CUtensorMap map_a, map_w;
   if (!make_map(&map_a, a, pairs, g.k, BM) || !make_map(&map_w, w, (long long)g.experts * g.n, g.k, BN))
     return DLLM_LAUNCH_FAILED;
@@ -222,7 +224,8 @@ int launch(const void* a, const void* w, const GroupedArgs& g, int pairs, int* s
     int device = 0;
     if (cudaGetDevice(&device) != cudaSuccess ||
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess || sms <= 0 ||
-        cudaFuncSetAttribute(grouped_tcgen05_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess) {
+        cudaFuncSetAttribute(grouped_tcgen05_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) !=
+            cudaSuccess) {
       sms = 0;
       return DLLM_LAUNCH_FAILED;
     }
@@ -260,7 +263,8 @@ DLLM_EXPORT int dllm_moe_grouped_tcgen05_up(void* act, const void* rows, int wid
   if (!act || !rows || !w_up || !offsets || kind < 0 || kind > 3) return DLLM_BAD_ARGUMENT;
   const GroupedArgs g = {kind == 0 ? 2 * ff : ff, width, experts, offsets, nullptr, (bf16*)act, nullptr, limit, alpha, shift,
                          kind};
-  return kind == 0 ? launch<EPI_GLU>(rows, w_up, g, pairs, status, stream) : launch<EPI_ACT>(rows, w_up, g, pairs, status, stream);
+  return kind == 0 ? launch<EPI_GLU>(rows, w_up, g, pairs, status, stream)
+                   : launch<EPI_ACT>(rows, w_up, g, pairs, status, stream);
 }
 
 // y [pairs, width] float32 by pair from act [pairs, ff] in expert order; w_down [experts, width, ff].

@@ -22,7 +22,8 @@
 
 namespace {
 typedef __nv_bfloat16 bf16;
-constexpr int CHUNK = 64, COLS = 64, WARPS = 8, THREADS = WARPS * 32;  // (warps: four of sixteen rows, two halves of columns)
+// (a block's warps: four times sixteen rows of a tile, two halves of its columns)
+constexpr int CHUNK = 64, COLS = 64, WARPS = 8, THREADS = WARPS * 32;
 constexpr int LDX = COLS + 8;
 
 struct ChunkArgs {
@@ -199,7 +200,8 @@ __global__ void __launch_bounds__(THREADS) left_kernel(ChunkArgs a) {
 #pragma unroll
     for (int i = 0; i < N / 16; ++i) {
       const int n = n0 + i * 8 + (lane & 3) * 2;
-      if (n < a.dim) *reinterpret_cast<float2*>(dst + (size_t)col * a.dim + n) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
+      if (n < a.dim)
+        *reinterpret_cast<float2*>(dst + (size_t)col * a.dim + n) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
     }
   }
   if (blockIdx.x == 0 && threadIdx.x == 0) a.decays[(size_t)blockIdx.z * a.heads + head] = expf((float)sums[CHUNK - 1]);

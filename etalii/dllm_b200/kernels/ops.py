@@ -255,7 +255,8 @@ _functions: dict[tuple[str, str], ctypes._CFuncPtr] = {}
 
 
 launches = 0
-"""How many kernels this module has launched (every call below launches exactly one)."""
+"""How many calls below have launched (nearly every call launches one kernel; those over several stretches of a step count
+once)."""
 
 trace: list | None = None
 """A list while a measurement wants every launch timed: each launch appends (name, CUDA event recorded behind it).
@@ -1269,7 +1270,7 @@ def moe_grouped_supported(tokens: int, dtype, width: int, ff: int) -> bool:
 MOE_TCGEN05_FROM = 1 << 17
 """Values of an expert's matrix from which a grouped step's products run on the 5th-generation tensor cores: below, tiles of
 128 x 256 are mostly empty (the products of 2,048 tokens, two of eight experts of 4096 x 2752: 250 us against 689, of 1024 x
-704: 57 against 81; of 128 tokens and 2048 x 1408: 55 against 87; of 1,117 tokens and 320 x 64: 33 against 28)."""
+704: 57 against 81; of 128 tokens and 2048 x 1408: 55 against 87; matrices of a few tens of thousands of values lose up to a fifth)."""
 
 
 def moe_tcgen05_supported(width: int, ff: int) -> bool:

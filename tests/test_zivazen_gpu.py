@@ -613,7 +613,7 @@ LEFT_SHAPES = {
     "unequal": _left(3, 1, 10, 14, 9, 4),
     "odd_values": _left(5, 5, 4, 7, 70, None),
     "squares": _left(6, 3, 64, 64, 33, 64, scale=0.12),
-    "half_turned": _left(6, 3, 128, 128, 50, 64, scale=0.08),
+    "half_turned": _left(4, 1, 128, 128, 50, 96, scale=0.08),
     "no_window": _left(3, 3, 48, 48, 0, 48, scale=0.15),
     "window_of_one": _left(2, 1, 32, 32, 1, 32),
     "beyond_tiles": _left(2, 1, 136, 200, 60, 100, scale=0.1),
@@ -885,7 +885,7 @@ class NestedHarness(PartHarness):
 
 PARALLEL_SHAPES = {
     "tiles": C.parallel(4, 1, 64, 64, 100, 64, 0.12, (6, 32, 32, 2, 4, 3)),
-    "half_turned": C.parallel(6, 3, 128, 128, 50, 64, 0.08, (6, 32, 32, 1, 3, 1), 0.8, 0.5),
+    "half_turned": C.parallel(4, 2, 112, 112, 50, 48, 0.09, (8, 24, 40, 4, 2, 2), 0.9, 0.6),
     "values_of_their_own": C.parallel(4, 2, 24, 40, 33, 8, 0.2, (4, 12, 10, 2, 3, 2), 1.0, 2.0),
     "rows_that_end_anywhere": C.parallel(3, 1, 10, 14, 9, 4, 0.3, (6, 7, 9, 3, 1, 1)),
     "odd_inner": C.parallel(2, 2, 32, 32, 40, 32, 0.2, (3, 7, 9, 1, 2, 3), 0.3, -0.9),
